@@ -64,6 +64,13 @@ class AttentionSpec:
     weights of that size (slots "q_norm" [heads * head_dim], "k_norm" [kv_heads * head_dim]), before the rotation.
     values "keys": there is no value projection; a value head is its key head as projected, before norm and rotation.
     head_gate: head h's output is multiplied by sigmoid(g_h . x), one number a head (slot "wg", [heads, hidden]).
+    bias: q, k and v have biases, added in the projection (slots "bq", "bk", "bv"). q_temperature (coef, every): after its
+    norm, q at position p is multiplied by 1 + coef * ln(floor((p + 1) / every) + 1).
+    weights "sigmoid": there is no softmax; the weight of a key a token sees is sigmoid(score), each key for itself and
+    not normalized over the keys, in float32. Only such weights take: slopes, a number per head, slopes[h] * (i - j) taken
+    off the score of key j seen from i (after the cap); shift, a learned number per head (slot "shift", [heads]) added to
+    the score; mix, the heads' weights mixed before they meet the values, w_h <- sum_g M[h, g] w_g (slot "mix",
+    [heads, heads]), head h's mixed weights applied to the values of its own kv head.
     """
     hidden: int
     n_heads: int
@@ -83,6 +90,12 @@ class AttentionSpec:
     norm_over: str = "head"
     values: str = "own"
     head_gate: bool = False
+    bias: bool = False
+    q_temperature: Optional[tuple] = None
+    weights: str = "softmax"
+    slopes: Optional[tuple] = None
+    shift: bool = False
+    mix: bool = False
     kind: str = "attention"
 
 
@@ -229,6 +242,20 @@ class WkvSpec:
 
 
 @dataclass(frozen=True)
+class GatedAverageSpec:
+    """A recurrent mixer: a running average per channel whose gate and candidate read the current token alone (a minimal
+    gated recurrent unit).
+
+    z = sigmoid(Wz x + bz), u = Wu x + bu, both [width]; the candidate c is u + 1/2 where u >= 0, sigmoid(u) where u < 0
+    (positive, and continuous at 0). Channel by channel S <- (1 - z) S + z c, float32, zero at a sequence's start; the
+    output is Wo (S * silu(Wg x)).
+    """
+    hidden: int
+    width: int
+    kind: str = "gated_average"
+
+
+@dataclass(frozen=True)
 class ExpertSpec:
     """A small feed-forward: down(act(up(x))), or, with activation "silu_gated", down(silu(gate(x)) * up(x))."""
     inter: int
@@ -265,7 +292,7 @@ class RoutedMLPSpec:
 
 @dataclass(frozen=True)
 class GatedMLPSpec:
-    """down(act(gate(x)) * up(x)) as src/model.c:274-282, 307-309."""
+    """down(act(gate(x)) * up(x)) as src/model.c:274-282, 307-309; act "silu" or "relu"."""
     hidden: int
     inter: int
     activation: str = "silu"
@@ -287,6 +314,19 @@ class BlockSpec:
     @property
     def kind(self):
         return self.arrangement
+
+
+@dataclass(frozen=True)
+class SandwichBlockSpec:
+    """One layer with a norm before and after each branch: x += mixer_post_norm(mixer(mixer_norm(x))), then
+    x += ffn_post_norm(ffn(ffn_norm(x))). ffn None: the mixer's branch alone."""
+    mixer_norm: object
+    mixer: object
+    mixer_post_norm: object
+    ffn_norm: object = None
+    ffn: object = None
+    ffn_post_norm: object = None
+    kind: str = "sandwich_norm"
 
 
 @dataclass(frozen=True)
@@ -327,6 +367,14 @@ class PositionEmbeddingSpec:
     add it to the stream again (ScheduleEntry.rejoin)."""
     max_positions: int
     keep: bool = False
+
+
+@dataclass(frozen=True)
+class SinusoidEmbeddingSpec:
+    """The frame "sinusoids": x = table[token] + s(position), a fixed vector per position: element 2i of s(p) is
+    sin(p * base^(-2i / hidden)), element 2i + 1 the cosine of the same angle. The logits are multiplied by logit_scale."""
+    base: float = 10000.0
+    logit_scale: float = 1.0
 
 
 @dataclass(frozen=True)

@@ -171,6 +171,12 @@ __device__ __forceinline__ float silu_mul_fast(float gate, float up) {
     return gate * r * up;
 }
 
+// The activation of a gated feed-forward times its up value, in the bfloat16 path: ABK_SILU (above) or ABK_RELU.
+enum { ABK_SILU = 0, ABK_RELU = 1 };
+__device__ __forceinline__ float gated_mul(int act, float gate, float up) {
+    return act == ABK_RELU ? fmaxf(gate, 0.0f) * up : silu_mul_fast(gate, up);
+}
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

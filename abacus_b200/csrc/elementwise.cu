@@ -32,6 +32,46 @@ extern "C" int abk_embed(const int *tokens, const void *table, int table_dtype, 
     return ABK_LAUNCH_RESULT();
 }
 
+// x[t, :] = float(table[tokens[t], :]) + s(position of t): a fixed sinusoid per position, element 2i the sine and element
+// 2i + 1 the cosine of position * f_i. The angle's sine and cosine come from two small float32 tables made in float64,
+// position = 256 a + b: coarse [a][i] = (sin, cos)(256 a f_i), fine [b][i] = (sin, cos)(b f_i), joined by the sum of angles.
+template <typename TW>
+__global__ void embed_sinusoids_kernel(const int *__restrict__ tokens, const int *__restrict__ token_seq, const int *__restrict__ token_pos,
+                                       const TW *__restrict__ table, const float2 *__restrict__ coarse, const float2 *__restrict__ fine,
+                                       float *__restrict__ x, int d, int vocab, int n_positions, int *status) {
+    pdl_wait();
+    const int t = blockIdx.x;
+    const bool pad = token_seq[t] < 0;
+    const int tok = pad ? 0 : tokens[t], pos = pad ? 0 : token_pos[t];
+    const bool bad = tok < 0 || tok >= vocab || pos < 0 || pos >= n_positions;
+    if (bad && threadIdx.x == 0) atomicOr(status, 1);
+    const TW *row = table + (long long)(bad ? 0 : tok) * d;
+    float *out = x + (long long)t * d;
+    const int half = (d + 1) / 2;
+    const float2 *ca = coarse + (long long)(bad ? 0 : pos >> 8) * half, *fb = fine + (long long)(bad ? 0 : pos & 255) * half;
+    for (int i = threadIdx.x; i < half; i += blockDim.x) {
+        const float2 a = ca[i], b = fb[i];
+        const float sn = fmaf(a.x, b.y, a.y * b.x), cs = fmaf(a.y, b.y, -a.x * b.x);
+        out[2 * i] = bad || pad ? 0.0f : to_float(row[2 * i]) + sn;
+        if (2 * i + 1 < d) out[2 * i + 1] = bad || pad ? 0.0f : to_float(row[2 * i + 1]) + cs;
+    }
+}
+
+extern "C" int abk_embed_sinusoids(const int *tokens, const int *token_seq, const int *token_pos, const void *table, int table_dtype,
+                                   const float *coarse, const float *fine, float *x, int n_tokens, int d, int vocab, int n_positions,
+                                   int *status, void *stream) {
+    if (n_tokens <= 0) return 0;
+    const int threads = d >= 1024 ? 256 : 128;
+    cudaStream_t s = (cudaStream_t)stream;
+    if (table_dtype == ABK_BF16)
+        abk_launch(embed_sinusoids_kernel<__nv_bfloat16>, dim3(n_tokens), dim3(threads), 0, s, tokens, token_seq, token_pos, (const __nv_bfloat16 *)table,
+                   (const float2 *)coarse, (const float2 *)fine, x, d, vocab, n_positions, status);
+    else
+        abk_launch(embed_sinusoids_kernel<float>, dim3(n_tokens), dim3(threads), 0, s, tokens, token_seq, token_pos, (const float *)table,
+                   (const float2 *)coarse, (const float2 *)fine, x, d, vocab, n_positions, status);
+    return ABK_LAUNCH_RESULT();
+}
+
 // ------------------------------------------------------------------ residual add + RMSNorm
 // x += y (when y is given); out = w * (x / sqrt(mean(x^2) + eps))      (src/model.c:238-244, 164-169)
 // With `rows`, output row r is made from row rows[r] of x (+ y) and x is left as it is: the
@@ -139,13 +179,137 @@ extern "C" int abk_add_rmsnorm(float *x, const float *y, const float *w, void *o
     return ABK_LAUNCH_RESULT();
 }
 
+// ------------------------------------------------------------------ a branch's output normed, added, and the stream normed
+// x += wy * (y / sqrt(mean(y^2) + eps_y)); out = w * (x / sqrt(mean(x^2) + eps)): the norm behind a branch, the residual
+// sum and the norm ahead of the next branch. y null: nothing is added. With `rows`, output row r is made from row rows[r]
+// and x is left as it is.
+template <typename TO>
+__global__ void __launch_bounds__(256) normed_add_rmsnorm_kernel(float *__restrict__ x, const float *__restrict__ y, const float *__restrict__ wy,
+                                                                 const float *__restrict__ w, TO *__restrict__ out, const int *__restrict__ rows,
+                                                                 int d, float eps_y, float eps) {
+    __shared__ float scratch[33];
+    pdl_wait();
+    const int r = blockIdx.x;
+    const long long src = rows ? rows[r] : r;
+    float *xr = x + src * d;
+    const float *yr = y ? y + src * d : nullptr;
+    float sy = 0.0f, scale_y = 0.0f;
+    if (yr) {
+        for (int j = threadIdx.x; j < d; j += blockDim.x) sy = fmaf(yr[j], yr[j], sy);
+        sy = block_sum(sy, scratch);
+        scale_y = 1.0f / sqrtf(sy / (float)d + eps_y);
+    }
+    float ss = 0.0f;
+    for (int j = threadIdx.x; j < d; j += blockDim.x) {
+        float v = xr[j];
+        if (yr) v += wy[j] * (yr[j] * scale_y);
+        if (yr && !rows) xr[j] = v;
+        ss += v * v;
+    }
+    ss = block_sum(ss, scratch);
+    const float scale = 1.0f / sqrtf(ss / (float)d + eps);
+    TO *o = out + (long long)r * d;
+    for (int j = threadIdx.x; j < d; j += blockDim.x) {
+        float v = xr[j];
+        if (yr && rows) v += wy[j] * (yr[j] * scale_y);
+        o[j] = from_float<TO>(w[j] * (v * scale));
+    }
+}
+
+// The sum over a block of 256 threads in two barriers' time fewer than block_sum: every warp leaves its sum, everyone adds
+// the eight in one order. `slots` (8 floats) is not used again by the same kernel.
+__device__ __forceinline__ float block_sum_256(float v, float *slots) {
+    v = warp_sum(v);
+    if ((threadIdx.x & 31) == 0) slots[threadIdx.x >> 5] = v;
+    __syncthreads();
+    const float4 a = *(const float4 *)slots, b = *(const float4 *)(slots + 4);
+    return ((a.x + a.y) + (a.z + a.w)) + ((b.x + b.y) + (b.z + b.w));
+}
+
+// The same with a row in registers (d a multiple of 4 up to 1024 * V, V float4 a thread): both weights come in before
+// pdl_wait(), x and y are read once.
+template <typename TO, int V>
+__global__ void __launch_bounds__(256) normed_add_rmsnorm_row_kernel(float *__restrict__ x, const float *__restrict__ y,
+                                                                     const float *__restrict__ wy, const float *__restrict__ w,
+                                                                     TO *__restrict__ out, const int *__restrict__ rows, int d,
+                                                                     float eps_y, float eps) {
+    __shared__ __align__(16) float slots[16];
+    float4 wv[V], wb[V], v[V], u[V];
+    const float4 zero = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+#pragma unroll
+    for (int i = 0; i < V; i++) {
+        const int j = 4 * (threadIdx.x + 256 * i);
+        wv[i] = j < d ? *(const float4 *)(w + j) : zero;
+        wb[i] = y && j < d ? *(const float4 *)(wy + j) : zero;
+    }
+    pdl_wait();
+    const int r = blockIdx.x;
+    const long long src = rows ? rows[r] : r;
+    float *xr = x + src * d;
+    float sy = 0.0f;
+#pragma unroll
+    for (int i = 0; i < V; i++) {
+        const int j = 4 * (threadIdx.x + 256 * i);
+        v[i] = j < d ? *(const float4 *)(xr + j) : zero;
+        u[i] = y && j < d ? *(const float4 *)(y + src * d + j) : zero;
+        sy += u[i].x * u[i].x + u[i].y * u[i].y + u[i].z * u[i].z + u[i].w * u[i].w;
+    }
+    if (y) {
+        const float scale_y = 1.0f / sqrtf(block_sum_256(sy, slots) / (float)d + eps_y);
+#pragma unroll
+        for (int i = 0; i < V; i++) {
+            const int j = 4 * (threadIdx.x + 256 * i);
+            v[i].x += wb[i].x * (u[i].x * scale_y), v[i].y += wb[i].y * (u[i].y * scale_y);
+            v[i].z += wb[i].z * (u[i].z * scale_y), v[i].w += wb[i].w * (u[i].w * scale_y);
+            if (!rows && j < d) *(float4 *)(xr + j) = v[i];
+        }
+    }
+    float ss = 0.0f;
+#pragma unroll
+    for (int i = 0; i < V; i++) ss += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
+    const float scale = 1.0f / sqrtf(block_sum_256(ss, slots + 8) / (float)d + eps);
+    TO *o = out + (long long)r * d;
+#pragma unroll
+    for (int i = 0; i < V; i++) {
+        const int j = 4 * (threadIdx.x + 256 * i);
+        if (j < d) store4(o + j, wv[i].x * (v[i].x * scale), wv[i].y * (v[i].y * scale), wv[i].z * (v[i].z * scale),
+                          wv[i].w * (v[i].w * scale));
+    }
+}
+
+extern "C" int abk_normed_add_rmsnorm(float *x, const float *y, const float *wy, const float *w, void *out, int out_dtype,
+                                      const int *rows, int n_rows, int d, float eps_y, float eps, void *stream) {
+    if (n_rows <= 0) return 0;
+    if (y && !wy) ABK_REFUSE("normed_add_rmsnorm: a branch's output comes with its norm's weight");
+    cudaStream_t s = (cudaStream_t)stream;
+    const bool aligned = !(((uintptr_t)x | (uintptr_t)y | (uintptr_t)wy | (uintptr_t)w | (uintptr_t)out) & 15);
+    if (d % 4 == 0 && d <= 4096 && aligned) {
+#define NORMED_LAUNCH(TO, V) \
+    abk_launch(normed_add_rmsnorm_row_kernel<TO, V>, dim3(n_rows), dim3(256), 0, s, x, y, wy, w, (TO *)out, rows, d, eps_y, eps)
+#define NORMED_BY_D(TO)                       \
+    if (d <= 1024) NORMED_LAUNCH(TO, 1);      \
+    else if (d <= 2048) NORMED_LAUNCH(TO, 2); \
+    else if (d <= 3072) NORMED_LAUNCH(TO, 3); \
+    else NORMED_LAUNCH(TO, 4);
+        if (out_dtype == ABK_BF16) { NORMED_BY_D(__nv_bfloat16) } else { NORMED_BY_D(float) }
+#undef NORMED_BY_D
+#undef NORMED_LAUNCH
+        return ABK_LAUNCH_RESULT();
+    }
+    if (out_dtype == ABK_BF16)
+        abk_launch(normed_add_rmsnorm_kernel<__nv_bfloat16>, dim3(n_rows), dim3(256), 0, s, x, y, wy, w, (__nv_bfloat16 *)out, rows, d, eps_y, eps);
+    else
+        abk_launch(normed_add_rmsnorm_kernel<float>, dim3(n_rows), dim3(256), 0, s, x, y, wy, w, (float *)out, rows, d, eps_y, eps);
+    return ABK_LAUNCH_RESULT();
+}
+
 // ------------------------------------------------------------------ SwiGLU
 // act[t, j] = silu(gate[t, j]) * up[t, j]                              (src/model.c:274-282)
 // A row of gate_up holds gate and up in turns of `block` columns: gate of features [0, block), up of the same,
 // gate of [block, 2 block), ... With block = inter that is all gates and then all ups (src/model.c:98).
 __device__ __forceinline__ long long gate_column(int j, int block) { return (long long)(j / block) * 2 * block + j % block; }
 template <typename T>
-__global__ void swiglu_kernel(const T *__restrict__ gate_up, T *__restrict__ act, long long total, int inter, int block) {
+__global__ void swiglu_kernel(const T *__restrict__ gate_up, T *__restrict__ act, long long total, int inter, int block, int kind) {
     pdl_wait();
     for (long long e = (long long)blockIdx.x * blockDim.x + threadIdx.x; e < total;
          e += (long long)gridDim.x * blockDim.x) {
@@ -153,13 +317,13 @@ __global__ void swiglu_kernel(const T *__restrict__ gate_up, T *__restrict__ act
         int j = (int)(e - t * inter);
         float g = to_float(gate_up[t * 2 * inter + gate_column(j, block)]);
         float u = to_float(gate_up[t * 2 * inter + gate_column(j, block) + block]);
-        act[e] = from_float<T>(sizeof(T) == 2 ? silu_mul_fast(g, u) : g / (1.0f + expf(-g)) * u);
+        act[e] = from_float<T>(sizeof(T) == 2 || kind != ABK_SILU ? gated_mul(kind, g, u) : g / (1.0f + expf(-g)) * u);
     }
 }
 
 // bfloat16 with inter and block multiples of 8: eight elements a thread, read and written as 16-byte vectors.
 __global__ void swiglu_bf16x8_kernel(const __nv_bfloat16 *__restrict__ gate_up, __nv_bfloat16 *__restrict__ act,
-                                     long long groups, int inter, int block) {
+                                     long long groups, int inter, int block, int kind) {
     pdl_wait();
     const int per_row = inter >> 3;
     for (long long g = (long long)blockIdx.x * blockDim.x + threadIdx.x; g < groups; g += (long long)gridDim.x * blockDim.x) {
@@ -173,13 +337,14 @@ __global__ void swiglu_bf16x8_kernel(const __nv_bfloat16 *__restrict__ gate_up, 
 #pragma unroll
         for (int e = 0; e < 4; e++) {
             float2 gv = __bfloat1622float2(gp[e]), uv = __bfloat1622float2(up[e]);
-            op[e] = __floats2bfloat162_rn(silu_mul_fast(gv.x, uv.x), silu_mul_fast(gv.y, uv.y));
+            op[e] = __floats2bfloat162_rn(gated_mul(kind, gv.x, uv.x), gated_mul(kind, gv.y, uv.y));
         }
         *(uint4 *)(act + t * inter + j) = out;
     }
 }
 
-extern "C" int abk_swiglu(const void *gate_up, void *act, int dtype, int n_tokens, int inter, int block, void *stream) {
+// The same with the activation ABK_SILU or ABK_RELU (relu(gate) * up).
+extern "C" int abk_gated_act(const void *gate_up, void *act, int dtype, int n_tokens, int inter, int block, int kind, void *stream) {
     long long total = (long long)n_tokens * inter;
     if (total <= 0) return 0;
     if (block <= 0 || inter % block) ABK_REFUSE("swiglu: turns of %d columns do not divide %d", block, inter);
@@ -187,7 +352,7 @@ extern "C" int abk_swiglu(const void *gate_up, void *act, int dtype, int n_token
         long long groups = total >> 3, want = (groups + 255) / 256;
         int blocks = (int)(want > abk_sm_count() * 16 ? abk_sm_count() * 16 : want);
         abk_launch(swiglu_bf16x8_kernel, dim3(blocks), dim3(256), 0, (cudaStream_t)stream, (const __nv_bfloat16 *)gate_up,
-                   (__nv_bfloat16 *)act, groups, inter, block);
+                   (__nv_bfloat16 *)act, groups, inter, block, kind);
         return ABK_LAUNCH_RESULT();
     }
     int threads = 256;
@@ -195,10 +360,14 @@ extern "C" int abk_swiglu(const void *gate_up, void *act, int dtype, int n_token
     if (blocks > abk_sm_count() * 32) blocks = abk_sm_count() * 32;
     cudaStream_t s = (cudaStream_t)stream;
     if (dtype == ABK_BF16)
-        abk_launch(swiglu_kernel<__nv_bfloat16>, dim3((int)blocks), dim3(threads), 0, s, (const __nv_bfloat16 *)gate_up, (__nv_bfloat16 *)act, total, inter, block);
+        abk_launch(swiglu_kernel<__nv_bfloat16>, dim3((int)blocks), dim3(threads), 0, s, (const __nv_bfloat16 *)gate_up, (__nv_bfloat16 *)act, total, inter, block, kind);
     else
-        abk_launch(swiglu_kernel<float>, dim3((int)blocks), dim3(threads), 0, s, (const float *)gate_up, (float *)act, total, inter, block);
+        abk_launch(swiglu_kernel<float>, dim3((int)blocks), dim3(threads), 0, s, (const float *)gate_up, (float *)act, total, inter, block, kind);
     return ABK_LAUNCH_RESULT();
+}
+
+extern "C" int abk_swiglu(const void *gate_up, void *act, int dtype, int n_tokens, int inter, int block, void *stream) {
+    return abk_gated_act(gate_up, act, dtype, n_tokens, inter, block, ABK_SILU, stream);
 }
 
 // ------------------------------------------------------------------ q/k/v preparation
@@ -547,7 +716,9 @@ extern "C" int abk_advance_decode(const int *token_seq, int *token_pos, int n_ro
 // ------------------------------------------------------------------ q and k normed over their whole rows, values that are keys
 // Per token: src row [q (heads * hd) | k (kv heads * hd) | ...] as projected; dst row [q | k | v] for the attention
 // kernels. q and k are each normed over their whole row (all heads at once: w * z / sqrt(mean(z^2) + eps), weights of
-// the row's size), then rotated head by head; a value head is its key head as projected, before norm and rotation.
+// the row's size), then rotated head by head; a value head is its key head as projected, before norm and rotation, or
+// (v_dim > 0) has a projection of its own, in the src row behind k. Options: biases added to the row as projected; a query
+// temperature, q times 1 + coef * ln(floor((position + 1) / every) + 1).
 // k and v go to the paged cache. A CTA a token; float32 arithmetic.
 struct QkvWhole {
     const void *src;
@@ -562,6 +733,9 @@ struct QkvWhole {
     void *k_pool, *v_pool;
     PagedCache cache;
     const int *token_seq, *token_pos, *seq_slot, *seq_len_after;
+    int v_dim;                     // 0: values are keys as projected; else the size of a value head of its own
+    const float *bias;             // [row as projected], or null
+    float temp_coef, temp_every;   // temp_every > 0: the query temperature
 };
 
 // VEC elements at a time: 8 for bfloat16 rows whose heads are a multiple of 8 (16-byte pieces), else 1.
@@ -607,27 +781,35 @@ template <typename T, int VEC> __global__ void __launch_bounds__(256) qkv_prep_w
     T *dst = (T *)p.dst + (long long)t * p.ldd;
     const bool keeps = p.k_pool && cache_keeps(p.cache, pos, p.seq_len_after[seq]);
     const int page = keeps ? cache_page(p.cache, p.seq_slot[seq], pos) : 0;
+    const int vd = p.v_dim > 0 ? p.v_dim : hd, own_v = p.v_dim > 0 ? p.n_kv_heads * vd : 0;
     float sq = 0.0f, sk = 0.0f;
-    for (int j = tid * VEC; j < q_size + k_size; j += 256 * VEC) {
+    for (int j = tid * VEC; j < q_size + k_size + own_v; j += 256 * VEC) {
         float f[VEC];
         whole_load<T, VEC>(src + j, f);
+        if (p.bias) {
+#pragma unroll
+            for (int e = 0; e < VEC; e++) f[e] += p.bias[j + e];
+        }
+        const int jv = own_v ? j - q_size - k_size : j - q_size;  // its place among the values, if it is one
+        if (jv >= 0)  // a value, stored to the row and to the cache as it is
+            whole_store<T, VEC>(dst + q_size + k_size + jv,
+                                keeps ? (T *)p.v_pool + cache_offset(p.cache, page, jv / vd, p.n_kv_heads, pos, vd) + jv % vd : nullptr, f);
+        if (own_v && jv >= 0) continue;
         float ss = 0.0f;
 #pragma unroll
         for (int e = 0; e < VEC; e++) whole[j + e] = f[e], ss = fmaf(f[e], f[e], ss);
         if (j < q_size) sq += ss;
-        else {  // a key as projected is its value: to the row and to the cache as it is
-            sk += ss;
-            const int jk = j - q_size;
-            whole_store<T, VEC>(dst + q_size + k_size + jk,
-                                keeps ? (T *)p.v_pool + cache_offset(p.cache, page, jk / hd, p.n_kv_heads, pos, hd) + jk % hd : nullptr, f);
-        }
+        else sk += ss;
     }
     sq = block_sum(sq, scratch);
     sk = block_sum(sk, scratch);
+    const float heat = p.temp_every > 0.0f ? fmaf(p.temp_coef, logf(floorf((float)(pos + 1) / p.temp_every) + 1.0f), 1.0f) : 1.0f;
     if (p.q_norm) {
-        const float rq = 1.0f / sqrtf(sq / (float)q_size + p.eps), rk = 1.0f / sqrtf(sk / (float)k_size + p.eps);
+        const float rq = heat / sqrtf(sq / (float)q_size + p.eps), rk = 1.0f / sqrtf(sk / (float)k_size + p.eps);
         for (int j = tid; j < q_size + k_size; j += 256)
             whole[j] = j < q_size ? p.q_norm[j] * (whole[j] * rq) : p.k_norm[j - q_size] * (whole[j] * rk);
+    } else if (p.temp_every > 0.0f) {
+        for (int j = tid; j < q_size; j += 256) whole[j] *= heat;
     }
     __syncthreads();
     if (p.cos) {
@@ -650,7 +832,8 @@ template <typename T, int VEC> __global__ void __launch_bounds__(256) qkv_prep_w
 }
 
 extern "C" int abk_qkv_prep_whole(const void *src, long long lds, void *dst, long long ldd, int dtype, int n_tokens, int n_heads,
-                                  int n_kv_heads, int head_dim, const int *token_seq, const int *token_pos, const int *seq_slot,
+                                  int n_kv_heads, int head_dim, int v_dim, const float *bias, float temp_coef, float temp_every,
+                                  const int *token_seq, const int *token_pos, const int *seq_slot,
                                   const int *seq_len_after, const float *q_norm, const float *k_norm, float eps,
                                   const float *cos, const float *sin, int rotary_dim, int interleaved, void *k_pool,
                                   void *v_pool, const int *page_table, int table_width, int ring_pages, int tokens_per_page,
@@ -668,8 +851,9 @@ extern "C" int abk_qkv_prep_whole(const void *src, long long lds, void *dst, lon
     p.cache.page_table = page_table, p.cache.table_width = table_width, p.cache.ring_pages = ring_pages;
     p.cache.tokens_per_page = tokens_per_page, p.cache.pinned_pages = pinned_pages;
     p.token_seq = token_seq, p.token_pos = token_pos, p.seq_slot = seq_slot, p.seq_len_after = seq_len_after;
+    p.v_dim = v_dim, p.bias = bias, p.temp_coef = temp_coef, p.temp_every = temp_every;
     cudaStream_t s = (cudaStream_t)stream;
-    const bool pieces = dtype == ABK_BF16 && head_dim % 8 == 0 && lds % 8 == 0 && ldd % 8 == 0 &&
+    const bool pieces = dtype == ABK_BF16 && head_dim % 8 == 0 && v_dim % 8 == 0 && lds % 8 == 0 && ldd % 8 == 0 &&
                         ((uintptr_t)src | (uintptr_t)dst | (uintptr_t)k_pool | (uintptr_t)v_pool) % 16 == 0;
 #define WHOLE_LAUNCH(KERNEL)                                                            \
     do {                                                                                \

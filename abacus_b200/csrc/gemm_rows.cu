@@ -55,7 +55,8 @@ template <int NT, int TILE, bool GATED, typename TO>
 __global__ void __launch_bounds__(ROWS_THREADS) gemm_rows_kernel(const __nv_bfloat16 *__restrict__ x,
                                                                  const __nv_bfloat16 *__restrict__ w, TO *__restrict__ out,
                                                                  int M, int N, int K, long long ldx, long long ldw,
-                                                                 long long ldo, int block, long long x_plane, int tanh_from) {
+                                                                 long long ldo, int block, long long x_plane, int tanh_from,
+                                                                 int act) {
     __shared__ float part[ROWS_WARPS][16][8 * NT + 1];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, r = lane >> 2, c = lane & 3;
     const int ranks = (int)tc::cluster_size(), rank = (int)tc::cluster_rank();  // the cluster splits K
@@ -161,7 +162,7 @@ __global__ void __launch_bounds__(ROWS_THREADS) gemm_rows_kernel(const __nv_bflo
                 // gate and up pass through bfloat16, as they do where they are stored between the product
                 // and the activation (larger steps): a token's result is the same on either way
                 sum = __bfloat162float(__float2bfloat16_rn(sum)), up = __bfloat162float(__float2bfloat16_rn(up));
-                sum = silu_mul_fast(sum, up);
+                sum = gated_mul(act, sum, up);
             }
             if (!GATED && n0 + row >= tanh_from) sum = tanhf(sum);  // (tanh_from beyond N: no feature)
             out[(long long)token * ldo + n0 + row] = from_float<TO>(sum);
@@ -193,7 +194,7 @@ static int gemm_rows_launch(const void *x, const void *w, void *out, int out_dty
     const __nv_bfloat16 *xb = (const __nv_bfloat16 *)x, *wb = (const __nv_bfloat16 *)w;
 #define ROWS_LAUNCH(NT, TILE, TO)                                                                                     \
     abk_launch_clusters(gemm_rows_kernel<NT, TILE, false, TO>, grid, dim3(ROWS_THREADS), 0, s, ranks, xb, wb, (TO *)out, M, \
-                        N, K, ldx, ldw, ldo, block, x_plane, tanh_from)
+                        N, K, ldx, ldw, ldo, block, x_plane, tanh_from, 0)
 #define ROWS_BY_M(TO)                                                                     \
     if (M <= 8) { if (narrow) ROWS_LAUNCH(1, 8, TO); else ROWS_LAUNCH(1, 16, TO); }       \
     else if (M <= 16) { if (narrow) ROWS_LAUNCH(2, 8, TO); else ROWS_LAUNCH(2, 16, TO); } \
@@ -221,8 +222,9 @@ extern "C" int abk_gemm_rows_planes(const void *x, const void *w, void *out, int
 // act[M, N] = silu(x . w_gate^T) * (x . w_up^T) where w [2 N, K] holds gate and up rows in turns of `block`
 // rows (a multiple of 8 that divides N; N itself: all gates, then all ups).
 // x, w bfloat16; act bfloat16. M <= 64, K a multiple of 32.
-extern "C" int abk_gemm_rows_swiglu(const void *x, const void *w, void *act, int M, int N, int K, long long ldx,
-                                    long long ldw, long long ldo, int block, void *stream) {
+// kind: the activation, ABK_SILU or ABK_RELU (relu(gate) * up).
+extern "C" int abk_gemm_rows_gated(const void *x, const void *w, void *act, int M, int N, int K, long long ldx,
+                                   long long ldw, long long ldo, int block, int kind, void *stream) {
     if (M <= 0 || N <= 0) return 0;
     if (block <= 0 || N % block || (block % 8 && block != N)) ABK_REFUSE("gemm_rows_swiglu: turns of %d rows do not fit %d features", block, N);
     if (M > 64) ABK_REFUSE("gemm_rows_swiglu: %d rows are more than 64", M);
@@ -232,11 +234,16 @@ extern "C" int abk_gemm_rows_swiglu(const void *x, const void *w, void *act, int
     cudaStream_t s = (cudaStream_t)stream;
     const __nv_bfloat16 *xb = (const __nv_bfloat16 *)x, *wb = (const __nv_bfloat16 *)w;
 #define GATED_LAUNCH(NT) \
-    abk_launch(gemm_rows_kernel<NT, 8, true, __nv_bfloat16>, grid, dim3(ROWS_THREADS), 0, s, xb, wb, (__nv_bfloat16 *)act, M, N, K, ldx, ldw, ldo, block, 0LL, 0x7fffffff)
+    abk_launch(gemm_rows_kernel<NT, 8, true, __nv_bfloat16>, grid, dim3(ROWS_THREADS), 0, s, xb, wb, (__nv_bfloat16 *)act, M, N, K, ldx, ldw, ldo, block, 0LL, 0x7fffffff, kind)
     if (M <= 8) GATED_LAUNCH(1);
     else if (M <= 16) GATED_LAUNCH(2);
     else if (M <= 32) GATED_LAUNCH(4);
     else GATED_LAUNCH(8);
 #undef GATED_LAUNCH
     return ABK_LAUNCH_RESULT();
+}
+
+extern "C" int abk_gemm_rows_swiglu(const void *x, const void *w, void *act, int M, int N, int K, long long ldx,
+                                    long long ldw, long long ldo, int block, void *stream) {
+    return abk_gemm_rows_gated(x, w, act, M, N, K, ldx, ldw, ldo, block, ABK_SILU, stream);
 }

@@ -49,6 +49,7 @@ struct GemmTc {
     int *status;
     int vec;  // stride_q == 1 and every 16-column run of a row starts on a 16-byte boundary
     int in_cluster;  // the splits of a tile are a thread-block cluster and add up through distributed shared memory
+    int gated_act = ABK_SILU;  // what EPI_GATED applies to the gate: ABK_SILU or ABK_RELU
     int weights_are_p;  // which operand is nobody's output (the weights): its first stages are asked for before pdl_wait()
 };
 
@@ -531,7 +532,7 @@ __global__ void __launch_bounds__(EPI == EPI_QKV ? QKV_THREADS : GEMM_THREADS) g
                     for (int j = 0; j < 32; j++) {
                         const float gate = __bfloat162float(__float2bfloat16_rn(__uint_as_float(gv[j])));
                         const float up = __bfloat162float(__float2bfloat16_rn(__uint_as_float(uv[j])));
-                        gv[j] = __float_as_uint(silu_mul_fast(gate, up));
+                        gv[j] = __float_as_uint(gated_mul(g.gated_act, gate, up));
                     }
                     if (p < g.P && f0 + c0 + 32 <= g.Q) {
                         store16(out + (long long)p * g.stride_p + f0 + c0, gv);
@@ -721,7 +722,7 @@ __global__ void __launch_bounds__(EPI == EPI_QKV ? QKV_THREADS : GEMM_THREADS) g
                     for (int j = 0; j < 32; j++) {
                         const float gate = __bfloat162float(__float2bfloat16_rn(__uint_as_float(gv[j])));
                         const float up = __bfloat162float(__float2bfloat16_rn(__uint_as_float(uv[j])));
-                        gv[j] = __float_as_uint(silu_mul_fast(gate, up));
+                        gv[j] = __float_as_uint(gated_mul(g.gated_act, gate, up));
                     }
                     if (p < g.P && f0 + c0 + 32 <= g.Q) {
                         store16(out + (long long)p * g.stride_p + f0 + c0, gv);
@@ -877,8 +878,9 @@ static int launch_persistent(const CUtensorMap &mp, const CUtensorMap &mq, const
 // act[M, N] = silu(x . gate^T) * (x . up^T), w [2 N, K] holding gate and up rows in turns of 128: the persistent
 // kernel with the activation in its epilogue. Many rows only (more than 256), N a multiple of 128, act bfloat16
 // with 16-byte aligned rows; other shapes are refused (the caller multiplies and activates in two steps).
-extern "C" int abk_gemm_tc_swiglu(const void *x, const void *w, void *act, int M, int N, int K, long long ldx,
-                                  long long ldw, long long ldo, int *status, void *stream) {
+// kind: the activation, ABK_SILU or ABK_RELU (relu(gate) * up).
+extern "C" int abk_gemm_tc_gated(const void *x, const void *w, void *act, int M, int N, int K, long long ldx,
+                                 long long ldw, long long ldo, int kind, int *status, void *stream) {
     if (M <= 0 || N <= 0) return 0;
     if (M <= 256 || N % 128 || K <= 0 || K % 8 || ldx % 8 || ldw % 8 || ldo % 8 || (((uintptr_t)x | (uintptr_t)w | (uintptr_t)act) & 15))
         ABK_REFUSE("gemm_tc_swiglu: %d rows, %d features, K = %d are not what the fused kernel takes", M, N, K);
@@ -887,7 +889,7 @@ extern "C" int abk_gemm_tc_swiglu(const void *x, const void *w, void *act, int M
     if (!rc) rc = tensor_map(w, 2LL * N, K, ldw, 256, &mw);
     if (rc) return rc;
     GemmTc g;
-    g.out = act, g.P = M, g.Q = N, g.K = K, g.stride_p = ldo, g.stride_q = 1;
+    g.out = act, g.P = M, g.Q = N, g.K = K, g.stride_p = ldo, g.stride_q = 1, g.gated_act = kind;
     g.k_blocks = (K + TILE_K - 1) / TILE_K, g.k_blocks_per_split = g.k_blocks, g.splits = 1;
     g.partials = nullptr, g.tickets = nullptr, g.status = status, g.vec = 1, g.in_cluster = 0, g.weights_are_p = 0;
     if (pairs_win(M, 2 * N) && !abk_pairs_off()) {
@@ -899,6 +901,11 @@ extern "C" int abk_gemm_tc_swiglu(const void *x, const void *w, void *act, int M
     }
     const int m_tiles = (M + TILE_P - 1) / TILE_P, tiles = m_tiles * (N / 128);
     return launch_persistent<256, 4, __nv_bfloat16, EPI_GATED>(mx, mw, g, m_tiles, tiles, (cudaStream_t)stream);
+}
+
+extern "C" int abk_gemm_tc_swiglu(const void *x, const void *w, void *act, int M, int N, int K, long long ldx,
+                                  long long ldw, long long ldo, int *status, void *stream) {
+    return abk_gemm_tc_gated(x, w, act, M, N, K, ldx, ldw, ldo, ABK_SILU, status, stream);
 }
 
 // qkv[M, :n_heads * 128] = the prepared q heads of x . w^T, and the prepared k and the v heads of every token that

@@ -100,17 +100,50 @@ def add_rmsnorm(x, y, weight, out, eps, rows=None, n_rows=None):
                                     _f(eps), _stream()), "add_rmsnorm")
 
 
-def swiglu(gate_up, act, block=None):
-    """act = silu(gate) * up (src/model.c:274-282). A row of gate_up holds gate and up in turns of `block`
-    columns (gate of features [0, block), up of the same, gate of the next block, ...); by default all gates
+def normed_add_rmsnorm(x, y, weight_y, eps_y, weight, out, eps, rows=None, n_rows=None):
+    """x += weight_y * y / sqrt(mean(y^2) + eps_y) (y None: nothing); out = weight * x / sqrt(mean(x^2) + eps): the norm
+    behind a branch, the residual sum and the norm ahead of the next branch. x, y float32 [tokens, d]. rows (int32): only
+    those rows are made, into out[0:len(rows)], and x is left as it is."""
+    _need_cuda(x, y, weight_y, weight, out, rows)
+    lib = load_module("elementwise")
+    d = x.shape[-1]
+    n = n_rows if n_rows is not None else (rows.numel() if rows is not None else x.shape[0])
+    assert x.dtype == weight.dtype == torch.float32 and weight.numel() == d and x.is_contiguous()
+    assert y is None or (y.dtype == weight_y.dtype == torch.float32 and y.is_contiguous() and y.shape[-1] == d == weight_y.numel())
+    assert out.is_contiguous() and out.shape[-1] == d and out.shape[0] >= n and (rows is not None or x.shape[0] >= n)
+    _check(lib, lib.abk_normed_add_rmsnorm(_p(x), _p(y), _p(weight_y if y is not None else None), _p(weight), _p(out), _i(_dt(out)),
+                                           _p(rows), _i(n), _i(d), _f(eps_y), _f(eps), _stream()), "normed_add_rmsnorm")
+
+
+def embed_sinusoids(batch, table, coarse, fine, n_positions, x, status):
+    """x[t] = table[token] + s(position), s(p)[2i], s(p)[2i + 1] the sine and cosine of p * f_i: the angle's from coarse
+    [ceil(n_positions / 256), ceil(d / 2), 2] (sine and cosine of 256 a f_i) and fine [256, ceil(d / 2), 2] (of b f_i),
+    float32. A token or a position outside its table sets bit 0 of status and gives zeros."""
+    _need_cuda(table, coarse, fine, x, status)
+    lib = load_module("elementwise")
+    n, d = batch.n_rows, x.shape[-1]
+    assert x.dtype == coarse.dtype == fine.dtype == torch.float32 and x.is_contiguous() and x.shape[0] >= n
+    assert table.is_contiguous() and table.shape[1] == d and coarse.is_contiguous() and fine.is_contiguous()
+    assert fine.shape == (256, (d + 1) // 2, 2) and coarse.shape[1:] == fine.shape[1:] and coarse.shape[0] * 256 >= n_positions
+    _check(lib, lib.abk_embed_sinusoids(_p(batch.tokens), _p(batch.token_seq), _p(batch.token_pos), _p(table), _i(_dt(table)),
+                                        _p(coarse), _p(fine), _p(x), _i(n), _i(d), _i(table.shape[0]), _i(n_positions),
+                                        _p(status), _stream()), "embed_sinusoids")
+
+
+ACTIVATIONS = {"silu": 0, "relu": 1}  # what a gated feed-forward applies to its gate (csrc/common.cuh)
+
+
+def swiglu(gate_up, act, block=None, activation="silu"):
+    """act = silu(gate) * up (src/model.c:274-282), or relu(gate) * up. A row of gate_up holds gate and up in turns of
+    `block` columns (gate of features [0, block), up of the same, gate of the next block, ...); by default all gates
     and then all ups."""
     _need_cuda(gate_up, act)
     lib = load_module("elementwise")
     n, two_i = gate_up.shape
     assert act.shape == (n, two_i // 2) and act.dtype == gate_up.dtype
     assert gate_up.is_contiguous() and act.is_contiguous()
-    _check(lib, lib.abk_swiglu(_p(gate_up), _p(act), _i(_dt(act)), _i(n), _i(two_i // 2), _i(block or two_i // 2),
-                               _stream()), "swiglu")
+    _check(lib, lib.abk_gated_act(_p(gate_up), _p(act), _i(_dt(act)), _i(n), _i(two_i // 2), _i(block or two_i // 2),
+                                  _i(ACTIVATIONS[activation]), _stream()), "swiglu")
 
 
 def qkv_prep(qkv, n_heads, n_kv_heads, head_dim, batch, q_norm, k_norm, eps, cos, sin, rotary_dim, interleaved,
@@ -250,8 +283,8 @@ def gemm_rows_planes(x, w, out, block, m=None, tanh_from=None):
            "gemm_rows_planes")
 
 
-def gemm_rows_swiglu(x, w_gate_up, act, m=None, block=None):
-    """act[:m] = silu(x . gate^T) * (x . up^T) for m <= 64 rows, w_gate_up [2 I, K] holding gate and up rows in
+def gemm_rows_swiglu(x, w_gate_up, act, m=None, block=None, activation="silu"):
+    """act[:m] = silu(x . gate^T) * (x . up^T) (or relu, by activation) for m <= 64 rows, w_gate_up [2 I, K] holding gate and up rows in
     turns of `block` rows (by default all gates, then all ups): the feed-forward's first product and its
     activation in one kernel (src/model.c:307-308)."""
     _need_cuda(x, w_gate_up, act)
@@ -259,9 +292,9 @@ def gemm_rows_swiglu(x, w_gate_up, act, m=None, block=None):
     m = x.shape[0] if m is None else m
     two_i, k = w_gate_up.shape
     assert x.shape[1] == k and act.shape[1] == two_i // 2 and act.dtype == torch.bfloat16 and act.stride(1) == 1
-    _check(lib, lib.abk_gemm_rows_swiglu(_p(x), _p(w_gate_up), _p(act), _i(m), _i(two_i // 2), _i(k), _ll(x.stride(0)),
-                                         _ll(w_gate_up.stride(0)), _ll(act.stride(0)), _i(block or two_i // 2), _stream()),
-           "gemm_rows_swiglu")
+    _check(lib, lib.abk_gemm_rows_gated(_p(x), _p(w_gate_up), _p(act), _i(m), _i(two_i // 2), _i(k), _ll(x.stride(0)),
+                                        _ll(w_gate_up.stride(0)), _ll(act.stride(0)), _i(block or two_i // 2),
+                                        _i(ACTIVATIONS[activation]), _stream()), "gemm_rows_swiglu")
 
 
 def gemm_tc_swiglu_takes(x, w_gate_up, act, m, block):
@@ -271,8 +304,8 @@ def gemm_tc_swiglu_takes(x, w_gate_up, act, m, block):
             and act.stride(0) % 8 == 0 and act.data_ptr() % 16 == 0 and gemm_tc_takes(x, w_gate_up, act))
 
 
-def gemm_tc_swiglu(x, w_gate_up, act, m=None):
-    """act[:m] = silu(x . gate^T) * (x . up^T) on the tcgen05 tensor cores for more than 256 rows, w_gate_up
+def gemm_tc_swiglu(x, w_gate_up, act, m=None, activation="silu"):
+    """act[:m] = silu(x . gate^T) * (x . up^T) (or relu, by activation) on the tcgen05 tensor cores for more than 256 rows, w_gate_up
     [2 I, K] holding gate and up rows in turns of 128: the activation runs in the product's epilogue, under the
     next tile's multiplication (src/model.c:307-308)."""
     _need_cuda(x, w_gate_up, act)
@@ -281,9 +314,9 @@ def gemm_tc_swiglu(x, w_gate_up, act, m=None):
     two_i, k = w_gate_up.shape
     assert x.dtype == torch.bfloat16 and w_gate_up.dtype == torch.bfloat16 and act.dtype == torch.bfloat16
     assert x.shape[1] == k and act.shape[1] == two_i // 2 and x.stride(1) == 1 and w_gate_up.stride(1) == 1 and act.stride(1) == 1
-    _check(lib, lib.abk_gemm_tc_swiglu(_p(x), _p(w_gate_up), _p(act), _i(m), _i(two_i // 2), _i(k), _ll(x.stride(0)),
-                                       _ll(w_gate_up.stride(0)), _ll(act.stride(0)), _p(_Scratch.of(x.device).status),
-                                       _stream()), "gemm_tc_swiglu")
+    _check(lib, lib.abk_gemm_tc_gated(_p(x), _p(w_gate_up), _p(act), _i(m), _i(two_i // 2), _i(k), _ll(x.stride(0)),
+                                      _ll(w_gate_up.stride(0)), _ll(act.stride(0)), _i(ACTIVATIONS[activation]),
+                                      _p(_Scratch.of(x.device).status), _stream()), "gemm_tc_swiglu")
 
 
 def gemm_tc_qkv_takes(x, w_qkv, qkv, m, n_heads, n_kv_heads, head_dim, cache, q_norm, k_norm, cos, sin, rotary_dim, interleaved):
@@ -1300,17 +1333,21 @@ def columns_norm(src, dst, count, weight, eps, n):
 
 # ------------------------------------------------------------------ attention whose values are its keys (csrc/elementwise.cu)
 def qkv_prep_whole(src, dst, n_heads, n_kv_heads, head_dim, batch, q_norm, k_norm, eps, cos, sin, rotary_dim, interleaved,
-                   cache):
+                   cache, v_dim=None, bias=None, temperature=None):
     """Between the q/k product and attention where q and k are each normed over their whole row (q_norm float32
     [heads * head_dim], k_norm [kv heads * head_dim]; None: no norm) and a value head is its key head as projected:
     src rows [q | k | ...] as projected, dst rows [q | k | v] normed, rotated (pairs of the first rotary_dim elements
-    of every head) and, for k and v, written to the cache (a cache.LayerKV, or None)."""
-    _need_cuda(src, dst, q_norm, k_norm, cos, sin)
+    of every head) and, for k and v, written to the cache (a cache.LayerKV, or None). v_dim: values of that size have a
+    projection of their own, src rows [q | k | v | ...]. bias (float32, a row's size): added to the row as projected.
+    temperature (coef, every): q times 1 + coef * ln(floor((position + 1) / every) + 1), after its norm."""
+    _need_cuda(src, dst, q_norm, k_norm, cos, sin, bias)
     lib = load_module("elementwise")
     n = batch.n_rows
-    heads_size = (n_heads + 2 * n_kv_heads) * head_dim
+    heads_size = (n_heads + n_kv_heads) * head_dim + n_kv_heads * (v_dim or head_dim)
     assert src.dtype == dst.dtype and src.stride(1) == 1 and dst.stride(1) == 1 and src.data_ptr() != dst.data_ptr()
-    assert src.shape[1] >= (n_heads + n_kv_heads) * head_dim and dst.shape[1] >= heads_size and min(src.shape[0], dst.shape[0]) >= n
+    projected = heads_size if v_dim else (n_heads + n_kv_heads) * head_dim
+    assert bias is None or (bias.dtype == torch.float32 and bias.is_contiguous() and bias.numel() >= projected)
+    assert src.shape[1] >= projected and dst.shape[1] >= heads_size and min(src.shape[0], dst.shape[0]) >= n
     if cos is not None:
         assert cos.dtype == torch.float32 and cos.shape == sin.shape and cos.shape[1] == rotary_dim // 2
         if batch.max_position >= cos.shape[0]:
@@ -1320,9 +1357,11 @@ def qkv_prep_whole(src, dst, n_heads, n_kv_heads, head_dim, batch, q_norm, k_nor
         assert q_norm.numel() == n_heads * head_dim and k_norm.numel() == n_kv_heads * head_dim
     if cache is not None:
         assert cache.k.dtype == dst.dtype and cache.k.shape[1:] == (n_kv_heads, cache.tokens_per_page, head_dim)
-        assert cache.v.shape == cache.k.shape
+        assert cache.v.shape[1:] == (n_kv_heads, cache.tokens_per_page, v_dim or head_dim)
+    coef, every = temperature if temperature is not None else (0.0, 0.0)
     _check(lib, lib.abk_qkv_prep_whole(
         _p(src), _ll(src.stride(0)), _p(dst), _ll(dst.stride(0)), _i(_dt(dst)), _i(n), _i(n_heads), _i(n_kv_heads), _i(head_dim),
+        _i(v_dim or 0), _p(bias), _f(coef), _f(every),
         _p(batch.token_seq), _p(batch.token_pos), _p(batch.seq_slot), _p(batch.seq_len_after), _p(q_norm), _p(k_norm),
         _f(eps or 0.0), _p(cos), _p(sin), _i(rotary_dim), _i(1 if interleaved else 0),
         _p(cache.k if cache is not None else None), _p(cache.v if cache is not None else None),
@@ -1440,3 +1479,54 @@ def add_vector(x, v, n):
     d = v.numel()
     assert x.dtype == v.dtype == torch.float32 and x.is_contiguous() and v.is_contiguous() and x.numel() // x.shape[0] == d
     _check(lib, lib.abk_add_vector(_p(x), _p(v), _i(n), _i(d), _stream()), "add_vector")
+
+
+# ------------------------------------------------------------------ attention without a softmax (csrc/attention_sigmoid.cu)
+def attention_sigmoid(qkv, out, n_heads, n_kv_heads, head_dim, scale, batch, cache, v_dim=None, softcap=None, slopes=None,
+                      shift=None, mix=None, row=None, ws=None):
+    """Causal attention whose weights are the sigmoids of the scores, each key for itself, mixed between the heads:
+        z_h = scale * (q_h . k), capped (softcap * tanh(z / softcap)), less slopes[h] * distance, plus shift[h];
+        out_h = sum_j m_h(j) v_j,   m_h = sum_g mix[h, g] sigmoid(z_g)
+    slopes, shift float32 [n_heads], mix float32 [n_heads, n_heads]; each may be None. q from qkv's rows (`row` elements
+    apart: [q | k | v | padding]); keys and values from the paged cache (which this step's have been written to). All but the
+    operands of the scores, and the values, is float32."""
+    _need_cuda(qkv, out, slopes, shift, mix)
+    vd = v_dim or head_dim
+    heads_size = (n_heads + n_kv_heads) * head_dim + n_kv_heads * vd
+    row = row or heads_size
+    n = batch.n_rows
+    assert qkv.is_contiguous() and qkv.shape[1] == row >= heads_size and out.is_contiguous() and out.dtype == qkv.dtype
+    assert out.shape[1] == n_heads * vd and out.shape[0] >= n and qkv.shape[0] >= n
+    assert cache is not None and cache.k.dtype == qkv.dtype and cache.v.shape[-1] == vd and not cache.ring_pages
+    assert all(t is None or (t.dtype == torch.float32 and t.numel() == n_heads) for t in (slopes, shift))
+    assert mix is None or (mix.dtype == torch.float32 and mix.shape == (n_heads, n_heads) and mix.is_contiguous())
+    lib = load_module("attention_sigmoid")
+    _check(lib, lib.abk_attention_sigmoid(
+        _p(qkv), _ll(row), _p(out), _i(_dt(qkv)), _i(n), _i(n_heads), _i(n_kv_heads), _i(head_dim), _i(vd), _f(scale),
+        _f(softcap or 0.0), _p(slopes), _p(shift), _p(mix), _p(batch.token_seq), _p(batch.token_pos), _p(batch.seq_slot),
+        _p(cache.k), _p(cache.v), _p(cache.page_table), _i(cache.table_width), _i(cache.tokens_per_page), _stream()),
+        "attention_sigmoid")
+
+
+# ------------------------------------------------------------------ a running average per channel (csrc/gated_average.cu)
+def gated_average(proj, z_at, u_at, g_at, width, bias_z, bias_u, state, out, batch):
+    """For every sequence of the step and every channel, float32:
+        z = sigmoid(z' + bias_z), u = u' + bias_u, c = u + 1/2 where u >= 0, sigmoid(u) where u < 0;
+        S <- (1 - z) S + z c;   out = S * silu(g)
+    proj [tokens, .] as stored, z', u', g at columns z_at, u_at, g_at; state float32 [slots, width]; out [tokens, >= width] of
+    proj's type (columns beyond width get zeros). A decode step is a thread a few channels; a step of prompts cuts every sequence into runs walked at
+    once by clusters of CTAs (as many CTAs a sequence as the step's mean length asks for)."""
+    _need_cuda(proj, bias_z, bias_u, state, out)
+    lib = load_module("gated_average")
+    assert proj.stride(1) == 1 and out.stride(1) == 1 and proj.dtype == out.dtype and out.shape[1] >= width
+    assert bias_z.dtype == bias_u.dtype == state.dtype == torch.float32 and bias_z.numel() == bias_u.numel() == width
+    assert state.is_contiguous() and state.shape[1:] == (width,) and proj.shape[1] >= max(z_at, u_at, g_at) + width
+    n, n_seqs = batch.n_rows, batch.seq_slot.numel()
+    assert proj.shape[0] >= n and out.shape[0] >= n
+    mean, ranks = n / max(1, n_seqs), 1
+    while ranks < 8 and ranks * 128 < mean:  # (a CTA has 128 tokens a turn)
+        ranks *= 2
+    _check(lib, lib.abk_gated_average(_p(proj), _ll(proj.stride(0)), _i(_dt(proj)), _i(z_at), _i(u_at), _i(g_at), _i(width),
+                                      _p(bias_z), _p(bias_u), _p(state), _p(out), _ll(out.stride(0)), _i(out.shape[1]), _i(n), _i(n_seqs),
+                                      _i(1 if batch.is_decode else 0), _i(ranks), _p(batch.token_seq), _p(batch.seq_start),
+                                      _p(batch.seq_slot), _stream()), "gated_average")

@@ -91,8 +91,8 @@ class Model:
         return list(plans.values())
 
     def prepare(self, max_positions):
-        for b in self.blocks:
-            prepare = getattr(b.mixer, "prepare", None)
+        for part in [self.frame] + [b.mixer for b in self.blocks]:
+            prepare = getattr(part, "prepare", None)
             if prepare:
                 prepare(max_positions, self.ctx.device)
 

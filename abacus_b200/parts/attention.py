@@ -7,7 +7,9 @@ its spec. q, k and v are one stacked matrix, as in src/model.c:88-93.
 Options of the spec that only the general kernels take: values of another size than keys, a sequence's first keys
 kept behind a window, a sink, float32 weights, a short causal convolution over time on every channel of q, k and v
 right after their projection (its last inputs are part of the sequence's state, beside the keys and values), keys
-seen only within the token's own chunk of positions, and capped scores.
+seen only within the token's own chunk of positions, and capped scores. A layer may do without a softmax altogether
+(weights "sigmoid": each key for itself, with a distance bias and a shift per head, the heads' weights mixed before
+they meet the values): the projection, its preparation and the cache are the same, the attention kernels its own.
 """
 import os
 
@@ -44,15 +46,26 @@ class Attention:
         # what only the general kernel takes: values of another size, kept first keys, a sink, float32 weights
         # q and k normed over their whole rows, values that are their keys, a gate per head: a preparation kernel of
         # their own (out of the projection's rows into the rows the attention kernels read), then the general kernels
-        self.whole = s.norm_over == "projection" or s.values == "keys"
+        self.whole = s.norm_over == "projection" or s.values == "keys" or s.bias or s.q_temperature is not None
         if s.norm_over not in ("head", "projection") or s.values not in ("own", "keys"):
             raise ValueError(f"norm_over {s.norm_over!r} is neither head nor projection, or values {s.values!r} neither own nor keys")
-        if self.whole and (s.conv_taps or (s.v_head_dim or s.head_dim) != s.head_dim
+        if self.whole and (s.conv_taps or (s.values == "keys" and self.v_dim != s.head_dim)
                            or (s.qk_norm_eps is not None and s.norm_over != "projection")):
-            raise ValueError("values that are their keys and norms over the whole projection go with neither a convolution, "
-                             "values of another size nor a norm per head")
+            raise ValueError("values that are their keys, norms over the whole projection, biases and a query temperature go "
+                             "with neither a convolution nor a norm per head, and values that are keys are of their size")
+        if s.bias and s.values == "keys":
+            raise ValueError("values that are their keys have no bias of their own")
+        self.sigmoid = s.weights == "sigmoid"
+        if s.weights not in ("softmax", "sigmoid"):
+            raise ValueError(f"weights {s.weights!r} are neither softmax nor sigmoid")
+        if self.sigmoid and (s.window is not None or s.chunk or s.sink or s.head_gate or not s.exact_weights):
+            raise ValueError("sigmoid weights are float32 and take no window, no chunk, no sink and no gate per head")
+        if not self.sigmoid and (s.slopes is not None or s.shift or s.mix):
+            raise ValueError("slopes, a shift per head and mixed heads go with sigmoid weights")
+        if s.slopes is not None and len(s.slopes) != s.n_heads:
+            raise ValueError(f"{len(s.slopes)} slopes for {s.n_heads} heads")
         self.general = (self.v_dim != s.head_dim or bool(s.keep_first) or s.sink or s.exact_weights or s.conv_taps > 0
-                        or bool(s.chunk) or bool(s.softcap) or self.whole or s.head_gate)
+                        or bool(s.chunk) or bool(s.softcap) or self.whole or s.head_gate or self.sigmoid)
         if s.conv_taps < 0 or s.conv_taps > 8:
             raise ValueError(f"conv_taps {s.conv_taps}: the convolution takes 1 to 8 taps")
         if s.chunk is not None and s.chunk < 1:
@@ -83,11 +96,11 @@ class Attention:
 
     def step_plans(self):
         """What this mixer wants made on the host for every step and sent with the step's indices."""
-        return [self.lists]
+        return [] if self.sigmoid else [self.lists]  # (attention without a softmax needs none)
 
     def step_weights(self):
         """The tensors a step reads once whatever its size (for the bytes a decode step must move)."""
-        return [self.qkv_proj.weight, self.o_proj.weight, self.q_norm, self.k_norm, self.sink, self.conv]
+        return [self.qkv_proj.weight, self.o_proj.weight, self.q_norm, self.k_norm, self.sink, self.conv, self.bias, self.mix]
 
     def param_shapes(self):
         s = self.spec
@@ -103,6 +116,12 @@ class Attention:
             shapes.update(q_norm=(s.head_dim,), k_norm=(s.head_dim,))
         if s.sink:
             shapes["sink"] = (s.n_heads,)
+        if s.bias:
+            shapes.update(bq=(self.q_size,), bk=(self.kv_size,), bv=(self.v_size,))
+        if s.shift:
+            shapes["shift"] = (s.n_heads,)
+        if s.mix:
+            shapes["mix"] = (s.n_heads, s.n_heads)
         if s.conv_taps:
             shapes.update(conv_q=(self.q_size, s.conv_taps), conv_k=(self.kv_size, s.conv_taps),
                           conv_v=(self.v_size, s.conv_taps))
@@ -121,6 +140,12 @@ class Attention:
         self.q_norm = to_device(params["q_norm"], ctx, torch.float32) if "q_norm" in params else None
         self.k_norm = to_device(params["k_norm"], ctx, torch.float32) if "k_norm" in params else None
         self.sink = to_device(params["sink"], ctx, torch.float32) if "sink" in params else None
+        self.bias = (to_device(torch.cat([params["bq"], params["bk"], params["bv"]]), ctx, torch.float32)
+                     if self.spec.bias else None)
+        self.shift = to_device(params["shift"], ctx, torch.float32) if self.spec.shift else None
+        self.mix = to_device(params["mix"], ctx, torch.float32) if self.spec.mix else None
+        self.slopes = (torch.tensor(self.spec.slopes, dtype=torch.float64).to(torch.float32).to(ctx.device)
+                       if self.spec.slopes is not None else None)
         self.conv = None
         if self.spec.conv_taps:  # one table for the whole row of q, k and v; the row's padding has taps of zero
             taps = torch.cat([params["conv_q"], params["conv_k"], params["conv_v"]], dim=0).to(torch.float32)
@@ -168,7 +193,8 @@ class Attention:
                 raise ops.KernelRefused("an attention entry whose values are its keys, or with gated heads, keeps keys of its own")
             if self.whole:
                 ops.qkv_prep_whole(proj, qkv, s.n_heads, s.n_kv_heads, s.head_dim, batch, self.q_norm, self.k_norm,
-                                   s.qk_norm_eps, self.cos, self.sin, rotary_dim, interleaved, cache.kv)
+                                   s.qk_norm_eps, self.cos, self.sin, rotary_dim, interleaved, cache.kv,
+                                   v_dim=self.v_dim if s.values == "own" else None, bias=self.bias, temperature=s.q_temperature)
                 prepared = True
             else:
                 qkv[:n, :self.gate_at].copy_(proj[:n, :self.gate_at])
@@ -201,6 +227,11 @@ class Attention:
         if from_step and (batch.any_continuation or not writes):
             raise ops.KernelRefused("windowed attention takes several tokens of a sequence only at its start, "
                                     "and only with keys of its own")
+        if self.sigmoid:
+            ops.attention_sigmoid(qkv, att, s.n_heads, s.n_kv_heads, s.head_dim, s.scale, batch, cache.kv, v_dim=self.v_dim,
+                                  softcap=s.softcap, slopes=self.slopes, shift=self.shift, mix=self.mix, row=self.row, ws=ws)
+            self.o_proj.forward(att, out, n)
+            return out
         mine = batch.plan.get(self.lists.name)
         gates = ws.get("qkv_proj", (n, self.proj_row), self.ctx.dtype)[:, self.gate_at:] if s.head_gate else None
         gated = ops.attention(qkv, att, s.n_heads, s.n_kv_heads, s.head_dim, s.scale, s.window, batch, cache.kv,

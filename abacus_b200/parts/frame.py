@@ -18,6 +18,7 @@ import torch
 from ..kernels import ops
 from .base import FRAMES, NORMS, to_device
 from .linear import Linear
+from .position import Sinusoids
 
 
 @FRAMES.register("plain")
@@ -242,5 +243,41 @@ class LoopInputFrame:
         if r:
             xn = ws.get("xn_final", (r, self.hidden), self.ctx.dtype)
             read_streams(x, pending, self.ones, self.final_norm, xn, rows=batch.logit_rows, n_rows=r)
+            self.head.forward(xn, out, r)
+        return out
+
+
+@FRAMES.register("sinusoids")
+class SinusoidsFrame(PlainFrame):
+    """x = table[token] + a fixed sinusoid per position (config.specs.SinusoidEmbeddingSpec, parts/position.py); the stream
+    is one row per token. The end: the pending branch with its norm (parts/block.py, sandwich_norm), the last norm, the
+    output matrix on the wanted rows, the logits times logit_scale (which is in the last norm's weight, so it costs nothing
+    and is taken in float32)."""
+
+    def __init__(self, spec):
+        super().__init__(spec)
+        self.options = spec.frame_spec
+        self.sinusoids = Sinusoids(spec.hidden, self.options.base)
+        self.coarse = self.fine = None
+
+    def bind(self, params, ctx):
+        super().bind(params, ctx)
+        self.final_norm.weight = (self.final_norm.weight * self.options.logit_scale).contiguous()
+
+    def prepare(self, max_positions, device):
+        self.n_positions = max_positions
+        self.coarse, self.fine = self.sinusoids.tables(max_positions, device)
+
+    def embed(self, batch, ws, status):
+        x = ws.get("x", (batch.n_rows, self.hidden), torch.float32)
+        ops.embed_sinusoids(batch, self.table, self.coarse, self.fine, self.n_positions, x, status)
+        return x
+
+    def logits(self, x, pending, batch, ws):
+        r = batch.n_logit_rows
+        out = ws.get("logits", (max(r, 1), self.vocab), torch.float32)[:r]
+        if r:
+            xn = ws.get("xn_final", (r, self.hidden), self.ctx.dtype)
+            self.final_norm.forward_normed(x, pending, xn, rows=batch.logit_rows, n_rows=r)
             self.head.forward(xn, out, r)
         return out

@@ -1,4 +1,4 @@
-"""Gated feed-forward: down(silu(gate(x)) * up(x)) (src/model.c:274-282, 307-309).
+"""Gated feed-forward: down(silu(gate(x)) * up(x)) (src/model.c:274-282, 307-309), or with relu in silu's place.
 
 gate and up are one matrix, as in src/model.c:98. In bfloat16, when the inner size allows, its rows come
 in turns of 128 (gate of features 0-127, up of the same, gate of 128-255, ...): a 256-column tile of the
@@ -16,8 +16,8 @@ class GatedMLP:
     capturable = True  # its forward launches kernels only; nothing in it depends on the step's contents
 
     def __init__(self, spec):
-        if spec.activation != "silu":
-            raise ValueError(f"activation {spec.activation!r} is not built (only silu)")
+        if spec.activation not in ops.ACTIVATIONS:
+            raise ValueError(f"activation {spec.activation!r} is not built (only {', '.join(ops.ACTIVATIONS)})")
         self.spec = spec
 
     def param_shapes(self):
@@ -39,16 +39,16 @@ class GatedMLP:
         return [self.gate_up.weight, self.down.weight]
 
     def forward(self, xn, out, batch, ws):
-        n, inter = batch.n_rows, self.spec.inter
+        n, inter, kind = batch.n_rows, self.spec.inter, self.spec.activation
         act = ws.get("act", (n, inter), self.ctx.dtype)
         w = self.gate_up.weight
         if rows_kernel_wins(n, w, gated=True) and ops.gemm_rows_takes(xn, w, act, n):
-            ops.gemm_rows_swiglu(xn, w, act, n, self.block)  # a handful of rows: product and activation in one
+            ops.gemm_rows_swiglu(xn, w, act, n, self.block, kind)  # a handful of rows: product and activation in one
         elif ops.gemm_tc_swiglu_takes(xn, w, act, n, self.block):
-            ops.gemm_tc_swiglu(xn, w, act, n)  # a prompt: the activation in the product's epilogue
+            ops.gemm_tc_swiglu(xn, w, act, n, kind)  # a prompt: the activation in the product's epilogue
         else:
             gate_up = ws.get("gate_up", (n, 2 * inter), self.ctx.dtype)
             self.gate_up.forward(xn, gate_up, n)
-            ops.swiglu(gate_up, act, self.block)
+            ops.swiglu(gate_up, act, self.block, kind)
         self.down.forward(act, out, n)
         return out

@@ -27,3 +27,10 @@ class RMSNorm:
     def forward(self, x, y, out, rows=None, n_rows=None):
         ops.add_rmsnorm(x, y, self.weight, out, self.spec.eps, rows=rows, n_rows=n_rows)
         return out
+
+    def forward_normed(self, x, pending, out, rows=None, n_rows=None):
+        """As forward(), where what is added to the stream has a norm of its own: pending is (y, that RMSNorm) or None."""
+        y, post = pending if pending is not None else (None, None)
+        ops.normed_add_rmsnorm(x, y, post.weight if post is not None else None, post.spec.eps if post is not None else 0.0,
+                               self.weight, out, self.spec.eps, rows=rows, n_rows=n_rows)
+        return out

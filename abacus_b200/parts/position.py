@@ -64,3 +64,30 @@ class Rotary:
                     torch.from_numpy(np.sin(angle, dtype=np.float32)).to(device))
             self._tables[key] = have
         return have
+
+
+class Sinusoids:
+    """Fixed sinusoids per position: element 2i of a vector is sin(p * base^(-2i / size)), element 2i + 1 its cosine.
+
+    tables(n_positions, device) -> (coarse, fine), float32 [.., ceil(size / 2), 2] (sine, cosine), made in float64: position
+    256 a + b has the sum of the angles of coarse[a] and fine[b], so a million positions take 4,096 + 256 rows.
+    """
+    FINE = 256
+
+    def __init__(self, size, base):
+        self.size, self.base = size, float(base)
+        self._tables = {}
+
+    def tables(self, n_positions, device):
+        key, rows = str(device), max(1, -(-n_positions // self.FINE))
+        have = self._tables.get(key)
+        if have is None or have[0].shape[0] < rows:
+            i = np.arange((self.size + 1) // 2, dtype=np.float64)
+            freq = np.power(self.base, -2.0 * i / self.size)
+
+            def table(positions):
+                angle = positions.astype(np.float64)[:, None] * freq[None, :]
+                return torch.from_numpy(np.stack([np.sin(angle), np.cos(angle)], axis=-1).astype(np.float32)).to(device)
+            have = (table(np.arange(rows) * self.FINE), table(np.arange(self.FINE)))
+            self._tables[key] = have
+        return have
