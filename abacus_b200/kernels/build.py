@@ -26,7 +26,7 @@ NVCC_FLAGS = ["-O3", "-std=c++17", "-lineinfo", "--shared", "-Xcompiler", "-fPIC
 MODULES = ("elementwise", "gemm_simt", "gemm_tc", "attention_generic", "attention_decode", "attention_mma", "gemm_rows",
            "sampling", "attention_decode_static", "attention_decode_ring", "attention_tc", "utility", "step", "streams",
            "delta_rule", "attention_window", "attention_split", "latent", "lightning", "moe", "gemm_grouped", "matrix_memory", "wkv",
-           "attention_sigmoid", "gated_average")
+           "attention_sigmoid", "attention_sigmoid_prompt", "attention_sigmoid_decode", "gated_average")
 
 
 # ABACUS_TRACE=1 builds every library with the launch-timeline records of csrc/common.cuh compiled in

@@ -1500,12 +1500,74 @@ def attention_sigmoid(qkv, out, n_heads, n_kv_heads, head_dim, scale, batch, cac
     assert cache is not None and cache.k.dtype == qkv.dtype and cache.v.shape[-1] == vd and not cache.ring_pages
     assert all(t is None or (t.dtype == torch.float32 and t.numel() == n_heads) for t in (slopes, shift))
     assert mix is None or (mix.dtype == torch.float32 and mix.shape == (n_heads, n_heads) and mix.is_contiguous())
-    lib = load_module("attention_sigmoid")
+    sizes = (qkv, out, n_heads, n_kv_heads, head_dim, vd, row)
+    if batch.is_decode and ws is not None and attention_sigmoid_decode_parts(qkv, n, n_heads, n_kv_heads, head_dim, vd, cache, 1):
+        return _attention_sigmoid_decode(*sizes, scale, batch, cache, softcap, slopes, shift, mix, ws)
+    if not batch.is_decode and not batch.any_continuation and attention_sigmoid_prompt_takes(*sizes[:1], *sizes[2:]):
+        return attention_sigmoid_prompt(*sizes, scale, batch, softcap, slopes, shift, mix)
+    return attention_sigmoid_general(*sizes, scale, batch, cache, softcap, slopes, shift, mix)
+
+
+def attention_sigmoid_general(qkv, out, n_heads, n_kv_heads, head_dim, vd, row, scale, batch, cache, softcap, slopes, shift, mix):
+    """The form for any sizes (csrc/attention_sigmoid.cu): the float32 path, portions of prompts, what the other two refuse."""
+    n, lib = batch.n_rows, load_module("attention_sigmoid")
     _check(lib, lib.abk_attention_sigmoid(
         _p(qkv), _ll(row), _p(out), _i(_dt(qkv)), _i(n), _i(n_heads), _i(n_kv_heads), _i(head_dim), _i(vd), _f(scale),
         _f(softcap or 0.0), _p(slopes), _p(shift), _p(mix), _p(batch.token_seq), _p(batch.token_pos), _p(batch.seq_slot),
         _p(cache.k), _p(cache.v), _p(cache.page_table), _i(cache.table_width), _i(cache.tokens_per_page), _stream()),
         "attention_sigmoid")
+
+
+def attention_sigmoid_prompt_takes(qkv, n_heads, n_kv_heads, head_dim, vd, row):
+    """Whether the tensor-core kernel for whole prompts takes these sizes: bfloat16, up to 32 heads, heads and values of
+    multiples of 8 (values up to 128), every part of a row 16-byte aligned, and what a CTA holds of shared memory."""
+    if not (qkv.dtype == torch.bfloat16 and n_heads <= 32 and head_dim % 8 == 0 and vd % 8 == 0 and vd <= 128 and row % 8 == 0
+            and qkv.data_ptr() % 16 == 0):
+        return False
+    # (as csrc/attention_sigmoid_prompt.cu lays it out, with 16 keys a tile)
+    warps = 4 if n_heads <= 4 else 8 if n_heads <= 8 else 16
+    per, pitch_k, pitch_v = n_heads // n_kv_heads, -(-head_dim // 16) * 32 + 16, -(-vd // 16) * 32 + 16
+    values = max((min((b + 1) * warps, n_heads) - 1) // per - b * warps // per + 1 for b in range(-(-n_heads // warps)))
+    chunk = max(-(-n_heads // 16) * 16 * 64, warps * 96) + 16
+    return 16 * (n_heads * pitch_k + n_kv_heads * pitch_k + values * pitch_v + chunk) <= 227 * 1024
+
+
+def attention_sigmoid_prompt(qkv, out, n_heads, n_kv_heads, head_dim, vd, row, scale, batch, softcap, slopes, shift, mix, ranks=0):
+    """attention_sigmoid for whole prompts on the tensor cores, keys and values from the step's own rows
+    (csrc/attention_sigmoid_prompt.cu). mix holds bfloat16 numbers. ranks: the CTAs that share a query tile's keys (0: chosen)."""
+    n, n_seqs, lib = batch.n_rows, batch.seq_slot.numel(), load_module("attention_sigmoid_prompt")
+    if batch.any_continuation:
+        raise KernelRefused("attention_sigmoid_prompt reads keys from the step's rows: every sequence must start at position 0")
+    _check(lib, lib.abk_attention_sigmoid_prompt(
+        _p(qkv), _ll(row), _p(out), _i(n_heads), _i(n_kv_heads), _i(head_dim), _i(vd), _i(n_heads * head_dim),
+        _i((n_heads + n_kv_heads) * head_dim), _f(scale), _f(softcap or 0.0), _p(slopes), _p(shift), _p(mix), _p(batch.seq_start),
+        _i(n_seqs), _i((n + 15) // 16 + n_seqs), _i(ranks), _stream()), "attention_sigmoid_prompt")
+
+
+def attention_sigmoid_decode_parts(qkv, n, n_heads, n_kv_heads, head_dim, vd, cache, max_keys):
+    """How many CTAs a row's keys are dealt to by the decode kernel (csrc/attention_sigmoid_decode.cu); 0: it does not take
+    these sizes (bfloat16, groups of up to 16, heads and values of multiples of 8, eight keys and values of all kv heads within a
+    CTA's shared memory)."""
+    if qkv.dtype != torch.bfloat16 or cache.tokens_per_page != 64 or cache.k.data_ptr() % 16 or cache.v.data_ptr() % 16:
+        return 0
+    return load_module("attention_sigmoid_decode").abk_attention_sigmoid_decode_parts(_i(n), _i(n_heads), _i(n_kv_heads),
+                                                                                      _i(head_dim), _i(vd), _i(max_keys))
+
+
+def _attention_sigmoid_decode(qkv, out, n_heads, n_kv_heads, head_dim, vd, row, scale, batch, cache, softcap, slopes, shift, mix, ws):
+    n, lib = batch.n_rows, load_module("attention_sigmoid_decode")
+    top = getattr(batch, "position_bound", None) or batch.max_len_after
+    if batch.max_len_after > top:
+        raise KernelError(f"a row at position {batch.max_len_after - 1} is beyond the bound {top}")
+    n_parts = attention_sigmoid_decode_parts(qkv, n, n_heads, n_kv_heads, head_dim, vd, cache, top)
+    parts = ws.get("attention_parts", (n * n_parts * n_heads * vd,), torch.float32)
+    assert cache.k.is_contiguous() and cache.v.is_contiguous()
+    pool_rows = cache.k.shape[0] * n_kv_heads * cache.tokens_per_page
+    _check(lib, lib.abk_attention_sigmoid_decode(
+        _p(qkv), _ll(row), _p(out), _i(n), _i(n_heads), _i(n_kv_heads), _i(head_dim), _i(vd), _f(scale), _f(softcap or 0.0),
+        _p(slopes), _p(shift), _p(mix), _p(batch.token_seq), _p(batch.token_pos), _p(batch.seq_slot), _p(cache.k), _p(cache.v),
+        _ll(pool_rows), _p(cache.page_table), _i(cache.table_width), _i(cache.tokens_per_page), _i(n_parts), _p(parts),
+        _p(_Scratch.of(qkv.device).status), _stream()), "attention_sigmoid_decode", kernels=2)
 
 
 # ------------------------------------------------------------------ a running average per channel (csrc/gated_average.cu)

@@ -565,6 +565,32 @@ def build_tilulorn(size):
     return model
 
 
+# Lilovik at the same widths, depths, heads, feed-forward and vocabulary: every fourth layer a running average per channel as
+# wide as the stream, the others attention without a softmax over every earlier key (heads of 128 over 8 key heads, a cap, a
+# distance bias, mixed heads); a gated feed-forward with relu in every layer.
+def build_lilovik(size):
+    import torch
+    from abacus_b200.config import get_architecture
+    from abacus_b200.config.lilovik import LilovikAttention, LilovikAverage, LilovikConfig, LilovikLayer
+    from abacus_b200.models import Model
+    from abacus_b200.weights import random_tensors
+    z = DESIGN_SIZES[size]
+    att = LilovikAttention(z["heads"], z["kv_heads"], z["dim"], z["dim"], z["dim"] ** -0.5, 30.0, 0.5, 256)
+    average = LilovikAverage(z["width"])
+    layers = tuple(LilovikLayer("mingru", average, z["ff"]) if i % 4 == 0 else LilovikLayer("attention", att, z["ff"])
+                   for i in range(z["layers"]))
+    config = LilovikConfig(vocab=z["vocab"], width=z["width"], layers=layers, eps=1e-6, logit_scale=1.0)
+    arch = get_architecture("Lilovik")
+    spec = config.to_spec()
+    expected, _ = arch.tensor_names(spec, None)
+    device = torch.device("cuda", 0)
+    tensors = random_tensors(expected, seed=5, std=0.02, device=device, rule=arch.random_moments)
+    model = Model(spec, arch.layout(spec), tensors, torch.bfloat16, device)
+    del tensors
+    torch.cuda.empty_cache()
+    return model
+
+
 def state_and_cache_bytes(model, tokens_held, n_seqs):
     """Bytes of keys, values and recurrent state a decode step moves for n_seqs sequences that hold tokens_held
     tokens together: a window's keys at most, the keys of the token's own chunk where attention sees no others, a state
@@ -606,7 +632,7 @@ def routed_expert_bytes(model, n_rows):
 
 
 def run_design(args):
-    """--design temetar | movarax | linonex | tilulorn: decode and prefill of the design at DESIGN_SIZES[--size] beside the Qwen3
+    """--design temetar | movarax | linonex | tilulorn | lilovik: decode and prefill of the design at DESIGN_SIZES[--size] beside the Qwen3
     shape of equal size (--beside: beside another design of equal size instead)."""
     import torch
     from abacus_b200.kernels import build_all
@@ -632,6 +658,8 @@ def run_design(args):
             model = build_linonex(args.size)
         elif which == "tilulorn":
             model = build_tilulorn(args.size)
+        elif which == "lilovik":
+            model = build_lilovik(args.size)
         else:
             model, _ = build_model(z["qwen"])
         prompts = prompts_for(args.batch, model.spec.vocab, 10 + args.batch)
@@ -740,10 +768,10 @@ def main():
     ap.add_argument("--config", default="0.6b", choices=sorted(CONFIGS), help="whose workload the line reports")
     ap.add_argument("--skip-large", action="store_true", help="leave the 4b and 8b workloads out of `points`")
     ap.add_argument("--ragged", action="store_true", help="with --only prefill: the configuration's own prompts")
-    ap.add_argument("--design", default=None, choices=["temetar", "movarax", "linonex", "tilulorn"],
+    ap.add_argument("--design", default=None, choices=["temetar", "movarax", "linonex", "tilulorn", "lilovik"],
                     help="instead of the default workload: this design at --size beside the Qwen3 shape of equal size")
     ap.add_argument("--size", default="s", choices=sorted(DESIGN_SIZES), help="with --design: the layer sizes")
-    ap.add_argument("--beside", default="qwen3", choices=["qwen3", "temetar", "movarax", "linonex"],
+    ap.add_argument("--beside", default="qwen3", choices=["qwen3", "temetar", "movarax", "linonex", "tilulorn"],
                     help="with --design: the model of equal size that runs beside it")
     args = ap.parse_args()
     if args.gpus != 1:
