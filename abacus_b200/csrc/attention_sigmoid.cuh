@@ -7,18 +7,17 @@
 //   no cap:  y = plain * dot + slope * back + base
 //   cap c:   c tanh(s / c) = c - 2 c / (1 + e^(2 s / c)), so  y = twice_cap / (1 + 2^(to_exp * dot)) + slope * back + base
 // The exponentials and reciprocals are the special-function unit's (float32, a few units in the last place).
-struct SigmoidHead {
+struct __align__(16) SigmoidHead {
     float to_exp, twice_cap, slope, base;
-    bool capped;
 };
 __device__ __forceinline__ SigmoidHead sigmoid_head(float scale, float cap, float slope, float shift) {
     const float l2e = 1.4426950408889634f;
     SigmoidHead c;
-    c.capped = cap > 0.0f;
-    c.to_exp = c.capped ? 2.0f * l2e * scale / cap : -l2e * scale;
+    const bool capped = cap > 0.0f;
+    c.to_exp = capped ? 2.0f * l2e * scale / cap : -l2e * scale;
     c.twice_cap = 2.0f * l2e * cap;
     c.slope = slope * l2e;
-    c.base = -shift * l2e - (c.capped ? l2e * cap : 0.0f);
+    c.base = -shift * l2e - (capped ? l2e * cap : 0.0f);
     return c;
 }
 __device__ __forceinline__ float sfu_exp2(float x) {
@@ -32,8 +31,8 @@ __device__ __forceinline__ float sfu_inverse(float x) {
     return y;
 }
 // away: slope * back + base of the key, made by the caller (a multiply-add, or less where keys follow one another)
-__device__ __forceinline__ float sigmoid_of(const SigmoidHead &c, float dot, float away) {
-    const float y = c.capped ? fmaf(c.twice_cap, sfu_inverse(1.0f + sfu_exp2(c.to_exp * dot)), away) : fmaf(c.to_exp, dot, away);
+__device__ __forceinline__ float sigmoid_of(bool capped, const SigmoidHead &c, float dot, float away) {
+    const float y = capped ? fmaf(c.twice_cap, sfu_inverse(1.0f + sfu_exp2(c.to_exp * dot)), away) : fmaf(c.to_exp, dot, away);
     return sfu_inverse(1.0f + sfu_exp2(y));
 }
 

@@ -66,11 +66,11 @@ template <int UNITS, int NT> __global__ void __launch_bounds__(SD_THREADS) atten
     float *a_s = (float *)((uint8_t *)q_s + sm.q), *m_s = a_s + H * sm.pitch_w, *mix_s = m_s + H * sm.pitch_w;
     SigmoidHead *head_s = (SigmoidHead *)((uint8_t *)mix_s + sm.mix);
     __shared__ uint64_t full[SD_MAX_STAGES];
-    __shared__ int failed;
+    __shared__ int failed[2];  // by the stage's parity: set before a stage's barriers, read after them
     const int part = blockIdx.x, t = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, r8 = lane >> 2, q2 = lane & 3;
     if (tid == 0) {
         for (int s = 0; s < p.stages; s++) tc::mbar_init(&full[s], 1);
-        failed = 0;
+        failed[0] = failed[1] = 0;
         tc::mbar_init_fence();
         tc::tma_prefetch_map(&map_k), tc::tma_prefetch_map(&map_v);
     }
@@ -117,7 +117,7 @@ template <int UNITS, int NT> __global__ void __launch_bounds__(SD_THREADS) atten
     for (int st = 0; st < n_st; st++) {
         const int s = st % p.stages, j0 = first + st * kp, nv = min(kp, n_keys - st * kp);
         const uint32_t k_s = tc::smem_addr(ring + s * sm.stage), v_s = k_s + G * sm.k_boxes * box;
-        if (!tc::mbar_wait(&full[s], (st / p.stages) & 1)) failed = 1;
+        if (!tc::mbar_wait(&full[s], (st / p.stages) & 1)) failed[st & 1] = 1;
         // scores: a warp takes a kv head and 16 keys at a time
         // (a stage of 8 keys fills half of a tile: the other half repeats them and is dropped, here and below)
         for (int u = warp; u < G * tiles16; u += SD_WARPS) {
@@ -161,7 +161,7 @@ template <int UNITS, int NT> __global__ void __launch_bounds__(SD_THREADS) atten
         for (int e = tid; e < H * kp; e += SD_THREADS) {
             const int h = e / kp, j = e - h * kp;
             const SigmoidHead hd = head_s[h];
-            w_s[h * sm.pitch_w + j] = j < nv ? sigmoid_of(hd, a_s[h * sm.pitch_w + j], fmaf(hd.slope, (float)(pos - j0 - j), hd.base)) : 0.0f;
+            w_s[h * sm.pitch_w + j] = j < nv ? sigmoid_of(p.softcap > 0.0f, hd, a_s[h * sm.pitch_w + j], fmaf(hd.slope, (float)(pos - j0 - j), hd.base)) : 0.0f;
         }
         __syncthreads();
         if (p.mix) {
@@ -204,8 +204,8 @@ template <int UNITS, int NT> __global__ void __launch_bounds__(SD_THREADS) atten
             }
         }
         __syncthreads();  // the stage and the weights are done with
-        if (warp == 0 && issued < n_st && !failed) issue(issued), issued++;
-        if (failed) {
+        if (warp == 0 && issued < n_st && !failed[st & 1]) issue(issued), issued++;
+        if (failed[st & 1]) {
             // a copy did not come: report it, and let the copies still in flight land (or run out of time) before the memory goes
             if (tid == 0) atomicOr(p.status + 2, 1);
             if (warp == 0)

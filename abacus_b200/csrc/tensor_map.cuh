@@ -71,4 +71,46 @@ static int bf16_rows_of_128_bytes(const void *ptr, long long rows, long long col
     return 0;
 }
 
+// A map over the heads of the rows of a step: bfloat16 [rows][heads][size], heads side by side (size elements apart), rows
+// `pitch` elements apart. Boxes of [box_rows, 1 head, 64] elements (128 bytes a row), 128-byte swizzle; what lies outside a
+// head or beyond the last row is zeros.
+static int bf16_heads(const void *ptr, int size, int heads, long long rows, long long pitch, int box_rows, CUtensorMap *out) {
+    struct HeadsKey {
+        const void *ptr;
+        int size, heads, box_rows;
+        long long rows, pitch;
+        bool operator==(const HeadsKey &o) const {
+            return ptr == o.ptr && size == o.size && heads == o.heads && box_rows == o.box_rows && rows == o.rows && pitch == o.pitch;
+        }
+    };
+    struct Hash {
+        size_t operator()(const HeadsKey &k) const {
+            size_t h = (size_t)k.ptr;
+            h = h * 1000003u ^ (size_t)k.rows, h = h * 1000003u ^ (size_t)k.pitch;
+            return h * 1000003u ^ (size_t)k.size ^ ((size_t)k.heads << 24) ^ ((size_t)k.box_rows << 48);
+        }
+    };
+    static std::unordered_map<HeadsKey, CUtensorMap, Hash> cache;
+    static std::mutex lock;
+    const HeadsKey key{ptr, size, heads, box_rows, rows, pitch};
+    std::lock_guard<std::mutex> guard(lock);
+    auto it = cache.find(key);
+    if (it != cache.end()) {
+        *out = it->second;
+        return 0;
+    }
+    EncodeTiled enc = encode_tiled();
+    if (!enc) ABK_REFUSE("the driver gives no cuTensorMapEncodeTiled");
+    if (((uintptr_t)ptr & 15) || size % 8 || pitch % 8) ABK_REFUSE("heads for TMA must be 16-byte aligned, of a multiple of 8 elements");
+    cuuint64_t dims[3] = {(cuuint64_t)size, (cuuint64_t)heads, (cuuint64_t)rows};
+    cuuint64_t strides[2] = {(cuuint64_t)size * 2, (cuuint64_t)pitch * 2};
+    cuuint32_t box[3] = {64, 1, (cuuint32_t)box_rows}, elem[3] = {1, 1, 1};
+    CUresult r = enc(out, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, (void *)ptr, dims, strides, box, elem, CU_TENSOR_MAP_INTERLEAVE_NONE,
+                     CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+    if (r != CUDA_SUCCESS) ABK_REFUSE("cuTensorMapEncodeTiled failed with %d", (int)r);
+    if (cache.size() > 4096) cache.clear();
+    cache[key] = *out;
+    return 0;
+}
+
 }  // namespace tmap

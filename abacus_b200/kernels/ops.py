@@ -1521,15 +1521,9 @@ def attention_sigmoid_general(qkv, out, n_heads, n_kv_heads, head_dim, vd, row, 
 def attention_sigmoid_prompt_takes(qkv, n_heads, n_kv_heads, head_dim, vd, row):
     """Whether the tensor-core kernel for whole prompts takes these sizes: bfloat16, up to 32 heads, heads and values of
     multiples of 8 (values up to 128), every part of a row 16-byte aligned, and what a CTA holds of shared memory."""
-    if not (qkv.dtype == torch.bfloat16 and n_heads <= 32 and head_dim % 8 == 0 and vd % 8 == 0 and vd <= 128 and row % 8 == 0
-            and qkv.data_ptr() % 16 == 0):
-        return False
-    # (as csrc/attention_sigmoid_prompt.cu lays it out, with 16 keys a tile)
-    warps = 4 if n_heads <= 4 else 8 if n_heads <= 8 else 16
-    per, pitch_k, pitch_v = n_heads // n_kv_heads, -(-head_dim // 16) * 32 + 16, -(-vd // 16) * 32 + 16
-    values = max((min((b + 1) * warps, n_heads) - 1) // per - b * warps // per + 1 for b in range(-(-n_heads // warps)))
-    chunk = max(-(-n_heads // 16) * 16 * 64, warps * 96) + 16
-    return 16 * (n_heads * pitch_k + n_kv_heads * pitch_k + values * pitch_v + chunk) <= 227 * 1024
+    return (qkv.dtype == torch.bfloat16 and head_dim % 8 == 0 and vd % 8 == 0 and row % 8 == 0 and qkv.data_ptr() % 16 == 0
+            and load_module("attention_sigmoid_prompt").abk_attention_sigmoid_prompt_takes(_i(n_heads), _i(n_kv_heads), _i(head_dim),
+                                                                                           _i(vd)) != 0)
 
 
 def attention_sigmoid_prompt(qkv, out, n_heads, n_kv_heads, head_dim, vd, row, scale, batch, softcap, slopes, shift, mix, ranks=0):
@@ -1539,9 +1533,9 @@ def attention_sigmoid_prompt(qkv, out, n_heads, n_kv_heads, head_dim, vd, row, s
     if batch.any_continuation:
         raise KernelRefused("attention_sigmoid_prompt reads keys from the step's rows: every sequence must start at position 0")
     _check(lib, lib.abk_attention_sigmoid_prompt(
-        _p(qkv), _ll(row), _p(out), _i(n_heads), _i(n_kv_heads), _i(head_dim), _i(vd), _i(n_heads * head_dim),
+        _p(qkv), _ll(row), _i(n), _p(out), _i(n_heads), _i(n_kv_heads), _i(head_dim), _i(vd), _i(n_heads * head_dim),
         _i((n_heads + n_kv_heads) * head_dim), _f(scale), _f(softcap or 0.0), _p(slopes), _p(shift), _p(mix), _p(batch.seq_start),
-        _i(n_seqs), _i((n + 15) // 16 + n_seqs), _i(ranks), _stream()), "attention_sigmoid_prompt")
+        _i(n_seqs), _i((n + 15) // 16 + n_seqs), _i(ranks), _p(_Scratch.of(qkv.device).status), _stream()), "attention_sigmoid_prompt")
 
 
 def attention_sigmoid_decode_parts(qkv, n, n_heads, n_kv_heads, head_dim, vd, cache, max_keys):
