@@ -62,8 +62,37 @@ struct SigmoidPromptSmem {
     }
 };
 
-// WPH: warps a head. PAIR: more than 16 heads, two CTAs of the cluster side by side. EXACT: 16 / WPH heads a CTA, D a multiple
-// of 64, values of 128: nothing in the inner loops depends on a size that is only known at run time.
+// ldmatrix and shared-memory accesses at a register's address plus a constant, which goes into the instruction: the inner
+// loops' addresses differ by constants, and a warp's time is the instructions it waits for, one after the other.
+template <int OFF> __device__ __forceinline__ void ldsm_at(uint32_t addr, uint32_t *r) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4+%5];"
+                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr), "n"(OFF));
+}
+template <int OFF> __device__ __forceinline__ void ldsm_t_at(uint32_t addr, uint32_t *r) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4+%5];"
+                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr), "n"(OFF));
+}
+template <int OFF> __device__ __forceinline__ float lds_at(uint32_t addr) {
+    float v;
+    asm volatile("ld.shared.f32 %0, [%1+%2];" : "=f"(v) : "r"(addr), "n"(OFF));
+    return v;
+}
+template <int OFF> __device__ __forceinline__ void sts_at(uint32_t addr, uint32_t v) {
+    asm volatile("st.shared.b32 [%0+%1], %2;" ::"r"(addr), "n"(OFF), "r"(v) : "memory");
+}
+// f(0), f(1), .. f(N - 1), each with its number as a constant (decltype(i)::value)
+template <int I> struct Number {
+    static constexpr int value = I;
+};
+template <int N, int I = 0, typename F> __device__ __forceinline__ void each(F &&f) {
+    if constexpr (I < N) {
+        f(Number<I>{});
+        each<N, I + 1>(f);
+    }
+}
+
+// WPH: warps a head. PAIR: more than 16 heads, two CTAs of the cluster side by side. EXACT: 16 / WPH heads a CTA, heads and
+// values of 128: nothing in the inner loops depends on a size that is only known at run time.
 template <int WPH, bool CAP, bool EXACT, bool PAIR>
 __global__ void __launch_bounds__(SP_THREADS, 1) attention_sigmoid_prompt_kernel(const __grid_constant__ CUtensorMap map_q,
                                                                                  const __grid_constant__ CUtensorMap map_k,
@@ -125,29 +154,32 @@ __global__ void __launch_bounds__(SP_THREADS, 1) attention_sigmoid_prompt_kernel
     // has no visible key)
     const int my_tiles = PAIR ? (key_tiles + ranks - 1) / ranks : rank < key_tiles ? (key_tiles - rank + ranks - 1) / ranks : 0;
 
-    // warp 0 asks for this CTA's i-th tile of keys (with the queries, the first time) and of values
+    // This CTA's i-th tile of keys (with the queries, the first time) and of values: a warp asks for every 16th box, so that no
+    // warp falls behind the others, and one thread says how many bytes are to come (some may have come by then).
+    const int k_count = kv_n * sm.k_boxes, v_count = kv_n * sm.v_boxes, q_count = heads_n * sm.k_boxes;
     auto load_keys = [&](int i) {
         const int s = p.k_stages == 2 ? i & 1 : 0, z = start + (rank + i * ranks) * NK;
-        if (lane == 0) tc::mbar_expect_tx(&k_full[s], kv_n * sm.k_boxes * (NK * 128) + (i == 0 ? heads_n * sm.k_boxes * (SP_ROWS * 128) : 0));
+        if (threadIdx.x == 0) tc::mbar_expect_tx(&k_full[s], k_count * (NK * 128) + (i == 0 ? q_count * (SP_ROWS * 128) : 0));
+        if (lane == 0) {
+            if (i == 0)
+                for (int e = warp; e < q_count; e += SP_WARPS)
+                    tc::tma_load_3d(q_s + e * (SP_ROWS * 128), &map_q, (e % sm.k_boxes) * 64, h0 + e / sm.k_boxes, start + r0, &k_full[s]);
+            for (int e = warp; e < k_count; e += SP_WARPS)
+                tc::tma_load_3d(k_s + s * sm.k + e * (NK * 128), &map_k, (e % sm.k_boxes) * 64, kv0 + e / sm.k_boxes, z, &k_full[s]);
+        }
         __syncwarp();
-        if (i == 0)
-            for (int e = lane; e < heads_n * sm.k_boxes; e += 32)
-                tc::tma_load_3d(q_s + e * (SP_ROWS * 128), &map_q, (e % sm.k_boxes) * 64, h0 + e / sm.k_boxes, start + r0, &k_full[s]);
-        for (int e = lane; e < kv_n * sm.k_boxes; e += 32)
-            tc::tma_load_3d(k_s + s * sm.k + e * (NK * 128), &map_k, (e % sm.k_boxes) * 64, kv0 + e / sm.k_boxes, z, &k_full[s]);
     };
     auto load_values = [&](int i) {
         const int z = start + (rank + i * ranks) * NK;
-        if (lane == 0) tc::mbar_expect_tx(&v_full, kv_n * sm.v_boxes * (NK * 128));
+        if (threadIdx.x == 0) tc::mbar_expect_tx(&v_full, v_count * (NK * 128));
+        if (lane == 0)
+            for (int e = warp; e < v_count; e += SP_WARPS)
+                tc::tma_load_3d(v_s + e * (NK * 128), &map_v, (e % sm.v_boxes) * 64, kv0 + e / sm.v_boxes, z, &v_full);
         __syncwarp();
-        for (int e = lane; e < kv_n * sm.v_boxes; e += 32)
-            tc::tma_load_3d(v_s + e * (NK * 128), &map_v, (e % sm.v_boxes) * 64, kv0 + e / sm.v_boxes, z, &v_full);
     };
     int k_asked = 0, v_asked = 0;
-    if (warp == 0) {
-        for (; k_asked < my_tiles && k_asked < p.k_stages; k_asked++) load_keys(k_asked);
-        if (my_tiles > 0) load_values(0), v_asked = 1;
-    }
+    for (; k_asked < my_tiles && k_asked < p.k_stages; k_asked++) load_keys(k_asked);
+    if (my_tiles > 0) load_values(0), v_asked = 1;
 
     float o[VT][4];
 #pragma unroll
@@ -161,6 +193,9 @@ __global__ void __launch_bounds__(SP_THREADS, 1) attention_sigmoid_prompt_kernel
     const uint32_t qa = q_s + (hg - h0) * sm.k_boxes * (SP_ROWS * 128) + row_a;
     const uint32_t kb = k_s + kv_of * sm.k_boxes * (NK * 128) + part * 2048 + row_k;
     const uint32_t vb = v_s + kv_of * sm.v_boxes * (NK * 128) + row_a;
+    uint32_t qx4[4], xk4[4], vx4[4];  // the four places of 16 columns within a box
+#pragma unroll
+    for (int c4 = 0; c4 < 4; c4++) qx4[c4] = qa + (x_a ^ (c4 << 5)), xk4[c4] = x_k ^ (c4 << 5), vx4[c4] = vb + (x_a ^ (c4 << 5));
     const uint32_t pb = p_s + (lane & 15) * sm.p_row + hl * 32 + (lane >> 4) * 16;
     // this thread's weights: query row r8 of the warp's 16 keys, the two keys 2 q2, + 1
     const uint32_t wb = w_s + (part * SP_ROWS + r8) * sm.w_row + ((hg >> 1) + (hg & 1) * (heads_in >> 1)) * 32 + q2 * 8;
@@ -176,19 +211,31 @@ __global__ void __launch_bounds__(SP_THREADS, 1) attention_sigmoid_prompt_kernel
 #pragma unroll
         for (int t = 0; t < 2; t++) c[t][0] = c[t][1] = c[t][2] = c[t][3] = 0.0f;
         uint32_t qx = qa, kx = kb + s * sm.k;
-        for (int left = d_steps; left > 0; left -= 4, qx += SP_ROWS * 128, kx += NK * 128) {
+        if constexpr (EXACT) {
+            each<8>([&](auto step) {
+                constexpr int c4 = decltype(step)::value % 4, box = decltype(step)::value / 4;
+                uint32_t a[4], b[4];
+                ldsm_at<box * SP_ROWS * 128>(qx4[c4], a);
+                ldsm_at<box * NK * 128>(kx + xk4[c4], b);
+                mma_bf16(c[0], a, b[0], b[1]);
+                mma_bf16(c[1], a, b[2], b[3]);
+            });
+        } else {
+            for (int left = d_steps; left > 0; left -= 4, qx += SP_ROWS * 128, kx += NK * 128) {
 #pragma unroll
-            for (int c4 = 0; c4 < 4; c4++) {
-                if (EXACT || c4 < left) {
-                    uint32_t a[4], b0, b1, b2, b3;
-                    ldsm_x4(qx + (x_a ^ (c4 << 5)), a[0], a[1], a[2], a[3]);
-                    ldsm_x4(kx + (x_k ^ (c4 << 5)), b0, b1, b2, b3);
-                    mma_bf16(c[0], a, b0, b1);
-                    mma_bf16(c[1], a, b2, b3);
+                for (int c4 = 0; c4 < 4; c4++) {
+                    if (c4 < left) {
+                        uint32_t a[4], b0, b1, b2, b3;
+                        ldsm_x4(qx + (x_a ^ (c4 << 5)), a[0], a[1], a[2], a[3]);
+                        ldsm_x4(kx + (x_k ^ (c4 << 5)), b0, b1, b2, b3);
+                        mma_bf16(c[0], a, b0, b1);
+                        mma_bf16(c[1], a, b2, b3);
+                    }
                 }
             }
         }
-        const float back = (float)(r0 + r8 - key0 - 2 * q2);  // of this thread's first row and key
+        const int first_back = r0 + r8 - key0 - 2 * q2;
+        const float back = (float)first_back;  // of this thread's first row and key
         const float away_a = fmaf(hd.slope, back, hd.base), away_b = fmaf(hd.slope, 8.0f, away_a);
 #pragma unroll
         for (int t = 0; t < 2; t++) {
@@ -218,43 +265,44 @@ __global__ void __launch_bounds__(SP_THREADS, 1) attention_sigmoid_prompt_kernel
             }
         }
     };
-    // tile i's weights mixed, a query row's 16 keys at a time
+    // tile i's weights mixed, a query row's 16 keys at a time (warp w has query row w, of the first 16 keys, then of the next)
+    const uint32_t mix_from = w_s + warp * sm.w_row + q2 * 32 + r8 * 4, mix_to = p_s + warp * sm.p_row + r8 * 32 + q2 * 4;
     auto mixing = [&](int i) {
 #pragma unroll
         for (int c = 0; c < WPH; c++) {
-            const int row = warp + c * SP_WARPS;  // (query row, 16 keys): 16 rows of the first 16 keys, then of the next
-            const float *w = (const float *)(sp_smem + (w_s - q_s) + (PAIR ? (i & 1) * buffer : 0) + row * sm.w_row) + q2 * 8 + r8;
-            const int odd = heads_in * 4;         // from an even head's weights to the next head's
+            const uint32_t w = mix_from + (PAIR ? (i & 1) * buffer : 0) + c * SP_WARPS * sm.w_row;
+            const uint32_t w_odd = w + heads_in * 16;  // an odd head's weights
             float m[2][4];
 #pragma unroll
             for (int half = 0; half < 2; half++) m[half][0] = m[half][1] = m[half][2] = m[half][3] = 0.0f;
-#pragma unroll
-            for (int s = 0; s < BLOCKS; s++) {
+            each<BLOCKS>([&](auto block) {
+                constexpr int s = decltype(block)::value;
                 const int gi = 16 * s + 2 * q2;   // (heads that are not there left nothing)
                 const bool in0 = EXACT || gi < H, in1 = EXACT || gi + 1 < H;
                 const bool in8 = EXACT ? WPH == 1 : gi + 8 < H, in9 = EXACT ? WPH == 1 : gi + 9 < H;
 #pragma unroll
                 for (int half = 0; half < 2; half++) {
-                    const float *at = w + half * heads_in * 8 + s * 64;
-                    const float x0 = in0 ? at[0] : 0.0f, x1 = in1 ? at[odd] : 0.0f, x8 = in8 ? at[32] : 0.0f, x9 = in9 ? at[odd + 32] : 0.0f;
+                    const uint32_t even = w + half * heads_in * 32, uneven = w_odd + half * heads_in * 32;
+                    const float x0 = in0 ? lds_at<s * 256>(even) : 0.0f, x1 = in1 ? lds_at<s * 256>(uneven) : 0.0f;
+                    const float x8 = in8 ? lds_at<s * 256 + 128>(even) : 0.0f, x9 = in9 ? lds_at<s * 256 + 128>(uneven) : 0.0f;
                     uint32_t b0[3], b1[3];
                     split3_pair(x0, x1, b0), split3_pair(x8, x9, b1);
 #pragma unroll
                     for (int k = 2; k >= 0; k--) mma_bf16(m[half], ta[s], b0[k], b1[k]);
                 }
-            }
-            const uint32_t to = p_s + row * sm.p_row + r8 * 32 + q2 * 4;
-#pragma unroll
-            for (int half = 0; half < 2; half++) {
+            });
+            const uint32_t to = mix_to + c * SP_WARPS * sm.p_row;
+            each<2>([&](auto which) {
+                constexpr int half = decltype(which)::value;
                 uint32_t lo[3], hi[3];
                 split3_pair(m[half][0], m[half][1], lo);
                 if (WPH == 1) split3_pair(m[half][2], m[half][3], hi);
-#pragma unroll
-                for (int k = 0; k < 3; k++) {
-                    asm volatile("st.shared.b32 [%0], %1;" ::"r"(to + k * HEADS * 32 + half * 16), "r"(lo[k]) : "memory");
-                    if (WPH == 1) asm volatile("st.shared.b32 [%0], %1;" ::"r"(to + k * HEADS * 32 + half * 16 + 8 * 32), "r"(hi[k]) : "memory");
-                }
-            }
+                each<3>([&](auto piece) {
+                    constexpr int k = decltype(piece)::value;
+                    sts_at<k * HEADS * 32 + half * 16>(to, lo[k]);
+                    if (WPH == 1) sts_at<k * HEADS * 32 + half * 16 + 8 * 32>(to, hi[k]);
+                });
+            });
         }
     };
     // every weight of tile i is there (PAIR: from both CTAs); its keys, and the values and mixed weights of the tile before, are
@@ -270,7 +318,7 @@ __global__ void __launch_bounds__(SP_THREADS, 1) attention_sigmoid_prompt_kernel
         scores(0);
         meet();
         bad = failed[0];
-        if (warp == 0 && k_asked < my_tiles && !bad) load_keys(k_asked), k_asked++;
+        if (k_asked < my_tiles && !bad) load_keys(k_asked), k_asked++;
         mixing(0);
         __syncthreads();
     }
@@ -292,16 +340,30 @@ __global__ void __launch_bounds__(SP_THREADS, 1) attention_sigmoid_prompt_kernel
                 uint32_t a[3][4];
 #pragma unroll
                 for (int k = 0; k < 3; k++) ldsm_x4(pb + c * SP_ROWS * sm.p_row + k * HEADS * 32, a[k][0], a[k][1], a[k][2], a[k][3]);
-#pragma unroll
-                for (int tp = 0; tp < VT / 2; tp++) {
-                    const int gt = part * (VT / 2) + tp;  // the pair of column tiles within the head
-                    if (EXACT || 2 * gt < n_vt) {
-                        uint32_t b0, b1, b2, b3;
-                        ldsm_x4_t(vb + (gt >> 2) * (NK * 128) + c * 2048 + (x_a ^ ((gt & 3) << 5)), b0, b1, b2, b3);
+                if constexpr (EXACT) {
+                    const uint32_t base = c * 2048 + part * (VT / 8) * (NK * 128);  // (a warp's columns are whole boxes)
+                    each<VT / 2>([&](auto tile) {
+                        constexpr int tp = decltype(tile)::value;
+                        uint32_t b[4];
+                        ldsm_t_at<(tp >> 2) * NK * 128>(vx4[tp & 3] + base, b);
 #pragma unroll
                         for (int k = 0; k < 3; k++) {
-                            mma_bf16(o[2 * tp], a[k], b0, b1);
-                            mma_bf16(o[2 * tp + 1], a[k], b2, b3);
+                            mma_bf16(o[2 * tp], a[k], b[0], b[1]);
+                            mma_bf16(o[2 * tp + 1], a[k], b[2], b[3]);
+                        }
+                    });
+                } else {
+#pragma unroll
+                    for (int tp = 0; tp < VT / 2; tp++) {
+                        const int gt = part * (VT / 2) + tp;  // the pair of column tiles within the head
+                        if (2 * gt < n_vt) {
+                            uint32_t b0, b1, b2, b3;
+                            ldsm_x4_t(vb + (gt >> 2) * (NK * 128) + c * 2048 + (x_a ^ ((gt & 3) << 5)), b0, b1, b2, b3);
+#pragma unroll
+                            for (int k = 0; k < 3; k++) {
+                                mma_bf16(o[2 * tp], a[k], b0, b1);
+                                mma_bf16(o[2 * tp + 1], a[k], b2, b3);
+                            }
                         }
                     }
                 }
@@ -310,7 +372,7 @@ __global__ void __launch_bounds__(SP_THREADS, 1) attention_sigmoid_prompt_kernel
         if (it + 1 == my_tiles) break;
         meet();
         bad = bad || failed[(it + 1) & 1];
-        if (warp == 0 && !bad) {
+        if (!bad) {
             load_values(v_asked), v_asked++;
             if (k_asked < my_tiles) load_keys(k_asked), k_asked++;
         }
@@ -434,7 +496,7 @@ extern "C" int abk_attention_sigmoid_prompt(const void *qkv, long long row, int 
     if ((long long)tiles * ranks * blocks > 0x7fffffffLL) ABK_REFUSE("attention_sigmoid_prompt: %d tiles are more than a grid takes", tiles);
     cudaStream_t s = (cudaStream_t)stream;
     // the sizes of larger models have kernels of their own
-    const bool exact = n_heads == 16 / plan.wph * blocks && head_dim % 64 == 0 && v_dim == 128;
+    const bool exact = n_heads == 16 / plan.wph * blocks && head_dim == 128 && v_dim == 128;
 #define SP_RUN(WPH, CAP, EXACT, PAIR) sp_launch<WPH, CAP, EXACT, PAIR>(mq, mk, mv, p, ranks * blocks, plan.smem, s)
 #define SP_BY_SIZE(WPH, CAP, PAIR) (exact ? SP_RUN(WPH, CAP, true, PAIR) : SP_RUN(WPH, CAP, false, PAIR))
     if (plan.pair) return softcap > 0.0f ? SP_BY_SIZE(1, true, true) : SP_BY_SIZE(1, false, true);
