@@ -4,10 +4,12 @@
 // The heads' weights are mixed per key, so a CTA takes a run of a row's keys for all heads. A row's keys are dealt to
 // `n_parts` CTAs in runs of whole stages; a CTA walks its run in stages of KP keys of every kv head, keys and values, which
 // TMA brings through a ring of stages (128-byte swizzle, a box of KP rows x 64 columns at a time):
-//   scores    keys are the 16 rows and a group's query heads the columns of a warp-level tensor-core tile, float32 sums
-//   weights   the sigmoids, then the mixing, in float32 on the CUDA cores (a key has heads x heads multiply-adds)
-//   values    a tile of 16 value columns x the group's heads, summed over the keys on the tensor cores, the weights as three
-//             bfloat16 parts that hold their 24 bits
+//   scores    keys are the 16 rows and a group's query heads the columns of a warp-level tensor-core tile, float32 sums; the
+//             lanes that hold them make the weights, float32, into shared memory
+//   values    a tile of 16 value columns x the group's heads, summed over the keys on the tensor cores. A lane mixes the
+//             weights of the keys and the head its fragment holds (heads multiply-adds each, float32) and splits them into
+//             three bfloat16 parts that hold their 24 bits
+// with one barrier a stage between the two (weights in two buffers; a stage is refilled behind the next one's barrier).
 // Since nothing is normalized over the keys, a CTA's sums are its part of the output; attention_sigmoid_fold adds the
 // parts of a row in order. How a row is cut depends on its own position and on n_parts.
 #define ABK_DEFINE_ERROR
@@ -43,14 +45,15 @@ __host__ __device__ inline int sd_span(int keys, int n_parts, int kp) {
 
 // The parts of shared memory behind the ring of stages (bytes).
 struct SigmoidDecodeSmem {
-    int k_boxes, v_boxes, stage, pitch_q, pitch_w, q, w, mix, head, total;
+    int k_boxes, v_boxes, stage, pitch_q, pitch_w, rows_w, pitch_m, q, w, mix, head, total;
     __host__ __device__ SigmoidDecodeSmem(int H, int G, int D, int VD, int kp, int stages) {
         k_boxes = (D + 63) / 64, v_boxes = (VD + 63) / 64;
         stage = G * (k_boxes + v_boxes) * kp * 128;
         pitch_q = (D + 15) / 16 * 16 + 8;  // elements of a query head's row
-        pitch_w = kp + 8;                  // floats of a head's weights: rows of a fragment in different banks
-        q = H * pitch_q * 2, w = H * pitch_w * 4, mix = (H * H * 4 + 15) & ~15, head = H * (int)sizeof(SigmoidHead);
-        total = 1024 + stages * stage + q + 2 * w + mix + ((head + 15) & ~15) + 64;
+        pitch_w = kp + 8;                  // floats of a head's weights
+        rows_w = (H + 3) & ~3, pitch_m = rows_w + 4;
+        q = H * pitch_q * 2, w = rows_w * pitch_w * 4, mix = H * pitch_m * 4, head = H * (int)sizeof(SigmoidHead);  // (w: a buffer)
+        total = 1024 + stages * stage + q + 2 * w + mix + head + 64;
     }
 };
 
@@ -63,8 +66,8 @@ template <int UNITS, int NT> __global__ void __launch_bounds__(SD_THREADS) atten
     const int H = p.n_heads, G = p.n_kv_heads, D = p.head_dim, VD = p.v_dim, R = H / G, kp = p.kp;
     const SigmoidDecodeSmem sm(H, G, D, VD, kp, p.stages);
     __nv_bfloat16 *q_s = (__nv_bfloat16 *)(ring + p.stages * sm.stage);
-    float *a_s = (float *)((uint8_t *)q_s + sm.q), *m_s = a_s + H * sm.pitch_w, *mix_s = m_s + H * sm.pitch_w;
-    SigmoidHead *head_s = (SigmoidHead *)((uint8_t *)mix_s + sm.mix);
+    float *const a_s = (float *)((uint8_t *)q_s + sm.q), *const mix_s = a_s + 2 * sm.w / 4;
+    SigmoidHead *const head_s = (SigmoidHead *)((uint8_t *)mix_s + sm.mix);
     __shared__ uint64_t full[SD_MAX_STAGES];
     __shared__ int failed[2];  // by the stage's parity: set before a stage's barriers, read after them
     const int part = blockIdx.x, t = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, r8 = lane >> 2, q2 = lane & 3;
@@ -74,8 +77,11 @@ template <int UNITS, int NT> __global__ void __launch_bounds__(SD_THREADS) atten
         tc::mbar_init_fence();
         tc::tma_prefetch_map(&map_k), tc::tma_prefetch_map(&map_v);
     }
-    if (p.mix)
-        for (int e = tid; e < H * H; e += SD_THREADS) mix_s[e] = p.mix[e];
+    for (int e = tid; e < H * sm.rows_w; e += SD_THREADS) {  // (columns that no head has: zeros, for weights of zero)
+        const int h = e / sm.rows_w, g = e - h * sm.rows_w;
+        mix_s[h * sm.pitch_m + g] = g >= H ? 0.0f : p.mix ? p.mix[h * H + g] : h == g ? 1.0f : 0.0f;
+    }
+    for (int e = H * sm.pitch_w + tid; e < sm.w / 4; e += SD_THREADS) a_s[e] = a_s[sm.w / 4 + e] = 0.0f;
     if (tid < H) head_s[tid] = sigmoid_head(p.scale, p.softcap, p.slopes ? p.slopes[tid] : 0.0f, p.shift ? p.shift[tid] : 0.0f);
     __syncthreads();
     pdl_wait();
@@ -84,30 +90,41 @@ template <int UNITS, int NT> __global__ void __launch_bounds__(SD_THREADS) atten
     const int pos = p.token_pos[t], slot = p.seq_slot[seq], span = sd_span(pos + 1, p.n_parts, kp), first = part * span;
     if (first > pos) return;  // (the fold knows how many parts a row has)
     const int n_keys = min(span, pos + 1 - first), n_st = (n_keys + kp - 1) / kp, box = kp * 128;
-    // a stage's boxes, kv head by kv head (a lane issues every 32nd), keys first; a stage lies within a page (kp divides it)
-    auto issue = [&](int st) {  // warp 0
-        const int s = st % p.stages, j = first + st * kp, page = cache_page(p.cache, slot, j), at = j % p.cache.tokens_per_page;
-        if (lane == 0) tc::mbar_expect_tx(&full[s], sm.stage);
-        __syncwarp();
-        for (int g = lane; g < G; g += 32) {
-            const int row = (page * G + g) * p.cache.tokens_per_page + at;
-            uint8_t *k = ring + s * sm.stage + g * sm.k_boxes * box, *v = ring + s * sm.stage + (G * sm.k_boxes + g * sm.v_boxes) * box;
-            for (int b = 0; b < sm.k_boxes; b++) tc::tma_load_2d(k + b * box, &map_k, b * 64, row, &full[s]);
-            for (int b = 0; b < sm.v_boxes; b++) tc::tma_load_2d(v + b * box, &map_v, b * 64, row, &full[s]);
+    // a stage's boxes, keys and values of every eighth kv head a warp, so that no warp falls behind the others; one thread says
+    // how many bytes are to come (some may have come by then). A stage lies within a page (kp divides its PAGE tokens).
+    int to_stage = 0, from_stage = 0, phase = 0;  // where the next boxes go; the stage that is read next, and its barrier's phase
+    auto issue = [&](int st) {
+        const int j = first + st * kp;
+        uint64_t *const bar = &full[to_stage];
+        if (tid == 0) tc::mbar_expect_tx(bar, sm.stage);
+        if (lane == 0) {
+            const int page = p.cache.page_table[(long long)slot * p.cache.table_width + j / PAGE];
+            uint8_t *const base = ring + to_stage * sm.stage;
+            for (int g = warp; g < G; g += SD_WARPS) {
+                const int row = (page * G + g) * PAGE + j % PAGE;
+                uint8_t *const k = base + g * sm.k_boxes * box, *const v = base + (G * sm.k_boxes + g * sm.v_boxes) * box;
+                for (int b = 0; b < sm.k_boxes; b++) tc::tma_load_2d(k + b * box, &map_k, b * 64, row, bar);
+                for (int b = 0; b < sm.v_boxes; b++) tc::tma_load_2d(v + b * box, &map_v, b * 64, row, bar);
+            }
         }
+        __syncwarp();
+        if (++to_stage == p.stages) to_stage = 0;
     };
     int issued = 0;
-    if (warp == 0)
-        for (; issued < n_st && issued < p.stages; issued++) issue(issued);
-    const int d16 = (D + 15) / 16 * 16, tiles16 = kp > 8 ? kp / 16 : 1, half15 = kp > 8 ? 15 : 7;
+    for (; issued < n_st && issued < p.stages; issued++) issue(issued);
+    const int d16 = (D + 15) / 16 * 16, tiles_log = kp > 32 ? 2 : kp > 16 ? 1 : 0, half15 = kp > 8 ? 15 : 7;
+    const bool capped = p.softcap > 0.0f;
     const __nv_bfloat16 *qg = p.q + (long long)t * p.q_row;
-    for (int e = tid; e < H * d16; e += SD_THREADS) {
-        const int h = e / d16, d = e - h * d16;
-        q_s[h * sm.pitch_q + d] = d < D ? qg[h * D + d] : __float2bfloat16_rn(0.0f);
+    for (int e = tid; e < H * (d16 / 8); e += SD_THREADS) {
+        const int h = e / (d16 / 8), d = (e - h * (d16 / 8)) * 8;
+        *(uint4 *)(q_s + h * sm.pitch_q + d) = d < D ? *(const uint4 *)(qg + h * D + d) : make_uint4(0, 0, 0, 0);
     }
     __syncthreads();
 
     const int col_tiles = (VD + 15) / 16, units = G * col_tiles, per_warp = (units + SD_WARPS - 1) / SD_WARPS, u0 = warp * per_warp;
+    const int g0 = u0 / col_tiles, ct0 = u0 - g0 * col_tiles;
+    // a lane's piece of 16 bytes under the swizzle: keys as rows, values transposed
+    const uint32_t x_a = ((lane >> 4) ^ (lane & 7)) << 4, x_v = (((lane >> 3) & 1) ^ (lane & 7)) << 4;
     float o[UNITS][NT][4];
 #pragma unroll
     for (int i = 0; i < UNITS; i++)
@@ -115,32 +132,48 @@ template <int UNITS, int NT> __global__ void __launch_bounds__(SD_THREADS) atten
         for (int c = 0; c < NT; c++) o[i][c][0] = o[i][c][1] = o[i][c][2] = o[i][c][3] = 0.0f;
 
     for (int st = 0; st < n_st; st++) {
-        const int s = st % p.stages, j0 = first + st * kp, nv = min(kp, n_keys - st * kp);
+        const int s = from_stage, j0 = first + st * kp, nv = min(kp, n_keys - st * kp);
+        float *const weights = a_s + (st & 1) * (sm.w / 4);
         const uint32_t k_s = tc::smem_addr(ring + s * sm.stage), v_s = k_s + G * sm.k_boxes * box;
-        if (!tc::mbar_wait(&full[s], (st / p.stages) & 1)) failed[st & 1] = 1;
+        if (!tc::mbar_wait(&full[s], phase)) failed[st & 1] = 1;
+        if (++from_stage == p.stages) from_stage = 0, phase ^= 1;
         // scores: a warp takes a kv head and 16 keys at a time
         // (a stage of 8 keys fills half of a tile: the other half repeats them and is dropped, here and below)
-        for (int u = warp; u < G * tiles16; u += SD_WARPS) {
-            const int g = u / tiles16, key = (u - g * tiles16) * 16;
+        for (int u = warp; u < G << tiles_log; u += SD_WARPS) {
+            const int g = u >> tiles_log, key = (u - (g << tiles_log)) * 16;
             float c[NT][4];
 #pragma unroll
             for (int i = 0; i < NT; i++) c[i][0] = c[i][1] = c[i][2] = c[i][3] = 0.0f;
-            const uint32_t kb = k_s + g * sm.k_boxes * box;
-#pragma unroll 4
-            for (int ks = 0; ks < d16 / 16; ks++) {
-                uint32_t a[4];
-                ldsm_x4(sw128(kb + (ks >> 2) * box, key + (lane & half15), (ks & 3) * 2 + (lane >> 4)), a[0], a[1], a[2], a[3]);
+            uint32_t kb = k_s + g * sm.k_boxes * box + (key + (lane & half15)) * 128;
+            const uint32_t *qr[NT];  // (columns beyond the group's heads repeat a head and are dropped)
 #pragma unroll
-                for (int i = 0; i < NT; i++) {
-                    const int hl = 8 * i + r8;
-                    const uint32_t *qr = (const uint32_t *)(q_s + (g * R + (hl < R ? hl : 0)) * sm.pitch_q + ks * 16 + 2 * q2);
-                    mma_bf16(c[i], a, hl < R ? qr[0] : 0u, hl < R ? qr[4] : 0u);
+            for (int i = 0; i < NT; i++) qr[i] = (const uint32_t *)(q_s + (g * R + min(8 * i + r8, R - 1)) * sm.pitch_q) + q2;
+            for (int left = d16 / 16; left > 0; left -= 4, kb += box) {
+#pragma unroll
+                for (int c4 = 0; c4 < 4; c4++) {
+                    if (c4 < left) {
+                        uint32_t a[4];
+                        ldsm_x4(kb + (x_a ^ (c4 << 5)), a[0], a[1], a[2], a[3]);
+#pragma unroll
+                        for (int i = 0; i < NT; i++) mma_bf16(c[i], a, qr[i][8 * c4], qr[i][8 * c4 + 4]);
+                    }
                 }
+#pragma unroll
+                for (int i = 0; i < NT; i++) qr[i] += 32;
             }
+            // the weights of this lane's keys (rows) and heads (columns)
+            const float back = (float)(pos - j0 - key - r8);
+            const bool in_a = key + r8 < nv, in_b = key + r8 + 8 < nv;
 #pragma unroll
             for (int i = 0; i < NT; i++) {
                 const int hl = 8 * i + 2 * q2;
-                float *to = a_s + (g * R + hl) * sm.pitch_w + key + r8;
+                if (hl >= R) continue;
+                const SigmoidHead e = head_s[g * R + hl], f = head_s[g * R + (hl + 1 < R ? hl + 1 : hl)];
+                c[i][0] = in_a ? sigmoid_of(capped, e, c[i][0], fmaf(e.slope, back, e.base)) : 0.0f;
+                c[i][1] = in_a ? sigmoid_of(capped, f, c[i][1], fmaf(f.slope, back, f.base)) : 0.0f;
+                c[i][2] = in_b ? sigmoid_of(capped, e, c[i][2], fmaf(e.slope, back - 8.0f, e.base)) : 0.0f;
+                c[i][3] = in_b ? sigmoid_of(capped, f, c[i][3], fmaf(f.slope, back - 8.0f, f.base)) : 0.0f;
+                float *to = weights + (g * R + hl) * sm.pitch_w + key + r8;
                 if (hl < R) to[0] = c[i][0];
                 if (hl + 1 < R) to[sm.pitch_w] = c[i][1];
                 if (kp > 8) {
@@ -156,26 +189,22 @@ template <int UNITS, int NT> __global__ void __launch_bounds__(SD_THREADS) atten
                 *(uint4 *)(ring + s * sm.stage + (G * sm.k_boxes + g * sm.v_boxes + (c >> 3)) * box + key * 128 + (c & 7) * 16) = make_uint4(0, 0, 0, 0);
             }
         }
-        __syncthreads();
-        float *w_s = p.mix ? a_s : m_s;
-        for (int e = tid; e < H * kp; e += SD_THREADS) {
-            const int h = e / kp, j = e - h * kp;
-            const SigmoidHead hd = head_s[h];
-            w_s[h * sm.pitch_w + j] = j < nv ? sigmoid_of(p.softcap > 0.0f, hd, a_s[h * sm.pitch_w + j], fmaf(hd.slope, (float)(pos - j0 - j), hd.base)) : 0.0f;
+        __syncthreads();  // the stage's weights are there; the stage before is done with
+        if (failed[st & 1]) {
+            // a copy did not come: report it, and let the copies still in flight land (or run out of time) before the memory goes
+            if (tid == 0) atomicOr(p.status + 2, 1);
+            if (warp == 0)
+                for (int i = st + 1; i < issued; i++) {
+                    tc::mbar_wait(&full[from_stage], phase);
+                    if (++from_stage == p.stages) from_stage = 0, phase ^= 1;
+                }
+            return;
         }
-        __syncthreads();
-        if (p.mix) {
-            for (int e = tid; e < H * kp; e += SD_THREADS) {
-                const int h = e / kp, j = e - h * kp;
-                float m = 0.0f;
-                for (int g = 0; g < H; g++) m = fmaf(mix_s[h * H + g], a_s[g * sm.pitch_w + j], m);
-                m_s[h * sm.pitch_w + j] = m;
-            }
-            __syncthreads();
-        }
+        if (st > 0 && p.stages > 1 && issued < n_st) issue(issued), issued++;
         // values: this warp's tiles, which follow one another, so that a kv head's weights are split once
         for (int key = 0; key < kp && key < nv; key += 16) {
-            int g = u0 / col_tiles, ct = u0 - g * col_tiles, have = -1;
+            int g = g0, ct = ct0, have = -1;
+            const uint32_t vb = v_s + (key + (((lane & 7) + (lane >> 4) * 8) & half15)) * 128;
             uint32_t b0[NT][3], b1[NT][3];
 #pragma unroll
             for (int i = 0; i < UNITS; i++) {
@@ -185,17 +214,29 @@ template <int UNITS, int NT> __global__ void __launch_bounds__(SD_THREADS) atten
 #pragma unroll
                     for (int c = 0; c < NT; c++) {
                         const int hl = 8 * c + r8;
-                        const float *w = m_s + (g * R + (hl < R ? hl : 0)) * sm.pitch_w + key + 2 * q2;
-                        float2 lo = *(const float2 *)w, hi = make_float2(0.0f, 0.0f);
-                        if (kp > 8) hi = *(const float2 *)(w + 8);
-                        if (hl >= R) lo = hi = make_float2(0.0f, 0.0f);
+                        const float *w = weights + key + 2 * q2, *m = mix_s + (g * R + (hl < R ? hl : 0)) * sm.pitch_m;
+                        float2 lo = make_float2(0.0f, 0.0f), hi = lo;
+                        if (hl < R) {
+                            for (int from = 0; from < sm.rows_w; from += 4, w += 4 * sm.pitch_w) {
+                                const float4 mx = *(const float4 *)(m + from);
+                                const float by[4] = {mx.x, mx.y, mx.z, mx.w};
+#pragma unroll
+                                for (int u = 0; u < 4; u++) {
+                                    const float2 x = *(const float2 *)(w + u * sm.pitch_w);
+                                    lo.x = fmaf(by[u], x.x, lo.x), lo.y = fmaf(by[u], x.y, lo.y);
+                                    if (kp > 8) {
+                                        const float2 y = *(const float2 *)(w + u * sm.pitch_w + 8);
+                                        hi.x = fmaf(by[u], y.x, hi.x), hi.y = fmaf(by[u], y.y, hi.y);
+                                    }
+                                }
+                            }
+                        }
                         split3_pair(lo.x, lo.y, b0[c]), split3_pair(hi.x, hi.y, b1[c]);
                     }
                 }
                 // rows: 16 value columns; the fragment is the transposed tile of 16 keys x 16 columns
                 uint32_t a[4];
-                const int chunk = 2 * ct + ((lane >> 3) & 1);
-                ldsm_x4_t(sw128(v_s + (g * sm.v_boxes + (chunk >> 3)) * box, key + (((lane & 7) + (lane >> 4) * 8) & half15), chunk & 7), a[0], a[1], a[2], a[3]);
+                ldsm_x4_t(vb + (g * sm.v_boxes + (ct >> 2)) * box + (x_v ^ ((ct & 3) << 5)), a[0], a[1], a[2], a[3]);
 #pragma unroll
                 for (int c = 0; c < NT; c++)
 #pragma unroll
@@ -203,18 +244,13 @@ template <int UNITS, int NT> __global__ void __launch_bounds__(SD_THREADS) atten
                 if (++ct == col_tiles) ct = 0, g++;
             }
         }
-        __syncthreads();  // the stage and the weights are done with
-        if (warp == 0 && issued < n_st && !failed[st & 1]) issue(issued), issued++;
-        if (failed[st & 1]) {
-            // a copy did not come: report it, and let the copies still in flight land (or run out of time) before the memory goes
-            if (tid == 0) atomicOr(p.status + 2, 1);
-            if (warp == 0)
-                for (int i = st + 1; i < issued; i++) tc::mbar_wait(&full[i % p.stages], (i / p.stages) & 1);
-            return;
+        if (p.stages == 1) {  // (a ring of one: its next keys come in when everyone is done with these)
+            __syncthreads();
+            if (issued < n_st) issue(issued), issued++;
         }
     }
     float *dst = p.parts + ((long long)t * p.n_parts + part) * H * VD;
-    int g = u0 / col_tiles, ct = u0 - g * col_tiles;
+    int g = g0, ct = ct0;
 #pragma unroll
     for (int i = 0; i < UNITS; i++) {
         if (u0 + i >= units || i >= per_warp) break;
@@ -303,8 +339,8 @@ extern "C" int abk_attention_sigmoid_decode(const void *q, long long q_row, void
     if (n_tokens <= 0) return 0;
     if (!abk_attention_sigmoid_decode_parts(n_tokens, n_heads, n_kv_heads, head_dim, v_dim, 1) || n_parts < 1 || n_parts > 65535)
         ABK_REFUSE("attention_sigmoid_decode: %d heads of %d over %d kv heads with values of %d", n_heads, head_dim, n_kv_heads, v_dim);
-    if (tokens_per_page % 64 || pool_rows > 0x7fffffffLL) ABK_REFUSE("attention_sigmoid_decode: pages of %d tokens", tokens_per_page);
-    if (((uintptr_t)k_pool | (uintptr_t)v_pool | (uintptr_t)parts) & 15 || (uintptr_t)out & 7)
+    if (tokens_per_page != PAGE || pool_rows > 0x7fffffffLL) ABK_REFUSE("attention_sigmoid_decode: pages of %d tokens", tokens_per_page);
+    if ((((uintptr_t)k_pool | (uintptr_t)v_pool | (uintptr_t)parts | (uintptr_t)q) & 15) || q_row % 8 || (uintptr_t)out & 7)
         ABK_REFUSE("attention_sigmoid_decode: the cache's pools and the output must be 16-byte aligned");
     SigmoidDecode p;
     p.q = (const __nv_bfloat16 *)q, p.q_row = q_row, p.parts = parts, p.out = (__nv_bfloat16 *)out;
