@@ -9,7 +9,8 @@
 //   values    a tile of 16 value columns x the group's heads, summed over the keys on the tensor cores. A lane mixes the
 //             weights of the keys and the head its fragment holds (heads multiply-adds each, float32) and splits them into
 //             three bfloat16 parts that hold their 24 bits
-// with one barrier a stage between the two (weights in two buffers; a stage is refilled behind the next one's barrier).
+// A warp's time is the instructions it waits for one after the other, so two teams of eight warps take a run's stages in turns,
+// each with weights and barriers of its own, and add their sums at the end.
 // Since nothing is normalized over the keys, a CTA's sums are its part of the output; attention_sigmoid_fold adds the
 // parts of a row in order. How a row is cut depends on its own position and on n_parts.
 #define ABK_DEFINE_ERROR
@@ -19,8 +20,8 @@
 #include "tc_common.cuh"
 #include "tensor_map.cuh"
 
-#define SD_WARPS 8
-#define SD_THREADS (32 * SD_WARPS)
+#define SD_WARPS 8                     // a team
+#define SD_TEAM_THREADS (32 * SD_WARPS)
 #define SD_MAX_STAGES 4
 
 struct SigmoidDecode {
@@ -54,11 +55,25 @@ struct SigmoidDecodeSmem {
         rows_w = (H + 3) & ~3, pitch_m = rows_w + 4;
         q = H * pitch_q * 2, w = rows_w * pitch_w * 4, mix = H * pitch_m * 4, head = H * (int)sizeof(SigmoidHead);  // (w: a buffer)
         total = 1024 + stages * stage + q + 2 * w + mix + head + 64;
+        const int sums = 1024 + SD_WARPS * 16 * 512;  // the second team's, at the end, from the ring's start
+        if (total < sums) total = sums;
     }
 };
 
-// UNITS: tiles of 16 value columns a warp sums; NT: tiles of 8 heads a group has.
-template <int UNITS, int NT> __global__ void __launch_bounds__(SD_THREADS) attention_sigmoid_decode_kernel(const __grid_constant__ CUtensorMap map_k,
+// Waits until stage st is asked for; false if that took longer than the library's limit.
+__device__ __forceinline__ bool sd_asked(const volatile int *asked, int st) {
+    if (*asked < st) {
+        const uint64_t start = tc::global_ns(), limit = tc::abk_wait_limit_ns;
+        while (*asked < st)
+            if (tc::global_ns() - start > limit) return false;
+    }
+    __threadfence_block();
+    return true;
+}
+
+// UNITS: tiles of 16 value columns a warp sums; NT: tiles of 8 heads a group has. ONE: eight kv heads of UNITS tiles each, so that
+// a warp's tiles are one head's.
+template <int UNITS, int NT, bool ONE, int TEAMS> __global__ void __launch_bounds__(SD_TEAM_THREADS * TEAMS) attention_sigmoid_decode_kernel(const __grid_constant__ CUtensorMap map_k,
                                                                                                         const __grid_constant__ CUtensorMap map_v,
                                                                                                         SigmoidDecode p) {
     extern __shared__ uint8_t sd_raw[];
@@ -69,19 +84,23 @@ template <int UNITS, int NT> __global__ void __launch_bounds__(SD_THREADS) atten
     float *const a_s = (float *)((uint8_t *)q_s + sm.q), *const mix_s = a_s + 2 * sm.w / 4;
     SigmoidHead *const head_s = (SigmoidHead *)((uint8_t *)mix_s + sm.mix);
     __shared__ uint64_t full[SD_MAX_STAGES];
-    __shared__ int failed[2];  // by the stage's parity: set before a stage's barriers, read after them
-    const int part = blockIdx.x, t = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, r8 = lane >> 2, q2 = lane & 3;
+    // the last stage that was asked for into each place of the ring. A place's stages may belong to either team, and a barrier's
+    // parity alone does not tell a phase from the one after next: a team waits on a barrier only once its own stage is asked for
+    // (which is after the place's stage before had come and was read).
+    __shared__ volatile int asked[SD_MAX_STAGES];
+    __shared__ int failed[2][2];  // by team and the parity of its stages: set before a stage's first barrier, read after it
+    const int part = blockIdx.x, t = blockIdx.y, tid = threadIdx.x, team = TEAMS == 1 ? 0 : tid / SD_TEAM_THREADS, warp = (tid >> 5) % SD_WARPS, lane = tid & 31, r8 = lane >> 2, q2 = lane & 3;
     if (tid == 0) {
-        for (int s = 0; s < p.stages; s++) tc::mbar_init(&full[s], 1);
-        failed[0] = failed[1] = 0;
+        for (int s = 0; s < p.stages; s++) tc::mbar_init(&full[s], 1), asked[s] = -1;
+        failed[0][0] = failed[0][1] = failed[1][0] = failed[1][1] = 0;
         tc::mbar_init_fence();
         tc::tma_prefetch_map(&map_k), tc::tma_prefetch_map(&map_v);
     }
-    for (int e = tid; e < H * sm.rows_w; e += SD_THREADS) {  // (columns that no head has: zeros, for weights of zero)
+    for (int e = tid; e < H * sm.rows_w; e += SD_TEAM_THREADS * TEAMS) {  // (columns that no head has: zeros, for weights of zero)
         const int h = e / sm.rows_w, g = e - h * sm.rows_w;
         mix_s[h * sm.pitch_m + g] = g >= H ? 0.0f : p.mix ? p.mix[h * H + g] : h == g ? 1.0f : 0.0f;
     }
-    for (int e = H * sm.pitch_w + tid; e < sm.w / 4; e += SD_THREADS) a_s[e] = a_s[sm.w / 4 + e] = 0.0f;
+    for (int e = H * sm.pitch_w + tid; e < sm.w / 4; e += SD_TEAM_THREADS * TEAMS) a_s[e] = a_s[sm.w / 4 + e] = 0.0f;
     if (tid < H) head_s[tid] = sigmoid_head(p.scale, p.softcap, p.slopes ? p.slopes[tid] : 0.0f, p.shift ? p.shift[tid] : 0.0f);
     __syncthreads();
     pdl_wait();
@@ -91,12 +110,16 @@ template <int UNITS, int NT> __global__ void __launch_bounds__(SD_THREADS) atten
     if (first > pos) return;  // (the fold knows how many parts a row has)
     const int n_keys = min(span, pos + 1 - first), n_st = (n_keys + kp - 1) / kp, box = kp * 128;
     // a stage's boxes, keys and values of every eighth kv head a warp, so that no warp falls behind the others; one thread says
-    // how many bytes are to come (some may have come by then). A stage lies within a page (kp divides its PAGE tokens).
-    int to_stage = 0, from_stage = 0, phase = 0;  // where the next boxes go; the stage that is read next, and its barrier's phase
-    auto issue = [&](int st) {
+    // how many bytes are to come (some may have come by then). A stage lies within a page (kp divides its PAGE tokens). Stage st lies
+    // in place st % stages of the ring; the team that has read it asks for stage st + stages.
+    auto issue = [&](int st, int to_stage) {
         const int j = first + st * kp;
         uint64_t *const bar = &full[to_stage];
-        if (tid == 0) tc::mbar_expect_tx(bar, sm.stage);
+        if (warp == 0 && lane == 0) {
+            tc::mbar_expect_tx(bar, sm.stage);
+            __threadfence_block();
+            asked[to_stage] = st;
+        }
         if (lane == 0) {
             const int page = p.cache.page_table[(long long)slot * p.cache.table_width + j / PAGE];
             uint8_t *const base = ring + to_stage * sm.stage;
@@ -108,14 +131,12 @@ template <int UNITS, int NT> __global__ void __launch_bounds__(SD_THREADS) atten
             }
         }
         __syncwarp();
-        if (++to_stage == p.stages) to_stage = 0;
     };
-    int issued = 0;
-    for (; issued < n_st && issued < p.stages; issued++) issue(issued);
+    for (int st = team; st < n_st && st < p.stages; st += TEAMS) issue(st, st);
     const int d16 = (D + 15) / 16 * 16, tiles_log = kp > 32 ? 2 : kp > 16 ? 1 : 0, half15 = kp > 8 ? 15 : 7;
     const bool capped = p.softcap > 0.0f;
     const __nv_bfloat16 *qg = p.q + (long long)t * p.q_row;
-    for (int e = tid; e < H * (d16 / 8); e += SD_THREADS) {
+    for (int e = tid; e < H * (d16 / 8); e += SD_TEAM_THREADS * TEAMS) {
         const int h = e / (d16 / 8), d = (e - h * (d16 / 8)) * 8;
         *(uint4 *)(q_s + h * sm.pitch_q + d) = d < D ? *(const uint4 *)(qg + h * D + d) : make_uint4(0, 0, 0, 0);
     }
@@ -131,12 +152,21 @@ template <int UNITS, int NT> __global__ void __launch_bounds__(SD_THREADS) atten
 #pragma unroll
         for (int c = 0; c < NT; c++) o[i][c][0] = o[i][c][1] = o[i][c][2] = o[i][c][3] = 0.0f;
 
-    for (int st = 0; st < n_st; st++) {
-        const int s = from_stage, j0 = first + st * kp, nv = min(kp, n_keys - st * kp);
-        float *const weights = a_s + (st & 1) * (sm.w / 4);
+    auto meet = [&]() {  // the team's warps
+        if (TEAMS == 1) __syncthreads();
+        else {
+            __syncwarp();  // (the barrier counts whole warps: lanes that waited or took other ways are together again)
+            asm volatile("bar.sync %0, %1;" ::"r"(1 + team), "n"(SD_TEAM_THREADS) : "memory");
+        }
+    };
+    float *const weights = a_s + team * (sm.w / 4);
+    int s = team, phase = 0, turn = 0;  // the stage's place in the ring, its barrier's phase, the parity of the team's stages
+    bool bad = false;
+    for (int st = team; st < n_st; st += TEAMS, turn ^= 1) {
+        const int j0 = first + st * kp, nv = min(kp, n_keys - st * kp);
         const uint32_t k_s = tc::smem_addr(ring + s * sm.stage), v_s = k_s + G * sm.k_boxes * box;
-        if (!tc::mbar_wait(&full[s], phase)) failed[st & 1] = 1;
-        if (++from_stage == p.stages) from_stage = 0, phase ^= 1;
+        __syncwarp();
+        if (!(sd_asked(&asked[s], st) && tc::mbar_wait(&full[s], phase))) failed[team][turn] = 1;
         // scores: a warp takes a kv head and 16 keys at a time
         // (a stage of 8 keys fills half of a tile: the other half repeats them and is dropped, here and below)
         for (int u = warp; u < G << tiles_log; u += SD_WARPS) {
@@ -184,32 +214,28 @@ template <int UNITS, int NT> __global__ void __launch_bounds__(SD_THREADS) atten
         }
         if (nv < kp) {  // the last stage: rows beyond the token's key hold what the page held; they count as zeros
             const int per = sm.v_boxes * 8;
-            for (int e = tid; e < G * (kp - nv) * per; e += SD_THREADS) {
+            for (int e = tid - team * SD_TEAM_THREADS; e < G * (kp - nv) * per; e += SD_TEAM_THREADS) {
                 const int row = e / per, c = e - row * per, g = row / (kp - nv), key = nv + row - g * (kp - nv);
                 *(uint4 *)(ring + s * sm.stage + (G * sm.k_boxes + g * sm.v_boxes + (c >> 3)) * box + key * 128 + (c & 7) * 16) = make_uint4(0, 0, 0, 0);
             }
         }
-        __syncthreads();  // the stage's weights are there; the stage before is done with
-        if (failed[st & 1]) {
-            // a copy did not come: report it, and let the copies still in flight land (or run out of time) before the memory goes
-            if (tid == 0) atomicOr(p.status + 2, 1);
-            if (warp == 0)
-                for (int i = st + 1; i < issued; i++) {
-                    tc::mbar_wait(&full[from_stage], phase);
-                    if (++from_stage == p.stages) from_stage = 0, phase ^= 1;
-                }
-            return;
+        meet();  // the stage's weights are there
+        if (failed[team][turn]) {  // a copy did not come: let the team's copies still in flight land (or run out of time)
+            for (int i = 0; i < p.stages; i++)
+                if (asked[i] >= 0) tc::mbar_wait(&full[i], (asked[i] / p.stages) & 1);
+            bad = true;
+            break;
         }
-        if (st > 0 && p.stages > 1 && issued < n_st) issue(issued), issued++;
         // values: this warp's tiles, which follow one another, so that a kv head's weights are split once
         for (int key = 0; key < kp && key < nv; key += 16) {
             int g = g0, ct = ct0, have = -1;
+            const uint32_t one = ONE ? g0 * sm.v_boxes * box : 0;
             const uint32_t vb = v_s + (key + (((lane & 7) + (lane >> 4) * 8) & half15)) * 128;
             uint32_t b0[NT][3], b1[NT][3];
 #pragma unroll
             for (int i = 0; i < UNITS; i++) {
-                if (u0 + i >= units || i >= per_warp) break;
-                if (g != have) {
+                if (!ONE && (u0 + i >= units || i >= per_warp)) break;
+                if (ONE ? i == 0 : g != have) {
                     have = g;
 #pragma unroll
                     for (int c = 0; c < NT; c++) {
@@ -236,17 +262,39 @@ template <int UNITS, int NT> __global__ void __launch_bounds__(SD_THREADS) atten
                 }
                 // rows: 16 value columns; the fragment is the transposed tile of 16 keys x 16 columns
                 uint32_t a[4];
-                ldsm_x4_t(vb + (g * sm.v_boxes + (ct >> 2)) * box + (x_v ^ ((ct & 3) << 5)), a[0], a[1], a[2], a[3]);
+                if (ONE) ct = i;
+                ldsm_x4_t(vb + (ONE ? one + (i >> 2) * box : (g * sm.v_boxes + (ct >> 2)) * box) + (x_v ^ ((ct & 3) << 5)), a[0], a[1], a[2], a[3]);
 #pragma unroll
                 for (int c = 0; c < NT; c++)
 #pragma unroll
                     for (int k = 0; k < 3; k++) mma_bf16(o[i][c], a, b0[c][k], b1[c][k]);
-                if (++ct == col_tiles) ct = 0, g++;
+                if (!ONE && ++ct == col_tiles) ct = 0, g++;
             }
         }
-        if (p.stages == 1) {  // (a ring of one: its next keys come in when everyone is done with these)
-            __syncthreads();
-            if (issued < n_st) issue(issued), issued++;
+        meet();  // the stage and the weights are done with
+        if (st + p.stages < n_st) issue(st + p.stages, s);
+        s += TEAMS;
+        if (s >= p.stages) s -= p.stages, phase ^= 1;
+    }
+    if (bad && lane == 0 && warp == 0) atomicOr(p.status + 2, 1);
+    if (TEAMS == 2) {  // the second team's sums, a warp's beside those of the first team's warp that has the same tiles
+        float4 *const sums = (float4 *)ring + warp * (UNITS * NT * 32) + lane;
+        __syncthreads();  // (the ring is done with)
+        if (team == 1) {
+#pragma unroll
+            for (int i = 0; i < UNITS; i++)
+#pragma unroll
+                for (int c = 0; c < NT; c++) sums[(i * NT + c) * 32] = make_float4(o[i][c][0], o[i][c][1], o[i][c][2], o[i][c][3]);
+        }
+        __syncthreads();
+        if (team == 1) return;
+#pragma unroll
+        for (int i = 0; i < UNITS; i++) {
+#pragma unroll
+            for (int c = 0; c < NT; c++) {
+                const float4 v = sums[(i * NT + c) * 32];
+                o[i][c][0] += v.x, o[i][c][1] += v.y, o[i][c][2] += v.z, o[i][c][3] += v.w;
+            }
         }
     }
     float *dst = p.parts + ((long long)t * p.n_parts + part) * H * VD;
@@ -312,7 +360,7 @@ static int sd_plan(int H, int G, int D, int VD, int &kp, int &stages) {
     return 0;
 }
 
-// The parts a row of a step of n_tokens rows is cut into (what the caller's scratch memory is sized by); 0: these sizes
+// The parts a row of a step of n_tokens rows is cut into, so that the step is about a CTA an SM (what the caller's scratch memory is sized by); 0: these sizes
 // are not taken.
 extern "C" int abk_attention_sigmoid_decode_parts(int n_tokens, int n_heads, int n_kv_heads, int head_dim, int v_dim, int max_keys) {
     if (n_heads < 1 || n_kv_heads < 1 || n_heads % n_kv_heads || head_dim % 8 || v_dim % 8 || head_dim < 8 || v_dim < 8) return 0;
@@ -321,9 +369,7 @@ extern "C" int abk_attention_sigmoid_decode_parts(int n_tokens, int n_heads, int
     if (units * nt > 32) return 0;
     int kp, stages;
     if (!sd_plan(n_heads, n_kv_heads, head_dim, v_dim, kp, stages)) return 0;
-    const int smem = SigmoidDecodeSmem(n_heads, n_kv_heads, head_dim, v_dim, kp, stages).total;
-    const int per_sm = smem <= 112 * 1024 ? 2 : 1;
-    int parts = per_sm * abk_sm_count() / n_tokens, most = (max_keys + 2 * kp - 1) / (2 * kp);
+    int parts = abk_sm_count() / n_tokens, most = (max_keys + 2 * kp - 1) / (2 * kp);
     if (parts > most) parts = most;
     return parts < 1 ? 1 : parts;
 }
@@ -358,19 +404,18 @@ extern "C" int abk_attention_sigmoid_decode(const void *q, long long q_row, void
     const int units = (n_kv_heads * ((v_dim + 15) / 16) + SD_WARPS - 1) / SD_WARPS, nt = n_heads / n_kv_heads > 8 ? 2 : 1;
     const dim3 grid(n_parts, n_tokens);
     cudaStream_t s = (cudaStream_t)stream;
-#define SD_LAUNCH(UNITS, NT)                                                                                              \
-    do {                                                                                                                  \
-        cudaError_t e = abk_allow_shared_memory((const void *)attention_sigmoid_decode_kernel<UNITS, NT>, smem);          \
-        if (e != cudaSuccess) return (int)e;                                                                              \
-        abk_launch(attention_sigmoid_decode_kernel<UNITS, NT>, grid, dim3(SD_THREADS), (size_t)smem, s, mk, mv, p);       \
+#define SD_LAUNCH(UNITS, NT, ONE, TEAMS)                                                                                             \
+    do {                                                                                                                             \
+        cudaError_t e = abk_allow_shared_memory((const void *)attention_sigmoid_decode_kernel<UNITS, NT, ONE, TEAMS>, smem);         \
+        if (e != cudaSuccess) return (int)e;                                                                                         \
+        abk_launch(attention_sigmoid_decode_kernel<UNITS, NT, ONE, TEAMS>, grid, dim3(SD_TEAM_THREADS * TEAMS), (size_t)smem, s, mk, mv, p); \
     } while (0)
-    if (nt == 2) {
-        if (units <= 4) SD_LAUNCH(4, 2);
-        else SD_LAUNCH(16, 2);
-    } else if (units <= 4) SD_LAUNCH(4, 1);
-    else if (units <= 8) SD_LAUNCH(8, 1);
-    else if (units <= 16) SD_LAUNCH(16, 1);
-    else SD_LAUNCH(32, 1);
+    const bool two = p.stages >= 2;  // (a ring of one stage is read by one team)
+    if (nt == 2) SD_LAUNCH(16, 2, false, 1);
+    else if (two && n_kv_heads == 8 && v_dim > 112 && v_dim <= 128) SD_LAUNCH(8, 1, true, 2);
+    else if (two && units <= 8) SD_LAUNCH(8, 1, false, 2);
+    else if (two && units <= 16) SD_LAUNCH(16, 1, false, 2);
+    else SD_LAUNCH(32, 1, false, 1);
 #undef SD_LAUNCH
     rc = ABK_LAUNCH_RESULT();
     if (rc) return rc;
