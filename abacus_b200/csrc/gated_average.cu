@@ -7,9 +7,9 @@
 //   step   one token a sequence: a thread a channel (or a pair, or four).
 //   scan   prompts: a step of the recurrence is the map S -> a S + b with a = 1 - z, b = z c, and maps compose, so a
 //          sequence is cut into runs that are all walked at once. A cluster of CTAs has one sequence and 32 channels (64 as
-//          pairs); each of its warps has a run of 16 tokens (the gates and candidates of which it keeps in registers)
-//          and makes the run's own map; the maps meet through shared memory, and between the CTAs through distributed
-//          shared memory; then every warp walks its run again from the state it now knows, for the outputs. Longer
+//          pairs); each of its warps has a run of 8 tokens (the gates and candidates of which it keeps in registers)
+//          and makes the run's own map; the maps meet in shared memory, a thread a channel, every CTA leaving its own map with
+//          all others (distributed shared memory); then every warp walks its run again from the state it now knows, for the outputs. Longer
 //          sequences go round in turns, the state carried.
 #define ABK_DEFINE_ERROR
 #include "common.cuh"
@@ -71,6 +71,22 @@ template <int VEC> __device__ __forceinline__ void ga_store(__nv_bfloat16 *p, co
     }
 }
 
+// VEC elements as they lie in memory: loads that are asked for early keep what they bring in this form, so that nothing waits
+// for them before they are needed.
+template <typename T, int VEC> struct GaRaw;
+template <> struct GaRaw<__nv_bfloat16, 2> { uint32_t v; };
+template <> struct GaRaw<__nv_bfloat16, 1> { unsigned short v; };
+template <> struct GaRaw<float, 2> { float2 v; };
+template <> struct GaRaw<float, 1> { float v; };
+template <typename T, int VEC> __device__ __forceinline__ GaRaw<T, VEC> ga_fetch(const T *p) { return *(const GaRaw<T, VEC> *)p; }
+__device__ __forceinline__ void ga_open(const GaRaw<__nv_bfloat16, 2> &r, float *f) {
+    const float2 v = __bfloat1622float2(*(const __nv_bfloat162 *)&r.v);
+    f[0] = v.x, f[1] = v.y;
+}
+__device__ __forceinline__ void ga_open(const GaRaw<__nv_bfloat16, 1> &r, float *f) { f[0] = __bfloat162float(*(const __nv_bfloat16 *)&r.v); }
+__device__ __forceinline__ void ga_open(const GaRaw<float, 2> &r, float *f) { f[0] = r.v.x, f[1] = r.v.y; }
+__device__ __forceinline__ void ga_open(const GaRaw<float, 1> &r, float *f) { f[0] = r.v; }
+
 // ---------------------------------------------------------------- one token a sequence
 template <typename T, int VEC> __global__ void __launch_bounds__(128) gated_average_step_kernel(GatedAverage p) {
     const int c = (blockIdx.x * 128 + threadIdx.x) * VEC, t = blockIdx.y;
@@ -102,13 +118,13 @@ template <typename T, int VEC> __global__ void __launch_bounds__(128) gated_aver
 }
 
 // ---------------------------------------------------------------- prompts
-#define GA_WARPS 8
-#define GA_RUN 16  // tokens of a warp's run
+#define GA_WARPS 16
+#define GA_RUN 8     // tokens of a warp's run
 
 template <typename T, int VEC> __global__ void __launch_bounds__(32 * GA_WARPS) gated_average_scan_kernel(GatedAverage p) {
     constexpr int CH = 32 * VEC;
-    __shared__ float run_a[GA_WARPS][CH], run_b[GA_WARPS][CH];
-    __shared__ float cta_a[2][CH], cta_b[2][CH];  // this CTA's map, by the turn's parity: the other CTAs read it
+    __shared__ float2 runs[GA_WARPS][CH];    // the runs' maps (a, b); then, in x, the states before the runs
+    __shared__ float2 ctas[2][8][CH];        // the CTAs' maps, by the turn's parity: every CTA leaves its own with all of them
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int ranks = (int)tc::cluster_size(), rank = (int)tc::cluster_rank();
     const int c = (blockIdx.x / ranks) * CH + lane * VEC, seq = blockIdx.y;
@@ -120,90 +136,95 @@ template <typename T, int VEC> __global__ void __launch_bounds__(32 * GA_WARPS) 
     pdl_wait();
     const int row0 = p.seq_start[seq], n = p.seq_start[seq + 1] - row0;
     if (n <= 0) return;  // (the whole cluster: a sequence of the step's padding)
-    float *slot = p.state + (long long)p.seq_slot[seq] * p.width + c;
-    float carry[VEC];  // the state before the turn, the same in every warp of the cluster
-#pragma unroll
-    for (int i = 0; i < VEC; i++) carry[i] = 0.0f;
-    if (real) ga_load<VEC>(slot, carry);
+    // the first CH threads each keep a channel's state before the turn, the same in every CTA of the cluster
+    const int own = (blockIdx.x / ranks) * CH + (int)threadIdx.x;
+    const bool keeper = threadIdx.x < CH, owns = keeper && own < p.width;
+    float *const slot = p.state + (long long)p.seq_slot[seq] * p.width + own;
+    float held = owns ? *slot : 0.0f;
     const int turn_tokens = ranks * GA_WARPS * GA_RUN;
     int parity = 0;
+    // a run's rows: gates and candidates are asked for a turn ahead, the outputs' gates with the turn before's outputs
+    // (loads that hang on no branch fly together: a row beyond the run repeats its last)
+    GaRaw<T, VEC> rz[GA_RUN], ru[GA_RUN], rg[GA_RUN];
+    const T *const all = (const T *)p.proj + (long long)row0 * p.ld + c;
+    auto run_of = [&](int t0, int &first) {
+        first = t0 + (rank * GA_WARPS + warp) * GA_RUN;
+        return min(GA_RUN, n - first);  // (not above zero: no run)
+    };
+    auto fetch = [&](int t0) {
+        int first;
+        const int cnt = run_of(t0, first);
+        if (!real || cnt <= 0) return;
+#pragma unroll
+        for (int k = 0; k < GA_RUN; k++) {
+            const T *r = all + (long long)(first + min(k, cnt - 1)) * p.ld;
+            rz[k] = ga_fetch<T, VEC>(r + p.z_at), ru[k] = ga_fetch<T, VEC>(r + p.u_at);
+        }
+    };
+    auto fetch_gates = [&](int t0) {
+        int first;
+        const int cnt = run_of(t0, first);
+        if (!real || cnt <= 0) return;
+#pragma unroll
+        for (int k = 0; k < GA_RUN; k++) rg[k] = ga_fetch<T, VEC>(all + (long long)(first + min(k, cnt - 1)) * p.ld + p.g_at);
+    };
+    fetch(0), fetch_gates(0);
+    if (ranks > 1) tc::cluster_sync();  // every CTA has started: maps may be left with it
     for (int t0 = 0; t0 < n; t0 += turn_tokens, parity ^= 1) {
-        const int first = t0 + (rank * GA_WARPS + warp) * GA_RUN, cnt = min(GA_RUN, n - first);  // (cnt may be negative: no run)
-        const T *rows = (const T *)p.proj + (long long)(row0 + first) * p.ld + c;
+        int first;
+        const int cnt = run_of(t0, first);
         float a[GA_RUN][VEC], b[GA_RUN][VEC], A[VEC], B[VEC];
 #pragma unroll
         for (int i = 0; i < VEC; i++) A[i] = 1.0f, B[i] = 0.0f;
         if (real && cnt > 0) {
 #pragma unroll
             for (int k = 0; k < GA_RUN; k++) {
-                const T *r = rows + (long long)min(k, cnt - 1) * p.ld;  // (loads that hang on no branch fly together)
-                ga_load<VEC>(r + p.z_at, a[k]), ga_load<VEC>(r + p.u_at, b[k]);
-            }
-#pragma unroll
-            for (int k = 0; k < GA_RUN; k++) {
+                float z[VEC], u[VEC];
+                ga_open(rz[k], z), ga_open(ru[k], u);
 #pragma unroll
                 for (int i = 0; i < VEC; i++) {
-                    float ka, kb;
-                    ga_map<T>(a[k][i] + bz[i], b[k][i] + bu[i], ka, kb);
-                    a[k][i] = ka, b[k][i] = kb;
-                    if (k < cnt) A[i] *= ka, B[i] = fmaf(ka, B[i], kb);
+                    ga_map<T>(z[i] + bz[i], u[i] + bu[i], a[k][i], b[k][i]);
+                    if (k < cnt) A[i] *= a[k][i], B[i] = fmaf(a[k][i], B[i], b[k][i]);
                 }
             }
         }
-        __syncthreads();  // the turn before has read the runs' maps
+        if (t0 + turn_tokens < n) fetch(t0 + turn_tokens);
+        __syncthreads();  // the turn before has read the states before its runs
 #pragma unroll
-        for (int i = 0; i < VEC; i++) run_a[warp][lane * VEC + i] = A[i], run_b[warp][lane * VEC + i] = B[i];
+        for (int i = 0; i < VEC; i++) runs[warp][lane * VEC + i] = make_float2(A[i], B[i]);
         __syncthreads();
-        float s[VEC];
-        if (ranks > 1) {
-            if (threadIdx.x < CH) {
-                float ca = 1.0f, cb = 0.0f;
-#pragma unroll
-                for (int w = 0; w < GA_WARPS; w++) {
-                    ca *= run_a[w][threadIdx.x];
-                    cb = fmaf(run_a[w][threadIdx.x], cb, run_b[w][threadIdx.x]);
-                }
-                cta_a[parity][threadIdx.x] = ca, cta_b[parity][threadIdx.x] = cb;
-            }
-            tc::cluster_sync();
-            // every CTA's map: all loads in flight, then the states before this CTA and after the last
-#pragma unroll
-            for (int i = 0; i < VEC; i++) {
-                const uint32_t at_a = (uint32_t)__cvta_generic_to_shared(&cta_a[parity][lane * VEC + i]);
-                const uint32_t at_b = (uint32_t)__cvta_generic_to_shared(&cta_b[parity][lane * VEC + i]);
-                float ra[8], rb[8];
-#pragma unroll
-                for (int k = 0; k < 8; k++) {
-                    ra[k] = 1.0f, rb[k] = 0.0f;
-                    if (k < ranks) {
-                        asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(ra[k]) : "r"(tc::peer_smem(at_a, k)));
-                        asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(rb[k]) : "r"(tc::peer_smem(at_b, k)));
-                    }
-                }
-                float v = carry[i];
-                s[i] = v;
-#pragma unroll
-                for (int k = 0; k < 8; k++) {
-                    if (k == rank) s[i] = v;
-                    if (k < ranks) v = fmaf(ra[k], v, rb[k]);
-                }
-                carry[i] = v;
-            }
-        } else {
-#pragma unroll
-            for (int i = 0; i < VEC; i++) s[i] = carry[i];
-        }
-        // from the CTA's start through the runs before this warp's (and, alone in the cluster, on to the turn's end)
-#pragma unroll
-        for (int i = 0; i < VEC; i++) {
-            float v = s[i];
+        float2 map[GA_WARPS];
+        if (keeper) {
+            float2 all = make_float2(1.0f, 0.0f);
 #pragma unroll
             for (int w = 0; w < GA_WARPS; w++) {
-                if (w == warp) s[i] = v;
-                v = fmaf(run_a[w][lane * VEC + i], v, run_b[w][lane * VEC + i]);
+                map[w] = runs[w][threadIdx.x];
+                all = make_float2(map[w].x * all.x, fmaf(map[w].x, all.y, map[w].y));
             }
-            if (ranks == 1) carry[i] = v;
+            const uint32_t at = (uint32_t)__cvta_generic_to_shared(&ctas[parity][rank][threadIdx.x]);
+            if (ranks == 1) ctas[parity][0][threadIdx.x] = all;
+            else for (int k = 0; k < ranks; k++)
+                asm volatile("st.shared::cluster.v2.f32 [%0], {%1, %2};" ::"r"(tc::peer_smem(at, k)), "f"(all.x), "f"(all.y) : "memory");
         }
+        if (ranks > 1) tc::cluster_sync();
+        if (keeper) {  // through the CTAs before this one and through its runs; and on to the turn's end
+            float v = held, mine = held;
+            for (int k = 0; k < ranks; k++) {
+                if (k == rank) mine = v;
+                const float2 m = ctas[parity][k][threadIdx.x];
+                v = fmaf(m.x, v, m.y);
+            }
+            held = v;
+#pragma unroll
+            for (int w = 0; w < GA_WARPS; w++) {
+                runs[w][threadIdx.x].x = mine;
+                mine = fmaf(map[w].x, mine, map[w].y);
+            }
+        }
+        __syncthreads();
+        float s[VEC];
+#pragma unroll
+        for (int i = 0; i < VEC; i++) s[i] = runs[warp][lane * VEC + i].x;
         if (!real && c < p.padded) {
             float zero[VEC];
 #pragma unroll
@@ -212,23 +233,23 @@ template <typename T, int VEC> __global__ void __launch_bounds__(32 * GA_WARPS) 
         }
         if (real && cnt > 0) {
             T *out = (T *)p.out + (long long)(row0 + first) * p.ldo + c;
-            float g[GA_RUN][VEC];
-#pragma unroll
-            for (int k = 0; k < GA_RUN; k++) ga_load<VEC>(rows + (long long)min(k, cnt - 1) * p.ld + p.g_at, g[k]);
 #pragma unroll
             for (int k = 0; k < GA_RUN; k++) {
                 if (k >= cnt) break;
+                float g[VEC];
+                ga_open(rg[k], g);
 #pragma unroll
                 for (int i = 0; i < VEC; i++) {
                     s[i] = fmaf(a[k][i], s[i], b[k][i]);
-                    g[k][i] = s[i] * ga_silu<T>(g[k][i]);
+                    g[i] = s[i] * ga_silu<T>(g[i]);
                 }
-                ga_store<VEC>(out + (long long)k * p.ldo, g[k]);
+                ga_store<VEC>(out + (long long)k * p.ldo, g);
             }
         }
+        if (t0 + turn_tokens < n) fetch_gates(t0 + turn_tokens);
     }
-    if (rank == 0 && warp == 0 && real) ga_store<VEC>(slot, carry);
-    if (ranks > 1) tc::cluster_sync();  // nobody leaves while its map may still be read
+    if (rank == 0 && owns) *slot = held;
+    if (ranks > 1) tc::cluster_sync();  // nobody leaves while a map may still be left with it
 }
 
 // padded: columns of out from width on up to there are written with zeros (a product with padded rows reads them).
