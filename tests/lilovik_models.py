@@ -36,7 +36,7 @@ CONFIGS = {
           "layers": [attention_layer(3, 3, 10, 7, 0.5, None, (0.5, 7)), average_layer(13), attention_layer(1, 1, 20, 33, 0.3, 9.0, None, ff=11),
                      attention_layer(4, 2, 12, 12, 0.45, 30.0, (1.0, 1), ff=9)]},
     "C": {"architecture": "Lilovik", "vocab": 77, "width": 80, "norm": {"eps": 1e-5}, "logit_scale": 2.0,
-          "layers": [attention_layer(20, 1, 16, 16, 0.4, 15.0, (0.3, 33), ff=64), attention_layer(24, 8, 64, 24, 0.2, 40.0, (0.6, 64)),
+          "layers": [attention_layer(20, 1, 16, 16, 0.4, 15.0, (0.3, 33), ff=64), attention_layer(24, 8, 64, 24, 0.2, 40.0, (0.6, 60)),
                      average_layer(200, ff=48)]},
     "D": {"architecture": "Lilovik", "vocab": 61, "width": 72, "norm": {"eps": 1e-5}, "logit_scale": 0.125,
           "layers": [average_layer(72), average_layer(24, ff=40), attention_layer(8, 8, 72, 40, 0.15, 30.0, (0.5, 20), ff=256)]},

@@ -43,7 +43,7 @@ def _attention_run(p, d, m, dtype):
 @pytest.mark.parametrize("dtype", BOTH)
 @pytest.mark.parametrize("H,G,K,V,cap,temp", [
     (6, 2, 16, 24, 12.0, (0.7, 9)), (3, 3, 10, 7, None, (0.5, 7)), (1, 1, 20, 33, 9.0, None), (20, 1, 16, 16, 15.0, (0.3, 33)),
-    (24, 8, 64, 24, 40.0, (0.6, 64)), (8, 8, 72, 40, 30.0, (0.5, 20)), (16, 8, 128, 128, 30.0, (0.5, 64)), (32, 8, 64, 64, None, None),
+    (24, 8, 64, 24, 40.0, (0.6, 60)), (8, 8, 72, 40, 30.0, (0.5, 20)), (16, 8, 128, 128, 28.0, (0.45, 70)), (32, 8, 64, 64, None, None),
     (4, 4, 96, 96, 30.0, (1.0, 1)), (2, 1, 256, 128, 20.0, (0.2, 10)), (5, 5, 8, 136, 20.0, (0.4, 50)), (15, 5, 24, 8, 7.0, (0.4, 16)),
 ])
 def test_attention_every_way(dtype, H, G, K, V, cap, temp):
@@ -114,7 +114,7 @@ class Rows:
         return dict(n_heads=H, n_kv_heads=G, head_dim=K, vd=V, row=self.row, scale=self.scale, softcap=self.cap, **self.dev)
 
 
-@pytest.mark.parametrize("H,G,K,V,cap", [(16, 8, 128, 128, 30.0), (8, 8, 96, 96, 25.0), (6, 3, 40, 24, None), (4, 1, 64, 128, 5.0), (32, 4, 64, 32, 30.0),
+@pytest.mark.parametrize("H,G,K,V,cap", [(16, 8, 128, 128, 30.0), (8, 8, 80, 96, 25.0), (6, 3, 40, 24, None), (4, 1, 64, 128, 5.0), (32, 4, 64, 32, 30.0),
                                          (1, 1, 8, 8, None), (17, 17, 16, 16, 10.0), (13, 13, 24, 40, 20.0), (32, 8, 128, 128, 30.0), (20, 5, 104, 56, None)])
 def test_the_prompt_kernel_against_float64(H, G, K, V, cap):
     """Unequal sequences, the keys of a query tile on one CTA and dealt to clusters of 2, 4 and 8; and the general kernel on
@@ -137,7 +137,7 @@ def test_the_prompt_kernel_against_float64(H, G, K, V, cap):
     rows.check(out, want, "general kernel")
 
 
-@pytest.mark.parametrize("H,G,K,V,cap", [(16, 8, 128, 128, 30.0), (8, 8, 96, 96, 25.0), (6, 3, 40, 24, None), (16, 1, 64, 128, 5.0), (32, 4, 64, 32, 30.0),
+@pytest.mark.parametrize("H,G,K,V,cap", [(16, 8, 128, 128, 30.0), (8, 8, 80, 96, 25.0), (6, 3, 40, 24, None), (16, 1, 64, 128, 5.0), (32, 4, 64, 32, 30.0),
                                          (1, 1, 8, 8, None), (17, 17, 16, 16, 10.0), (13, 13, 24, 40, 20.0), (32, 8, 128, 128, 30.0),
                                          (16, 16, 128, 128, 20.0), (20, 2, 72, 136, 30.0), (28, 28, 128, 128, 25.0)])
 def test_the_decode_kernel_against_float64(H, G, K, V, cap):
