@@ -18,10 +18,13 @@ class NormSpec:
     """RMSNorm as src/model.c:164-169: w * (x / sqrt(mean(x^2) + eps)).
 
     one_plus: the checkpoint stores the weight around zero and the norm multiplies by 1 + w.
+    gain: a learned factor per element behind the norm (slot "gain", [size]). mult: a constant factor behind it.
     """
     size: int
     eps: float
     one_plus: bool = False
+    gain: bool = False
+    mult: float = 1.0
     kind: str = "rmsnorm"
 
 
@@ -41,9 +44,12 @@ class RotarySpec:
     # fast, slow), the scaling known as YaRN: with where(t) = rotary_dim * ln(original / (2 pi t)) / (2 ln theta),
     # lo = max(floor(where(fast)), 0), hi = min(ceil(where(slow)), rotary_dim - 1) and
     # ramp_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1), pair i turns at f_i / factor * ramp_i + f_i * (1 - ramp_i),
-    # and cosines and sines are multiplied by 0.1 ln(factor) + 1.
+    # and cosines and sines are multiplied by 0.1 ln(factor) + 1. bands (factor, original, low, high), the scaling of
+    # Llama 3.1: a pair whose wavelength 2 pi / f is shorter than original / high keeps its f, one longer than original / low
+    # turns at f / factor, and in between s = (original f / (2 pi) - low) / (high - low) blends (1 - s) f / factor + s f.
     linear_factor: float = 1.0
     blend: Optional[tuple] = None
+    bands: Optional[tuple] = None
 
 
 @dataclass(frozen=True)
@@ -71,6 +77,11 @@ class AttentionSpec:
     off the score of key j seen from i (after the cap); shift, a learned number per head (slot "shift", [heads]) added to
     the score; mix, the heads' weights mixed before they meet the values, w_h <- sum_g M[h, g] w_g (slot "mix",
     [heads, heads]), head h's mixed weights applied to the values of its own kv head.
+    diff c (softmax weights, float32): differential attention. Every query head and every key head has two maps of head_dim,
+    laid out head by head as [map 1 | map 2] (q has heads * 2 * head_dim rows, k kv_heads * 2 * head_dim); norm and rotation
+    are each map's own (the norms' weights shared); each map is an attention of its own over the head's values. With
+    lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + c (slots "lq1", "lk1", "lq2", "lk2", [head_dim]), o = a1 - lambda a2, and the
+    head's output is (1 - c) o / sqrt(mean(o^2) + diff_eps).
     """
     hidden: int
     n_heads: int
@@ -96,6 +107,8 @@ class AttentionSpec:
     slopes: Optional[tuple] = None
     shift: bool = False
     mix: bool = False
+    diff: Optional[float] = None
+    diff_eps: float = 1e-5
     kind: str = "attention"
 
 
@@ -187,6 +200,7 @@ class LatentAttentionSpec:
     down-projection of its own and reads the cache of the schedule entry it names as its source.
     q_rank Q: the queries pass a latent of their own, q = Wuq norm(Wdq x; w) (slots "wdq" [Q, hidden], "q_norm" [Q],
     "wq" [heads * (head_dim + rot_dim), Q]). head_gate: head h's output is multiplied by sigmoid(g_h . x) (slot "wg").
+    window W: the last W keys are seen, the token's own included (the cache keeps no others).
     """
     hidden: int
     n_heads: int
@@ -201,6 +215,7 @@ class LatentAttentionSpec:
     shares_latents: bool = False
     q_rank: Optional[int] = None
     head_gate: bool = False
+    window: Optional[int] = None
     kind: str = "latent_attention"
 
 
@@ -257,9 +272,11 @@ class GatedAverageSpec:
 
 @dataclass(frozen=True)
 class ExpertSpec:
-    """A small feed-forward: down(act(up(x))), or, with activation "silu_gated", down(silu(gate(x)) * up(x))."""
+    """A small feed-forward: down(act(up(x))), or, with activation "silu_gated", down(silu(gate(x)) * up(x)), or, with
+    "clamped_gated", down(g sigmoid(1.702 g) (u + 1)), g = min(gate(x), limit), u = clamp(up(x), -limit, limit)."""
     inter: int
     activation: str = "relu_squared"
+    limit: float = 0.0
 
 
 @dataclass(frozen=True)
@@ -274,7 +291,8 @@ class RoutedMLPSpec:
     score "table": there is no router; row `token id` of an integer table (slot "table", [vocab, top]) names the token's
     experts, each with weight 1 / top.
     weight_on "input": the output is sum_e expert_e(w_e x); "output": sum_e w_e expert_e(x). shared (an ExpertSpec or
-    None) runs for every token and is added.
+    None) runs for every token and is added. router_bias: a learned number per output is added to z (slot "router_bias").
+    shared_gate: the shared expert's output is multiplied by sigmoid(s . x) (slot "shared_gate", [1, hidden]).
     """
     hidden: int
     experts: int
@@ -287,16 +305,29 @@ class RoutedMLPSpec:
     weight_scale: float = 1.0
     identity: int = 0
     vocab: int = 0  # rows of the table (score "table")
+    router_bias: bool = False
+    shared_gate: bool = False
     kind: str = "routed_mlp"
 
 
 @dataclass(frozen=True)
 class GatedMLPSpec:
-    """down(act(gate(x)) * up(x)) as src/model.c:274-282, 307-309; act "silu" or "relu"."""
+    """down(act(gate(x)) * up(x)) as src/model.c:274-282, 307-309; act "silu" or "relu", or "clamped_silu":
+    down(g sigmoid(1.702 g) (u + 1)), g = min(gate(x), limit), u = clamp(up(x), -limit, limit)."""
     hidden: int
     inter: int
     activation: str = "silu"
+    limit: float = 0.0
     kind: str = "gated_mlp"
+
+
+@dataclass(frozen=True)
+class PlainMLPSpec:
+    """down(act(up(x))); act "relu_squared"."""
+    hidden: int
+    inter: int
+    activation: str = "relu_squared"
+    kind: str = "plain_mlp"
 
 
 @dataclass(frozen=True)
@@ -327,6 +358,17 @@ class SandwichBlockSpec:
     ffn: object = None
     ffn_post_norm: object = None
     kind: str = "sandwich_norm"
+
+
+@dataclass(frozen=True)
+class PostNormBlockSpec:
+    """One layer with a norm on each branch's output only, the branches reading the stream itself:
+    x += mixer_post_norm(mixer(x)), then x += ffn_post_norm(ffn(x)). ffn None: the mixer's branch alone."""
+    mixer: object
+    mixer_post_norm: object
+    ffn: object = None
+    ffn_post_norm: object = None
+    kind: str = "post_norm"
 
 
 @dataclass(frozen=True)
@@ -375,6 +417,12 @@ class SinusoidEmbeddingSpec:
     sin(p * base^(-2i / hidden)), element 2i + 1 the cosine of the same angle. The logits are multiplied by logit_scale."""
     base: float = 10000.0
     logit_scale: float = 1.0
+
+
+@dataclass(frozen=True)
+class ScaledEmbeddingSpec:
+    """The frame "scaled": x = table[token] * scale (the output matrix, where it is the table, is not scaled)."""
+    scale: float = 1.0
 
 
 @dataclass(frozen=True)

@@ -7,7 +7,9 @@
 // seen from i when j <= i and (i - j < window or j < keep_first)); a sink, a learned score per head that
 // joins the softmax's denominator once, unscaled, without a key or a value; chunks (key j is seen from i only when
 // both lie in the same run of `chunk` positions, counted from the sequence's first); capped scores
-// (s <- cap * tanh(s / cap), after the scale).
+// (s <- cap * tanh(s / cap), after the scale); query heads in runs of `maps` that read the same kv head, each its own slice
+// of the key row, with one value (differential attention: each map is an attention of its own, and differential_heads
+// makes one head of the two, csrc/differential.cuh).
 // It serves prefill and decode alike and is the kernel every size falls back to; the float32
 // path of the model uses nothing else for attention.
 //
@@ -17,6 +19,7 @@
 // visible key, never at a batch-dependent place.
 #define ABK_DEFINE_ERROR
 #include "common.cuh"
+#include "differential.cuh"
 
 #define ATT_THREADS 128
 #define ATT_MAX_HEAD_DIM 640
@@ -25,8 +28,9 @@
 struct AttnGeneric {
     const void *q;      // row t, head h at q + (t * q_row + h * head_dim)
     long long q_row;    // elements between rows of q
-    void *out;          // [tokens, n_heads * head_dim]
+    void *out;          // [tokens, n_heads * v_dim]
     int n_heads, n_kv_heads, head_dim;
+    int maps;           // a key row holds maps * head_dim elements; query head h reads slice h % maps
     int v_dim;          // size of a value head (out is [tokens, n_heads * v_dim])
     float scale;
     int window;         // 0: all earlier keys
@@ -78,7 +82,7 @@ template <> __device__ __forceinline__ float dot_row<__nv_bfloat16>(const float 
 }
 
 // ROUNDED_P: the probabilities are a stored tensor in the model's type (bfloat16) for the second product.
-template <typename T, bool ROUNDED_P>
+template <typename T, bool ROUNDED_P, typename TO = T>
 __global__ void __launch_bounds__(ATT_THREADS) attention_generic_kernel(AttnGeneric p) {
     __shared__ float q_s[ATT_MAX_HEAD_DIM];
     __shared__ float p_s[ATT_THREADS];
@@ -86,13 +90,14 @@ __global__ void __launch_bounds__(ATT_THREADS) attention_generic_kernel(AttnGene
     __shared__ float scratch[33];
     int t = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, hd = p.head_dim, vd = p.v_dim;
     int seq = p.token_seq[t];
-    T *out = (T *)p.out + ((long long)t * p.n_heads + h) * vd;
+    TO *out = (TO *)p.out + ((long long)t * p.n_heads + h) * vd;
     if (seq < 0) {  // padding
-        for (int d = tid; d < vd; d += ATT_THREADS) out[d] = from_float<T>(0.0f);
+        for (int d = tid; d < vd; d += ATT_THREADS) out[d] = from_float<TO>(0.0f);
         return;
     }
     int pos = p.token_pos[t], slot = p.seq_slot[seq];
     int kvh = h / (p.n_heads / p.n_kv_heads);
+    const int kd = p.maps * hd, slice = h % p.maps * hd;  // a key row; where this head's part of it starts
     int lo = p.window > 0 && pos - p.window + 1 > 0 ? pos - p.window + 1 : 0;
     if (p.chunk > 0 && pos / p.chunk * p.chunk > lo) lo = pos / p.chunk * p.chunk;
     // the sequence's first keys that the window no longer reaches: positions [0, first_end)
@@ -116,12 +121,12 @@ __global__ void __launch_bounds__(ATT_THREADS) attention_generic_kernel(AttnGene
             long long vo;
             if (p.k_step) {
                 long long row = (long long)p.seq_start[seq] + j - p.seq_pos0[seq];
-                vo = row * p.kv_row + (long long)kvh * (p.values_in_keys ? hd : vd);
-                k = (const T *)p.k_step + row * p.kv_row + (long long)kvh * hd;
+                vo = row * p.kv_row + (long long)kvh * (p.values_in_keys ? kd : vd);
+                k = (const T *)p.k_step + row * p.kv_row + (long long)kvh * kd + slice;
             } else {
                 int page = cache_page(p.cache, slot, j);
-                vo = cache_offset(p.v_cache, page, kvh, p.n_kv_heads, j, p.values_in_keys ? hd : vd);
-                k = (const T *)p.k_pool + cache_offset(p.cache, page, kvh, p.n_kv_heads, j, hd);
+                vo = cache_offset(p.v_cache, page, kvh, p.n_kv_heads, j, p.values_in_keys ? kd : vd);
+                k = (const T *)p.k_pool + cache_offset(p.cache, page, kvh, p.n_kv_heads, j, kd) + slice;
             }
             v_off[tid] = vo;
             s = (p.vector_rows ? dot_row<T>(q_s, k, hd) : dot_row_plain<T>(q_s, k, hd)) * p.scale;
@@ -162,7 +167,7 @@ __global__ void __launch_bounds__(ATT_THREADS) attention_generic_kernel(AttnGene
     }
 #pragma unroll
     for (int u = 0; u < ATT_COLS; u++)
-        if (tid + u * ATT_THREADS < vd) out[tid + u * ATT_THREADS] = from_float<T>(acc[u] / l);
+        if (tid + u * ATT_THREADS < vd) out[tid + u * ATT_THREADS] = from_float<TO>(acc[u] / l);
 }
 
 static int attention_general(int values_in_keys, const void *q, long long q_row, void *out, int dtype, int n_tokens, int n_heads,
@@ -172,7 +177,7 @@ static int attention_general(int values_in_keys, const void *q, long long q_row,
                                      const int *page_table, int table_width, int ring_pages, int tokens_per_page,
                                      const void *k_step, const void *v_step, long long kv_row, int v_dim,
                                      int keep_first, int pinned_pages, const float *sink, int exact_weights,
-                                     void *stream, int chunk = 0, float softcap = 0.0f) {
+                                     void *stream, int chunk = 0, float softcap = 0.0f, int maps = 1, int out_f32 = 0) {
     if (n_tokens <= 0) return 0;
     if (v_dim <= 0) v_dim = head_dim;
     if (chunk < 0 || softcap < 0.0f) ABK_REFUSE("attention: a chunk of %d positions, a score cap of %g", chunk, softcap);
@@ -185,8 +190,11 @@ static int attention_general(int values_in_keys, const void *q, long long q_row,
     if (n_kv_heads < 1 || n_heads % n_kv_heads)
         ABK_REFUSE("attention: %d query heads do not divide into %d kv heads", n_heads, n_kv_heads);
     if (n_heads > 65535) ABK_REFUSE("attention: %d heads are more than a grid takes", n_heads);
+    if (maps < 1 || n_heads / n_kv_heads % maps || (maps > 1 && values_in_keys))
+        ABK_REFUSE("attention: %d query heads to a kv head in runs of %d maps", n_heads / n_kv_heads, maps);
+    if (out_f32 && dtype == ABK_BF16 && !exact_weights) ABK_REFUSE("attention: float32 outputs go with softmax weights in float32");
     AttnGeneric p;
-    p.q = q, p.q_row = q_row, p.out = out, p.n_heads = n_heads, p.n_kv_heads = n_kv_heads, p.head_dim = head_dim;
+    p.q = q, p.q_row = q_row, p.out = out, p.n_heads = n_heads, p.n_kv_heads = n_kv_heads, p.head_dim = head_dim, p.maps = maps;
     p.scale = scale, p.window = window, p.token_seq = token_seq, p.token_pos = token_pos, p.seq_slot = seq_slot;
     p.seq_start = seq_start, p.seq_pos0 = seq_pos0, p.k_pool = k_pool, p.v_pool = v_pool;
     p.cache.page_table = page_table, p.cache.table_width = table_width, p.cache.ring_pages = ring_pages;
@@ -204,6 +212,8 @@ static int attention_general(int values_in_keys, const void *q, long long q_row,
     cudaStream_t s = (cudaStream_t)stream;
     if (dtype == ABK_BF16 && !exact_weights)
         attention_generic_kernel<__nv_bfloat16, true><<<grid, ATT_THREADS, 0, s>>>(p);
+    else if (dtype == ABK_BF16 && out_f32)
+        attention_generic_kernel<__nv_bfloat16, false, float><<<grid, ATT_THREADS, 0, s>>>(p);
     else if (dtype == ABK_BF16)
         attention_generic_kernel<__nv_bfloat16, false><<<grid, ATT_THREADS, 0, s>>>(p);
     else
@@ -246,11 +256,62 @@ extern "C" int abk_attention_values_in_keys(const void *q, long long q_row, void
                                             int n_kv_heads, int head_dim, float scale, const int *token_seq,
                                             const int *token_pos, const int *seq_slot, const int *seq_start,
                                             const int *seq_pos0, const void *k_pool, const int *page_table,
-                                            int table_width, int tokens_per_page, int v_dim, const float *sink,
-                                            int exact_weights, void *stream) {
-    return attention_general(1, q, q_row, out, dtype, n_tokens, n_heads, n_kv_heads, head_dim, scale, 0, token_seq,
-                             token_pos, seq_slot, seq_start, seq_pos0, k_pool, k_pool, page_table, table_width, 0,
-                             tokens_per_page, nullptr, nullptr, 0, v_dim, 0, 0, sink, exact_weights, stream);
+                                            int table_width, int ring_pages, int tokens_per_page, const void *k_step,
+                                            long long kv_row, int v_dim, int window, const float *sink, int exact_weights,
+                                            void *stream) {
+    return attention_general(1, q, q_row, out, dtype, n_tokens, n_heads, n_kv_heads, head_dim, scale, window, token_seq,
+                             token_pos, seq_slot, seq_start, seq_pos0, k_pool, k_pool, page_table, table_width, ring_pages,
+                             tokens_per_page, k_step, k_step, kv_row, v_dim, 0, 0, sink, exact_weights, stream);
+}
+
+// The maps of differential attention over the paged cache: query heads in runs of `maps` read their own slices of a kv
+// head's key row (maps * head_dim elements) and the same value. out float32 [tokens, n_heads * v_dim], n_heads counting
+// every map of every head; abk_differential_heads makes the heads' outputs of it.
+extern "C" int abk_attention_maps(const void *q, long long q_row, float *out, int dtype, int n_tokens, int n_heads, int n_kv_heads,
+                                  int head_dim, int maps, float scale, int window, const int *token_seq, const int *token_pos,
+                                  const int *seq_slot, const int *seq_start, const int *seq_pos0, const void *k_pool,
+                                  const void *v_pool, const int *page_table, int table_width, int ring_pages, int tokens_per_page,
+                                  const void *k_step, const void *v_step, long long kv_row, int v_dim, int keep_first,
+                                  int pinned_pages, const float *sink, int chunk, float softcap, void *stream) {
+    return attention_general(0, q, q_row, out, dtype, n_tokens, n_heads, n_kv_heads, head_dim, scale, window, token_seq,
+                             token_pos, seq_slot, seq_start, seq_pos0, k_pool, v_pool, page_table, table_width, ring_pages,
+                             tokens_per_page, k_step, v_step, kv_row, v_dim, keep_first, pinned_pages, sink, 1, stream, chunk,
+                             softcap, maps, 1);
+}
+
+// out[t, h] = keep * o / sqrt(mean(o^2) + eps), o = maps[t, 2 h] - lambda * maps[t, 2 h + 1]: a CTA a head of a token.
+template <typename T>
+__global__ void __launch_bounds__(ATT_THREADS) differential_heads_kernel(const float *maps, T *out, int n_heads, int vd, DifferentialHead d) {
+    __shared__ float scratch[33];
+    const long long at = (long long)blockIdx.x * n_heads + blockIdx.y;
+    pdl_wait();
+    const float *a = maps + 2 * at * vd, *b = a + vd;
+    float o[ATT_COLS], ss = 0.0f;
+#pragma unroll
+    for (int u = 0; u < ATT_COLS; u++) {
+        const int c = threadIdx.x + u * ATT_THREADS;
+        o[u] = c < vd ? differential_value(d, a[c], b[c]) : 0.0f;
+        ss = fmaf(o[u], o[u], ss);
+    }
+    const float scale = differential_scale(d, block_sum(ss, scratch), vd);
+#pragma unroll
+    for (int u = 0; u < ATT_COLS; u++) {
+        const int c = threadIdx.x + u * ATT_THREADS;
+        if (c < vd) out[at * vd + c] = from_float<T>(o[u] * scale);
+    }
+}
+
+extern "C" int abk_differential_heads(const float *maps, void *out, int dtype, int n_tokens, int n_heads, int v_dim, float lambda,
+                                      float eps, float keep, void *stream) {
+    if (n_tokens <= 0) return 0;
+    if (v_dim < 1 || v_dim > ATT_MAX_HEAD_DIM || n_heads > 65535) ABK_REFUSE("differential_heads: %d heads of %d", n_heads, v_dim);
+    const DifferentialHead d = {lambda, eps, keep};
+    cudaStream_t s = (cudaStream_t)stream;
+    if (dtype == ABK_BF16)
+        abk_launch(differential_heads_kernel<__nv_bfloat16>, dim3(n_tokens, n_heads), dim3(ATT_THREADS), 0, s, maps, (__nv_bfloat16 *)out, n_heads, v_dim, d);
+    else
+        abk_launch(differential_heads_kernel<float>, dim3(n_tokens, n_heads), dim3(ATT_THREADS), 0, s, maps, (float *)out, n_heads, v_dim, d);
+    return ABK_LAUNCH_RESULT();
 }
 
 // The same without the options: values as large as keys, no kept first keys, no sink, probabilities in the model's type.

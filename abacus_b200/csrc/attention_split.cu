@@ -9,10 +9,14 @@
 //   p_j = exp(z_j - M) / (exp(sink - M) + sum_j exp(z_j - M)),  z_j = scale * (q . k_j),  out = sum_j p_j v_j
 //   (with a cap c of the scores, z_j = c tanh(scale * (q . k_j) / c))
 //
+// Differential attention (maps 2): query heads in runs of two read the two halves of a key row, each a map of its own over
+// the same values; the fold makes one head of the two (csrc/differential.cuh), so both maps' sums stay float32.
+//
 // A row's visible keys are numbered: first the kept first keys the window no longer reaches, then the window's
 // (or all). Part t has numbers [128 t, 128 t + 128). All arithmetic is float32.
 #define ABK_DEFINE_ERROR
 #include "common.cuh"
+#include "differential.cuh"
 
 #define AS_THREADS 128
 #define AS_MAX_GROUP 16
@@ -24,6 +28,8 @@ struct AttnSplit {
     float *parts;        // [tokens, heads, n_parts, v_dim + 2]: weighted values, then maximum and sum
     void *out;           // [tokens, heads * v_dim]
     int n_heads, n_kv_heads, head_dim, v_dim;
+    int maps;            // a key row holds maps * head_dim elements; query head h reads slice h % maps
+    DifferentialHead diff;  // maps 2: what makes a head of its two maps (out is then [tokens, n_heads / 2 * v_dim])
     float scale;
     float softcap;       // > 0: z <- softcap * tanh(z / softcap), after the scale
     int window, keep_first;
@@ -34,7 +40,7 @@ struct AttnSplit {
     PagedCache cache, v_cache;
     int n_parts;
     int values_in_keys;  // a value is the first v_dim elements of its key row (one pool)
-    int one_kv;          // the cache has one kv head; n_kv_heads counts runs of query heads that a CTA takes together
+    int runs;            // runs of query heads, a CTA each, that share a kv head of the cache; n_kv_heads counts the runs
     const void *gate;    // null, or a gate per token and head (of q's type, at gate + t * ldg + h): the head's output is
     long long ldg;       // multiplied by its sigmoid where the parts are folded
 };
@@ -107,11 +113,11 @@ __device__ __forceinline__ void as_split3(float x, float y, uint32_t &hi, uint32
 // stay float32 in effect.
 template <typename T, bool STAGED, int GMAX, bool TC = false> __global__ void __launch_bounds__(AS_THREADS) attention_split_kernel(AttnSplit p) {
     extern __shared__ __align__(16) float as_smem[];
-    const int group = p.n_heads / p.n_kv_heads, hd = p.head_dim, vd = p.v_dim;
+    const int group = p.n_heads / p.n_kv_heads, hd = p.head_dim, vd = p.v_dim, kd = p.maps * hd;  // kd: a key row
     float *q_s = as_smem;                      // [group][hd]
     float *p_s = q_s + group * hd;             // [group][128]
     float *red = p_s + group * AS_THREADS;     // [4][group] maxima, then sums
-    const int k_pitch = hd * (int)sizeof(T) + 16;
+    const int k_pitch = kd * (int)sizeof(T) + 16;
     uint8_t *k_s = (uint8_t *)(red + ((4 * group + 3) & ~3));  // [128][k_pitch]
     uint8_t *v_s = k_s;                                        // [128][vd], once the keys are done with
     __shared__ long long k_off[AS_THREADS], v_off[AS_THREADS];
@@ -129,16 +135,16 @@ template <typename T, bool STAGED, int GMAX, bool TC = false> __global__ void __
     if (valid) {
         const int j = number < kept ? number : lo + number - kept;
         const int page = cache_page(p.cache, slot, j);
-        const int ckv = p.one_kv ? 0 : kvh, cn = p.one_kv ? 1 : p.n_kv_heads;
-        v_off[tid] = cache_offset(p.v_cache, page, ckv, cn, j, p.values_in_keys ? hd : vd);
-        k_off[tid] = cache_offset(p.cache, page, ckv, cn, j, hd);
+        const int ckv = kvh / p.runs, cn = p.n_kv_heads / p.runs;
+        v_off[tid] = cache_offset(p.v_cache, page, ckv, cn, j, p.values_in_keys ? kd : vd);
+        k_off[tid] = cache_offset(p.cache, page, ckv, cn, j, kd);
     }
     const T *q = (const T *)p.q + (long long)t * p.q_row + (long long)kvh * group * hd;
     for (int e = tid; e < group * hd; e += AS_THREADS) q_s[e] = to_float(q[e]);
     __syncthreads();
     if (STAGED) {
         const uint32_t k_dst = (uint32_t)__cvta_generic_to_shared(k_s);
-        const int k_chunks = hd * (int)sizeof(T) / 16;
+        const int k_chunks = kd * (int)sizeof(T) / 16;
         for (int e = tid; e < n_valid * k_chunks; e += AS_THREADS) {
             const int r = e / k_chunks, c = e - r * k_chunks;
             asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(k_dst + r * k_pitch + c * 16),
@@ -182,7 +188,7 @@ template <typename T, bool STAGED, int GMAX, bool TC = false> __global__ void __
         const T *k = STAGED ? (const T *)(k_s + tid * k_pitch) : (const T *)p.k_pool + k_off[tid];
 #pragma unroll
         for (int g = 0; g < GMAX; g++)
-            if (g < group) sc[g] = score_of(p, dot_q<T>(q_s + g * hd, k, hd));
+            if (g < group) sc[g] = score_of(p, dot_q<T>(q_s + g * hd, k + (p.maps == 2 && (g & 1) ? hd : 0), hd));
     } else {
 #pragma unroll
         for (int g = 0; g < GMAX; g++) sc[g] = -INFINITY;
@@ -347,28 +353,70 @@ template <typename T> __global__ void __launch_bounds__(AS_THREADS) attention_fo
     if (tid + AS_THREADS < vd) out[tid + AS_THREADS] = from_float<T>(b / l * g);
 }
 
+// The same for differential attention: out[t, h] of the two maps 2 h and 2 h + 1. One CTA per (token, head).
+template <typename T> __global__ void __launch_bounds__(AS_THREADS) attention_fold_maps_kernel(AttnSplit p) {
+    __shared__ float scratch[33];
+    const int t = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, vd = p.v_dim, heads = p.n_heads / 2;
+    const float sinks[2] = {p.sink ? p.sink[2 * h] : -INFINITY, p.sink ? p.sink[2 * h + 1] : -INFINITY};
+    pdl_wait();
+    T *out = (T *)p.out + ((long long)t * heads + h) * vd;
+    const int seq = p.token_seq[t];
+    if (seq < 0) {
+        for (int d = tid; d < vd; d += AS_THREADS) out[d] = from_float<T>(0.0f);
+        return;
+    }
+    int lo, kept, total;
+    visible_keys(p, p.token_pos[t], lo, kept, total);
+    const int n = (total + AS_THREADS - 1) / AS_THREADS;
+    float a[2], b[2];
+#pragma unroll
+    for (int m = 0; m < 2; m++) {
+        const float *src = p.parts + ((long long)t * p.n_heads + 2 * h + m) * p.n_parts * (vd + 2);
+        float top = sinks[m];
+        for (int i = 0; i < n; i++) top = fmaxf(top, src[(long long)i * (vd + 2) + vd]);
+        float l = p.sink ? expf(sinks[m] - top) : 0.0f;
+        a[m] = b[m] = 0.0f;
+        for (int i = 0; i < n; i++) {
+            const float *part = src + (long long)i * (vd + 2);
+            const float w = expf(part[vd] - top);
+            l = fmaf(part[vd + 1], w, l);
+            if (tid < vd) a[m] = fmaf(part[tid], w, a[m]);
+            if (tid + AS_THREADS < vd) b[m] = fmaf(part[tid + AS_THREADS], w, b[m]);
+        }
+        a[m] /= l, b[m] /= l;
+    }
+    const float x = differential_value(p.diff, a[0], a[1]), y = differential_value(p.diff, b[0], b[1]);  // (0 beyond vd)
+    const float scale = differential_scale(p.diff, block_sum(fmaf(x, x, y * y), scratch), vd);
+    if (tid < vd) out[tid] = from_float<T>(x * scale);
+    if (tid + AS_THREADS < vd) out[tid + AS_THREADS] = from_float<T>(y * scale);
+}
+
 // max_keys: an upper bound of the keys any row of the step sees (its position + 1, or window + keep_first);
 // parts: float32 scratch of at least tokens * heads * ceil(max_keys / 128) * (v_dim + 2).
-static int attention_split(int values_in_keys, int chunk, float softcap, const void *q, long long q_row, void *out, int dtype, int n_tokens, int n_heads,
+static int attention_split(const DifferentialHead *diff, int values_in_keys, int chunk, float softcap, const void *q, long long q_row, void *out, int dtype, int n_tokens, int n_heads,
                                    int n_kv_heads, int head_dim, int v_dim, float scale, int window, int keep_first,
                                    const float *sink, const int *token_seq, const int *token_pos, const int *seq_slot,
                                    const void *k_pool, const void *v_pool, const int *page_table, int table_width,
                                    int ring_pages, int pinned_pages, int tokens_per_page, int max_keys, float *parts,
                                    long long parts_floats, const void *gate, long long ldg, void *stream) {
     if (n_tokens <= 0) return 0;
-    if (head_dim > AS_MAX_DIM || head_dim % 8 || head_dim < 8) ABK_REFUSE("attention_split: head_dim %d is not a multiple of 8 up to %d", head_dim, AS_MAX_DIM);
+    const int maps = diff ? 2 : 1;
+    if (maps * head_dim > 2 * AS_MAX_DIM || head_dim > AS_MAX_DIM || head_dim % 8 || head_dim < 8) ABK_REFUSE("attention_split: head_dim %d is not a multiple of 8 up to %d", head_dim, AS_MAX_DIM);
     if (v_dim < 1 || v_dim > AS_MAX_DIM) ABK_REFUSE("attention_split: value size %d is not 1 to %d", v_dim, AS_MAX_DIM);
-    int one_kv = 0;
-    if (values_in_keys && n_kv_heads == 1 && n_heads > AS_MAX_GROUP) {
-        // one kv head for more query heads than a CTA takes: the heads go in runs of the largest divisor up to 16,
-        // each run a CTA of its own over the same cache rows
+    int runs = 1;
+    if (n_kv_heads >= 1 && n_heads % n_kv_heads == 0 && n_heads / n_kv_heads > AS_MAX_GROUP) {
+        // more query heads to a kv head than a CTA takes: they go in runs of the largest divisor up to 16 (of whole heads,
+        // where a head has two maps), each run a CTA of its own over the same cache rows
+        const int group = n_heads / n_kv_heads;
         int run = AS_MAX_GROUP;
-        while (n_heads % run) run--;
-        n_kv_heads = n_heads / run, one_kv = 1;
+        while (run > 1 && (group % run || run % maps)) run--;
+        if (run % maps == 0) runs = group / run, n_kv_heads *= runs;
     }
     if (n_kv_heads < 1 || n_heads % n_kv_heads || n_heads / n_kv_heads > AS_MAX_GROUP)
         ABK_REFUSE("attention_split: %d query heads to %d kv heads (groups of up to %d)", n_heads, n_kv_heads, AS_MAX_GROUP);
-    if (n_heads > 65535 || max_keys < 1) ABK_REFUSE("attention_split: %d heads, %d keys", n_heads, max_keys);
+    if (maps == 2 && (n_heads / n_kv_heads % 2 || values_in_keys || gate))
+        ABK_REFUSE("attention_split: the two maps of a head go with values of their own and no gate");
+    if (n_heads > 65535 || n_kv_heads > 65535 || max_keys < 1) ABK_REFUSE("attention_split: %d heads, %d keys", n_heads, max_keys);
     AttnSplit p;
     p.q = q, p.q_row = q_row, p.parts = parts, p.out = out, p.n_heads = n_heads, p.n_kv_heads = n_kv_heads;
     p.head_dim = head_dim, p.v_dim = v_dim, p.scale = scale, p.window = window > 0 ? window : 0;
@@ -379,7 +427,8 @@ static int attention_split(int values_in_keys, int chunk, float softcap, const v
     p.cache.tokens_per_page = tokens_per_page, p.cache.pinned_pages = pinned_pages;
     p.v_cache = p.cache;
     p.n_parts = (max_keys + AS_THREADS - 1) / AS_THREADS;
-    p.values_in_keys = values_in_keys, p.one_kv = one_kv, p.gate = gate, p.ldg = ldg;
+    p.values_in_keys = values_in_keys, p.runs = runs, p.gate = gate, p.ldg = ldg;
+    p.maps = maps, p.diff = diff ? *diff : DifferentialHead();
     if (values_in_keys && v_dim > head_dim) ABK_REFUSE("attention_split: values of %d inside keys of %d", v_dim, head_dim);
     if (p.n_parts > 65535) ABK_REFUSE("attention_split: %d keys are more than a grid takes", max_keys);
     if ((long long)n_tokens * n_heads * p.n_parts * (v_dim + 2) > parts_floats)
@@ -389,7 +438,7 @@ static int attention_split(int values_in_keys, int chunk, float softcap, const v
     const bool bf = dtype == ABK_BF16;
     const int esize = bf ? 2 : 4;
     const size_t small = (size_t)(group * head_dim + group * AS_THREADS + ((4 * group + 3) & ~3)) * 4;
-    size_t rows = (size_t)AS_THREADS * (head_dim * esize + 16);  // the keys' rows, then the values' in the same place
+    size_t rows = (size_t)AS_THREADS * (maps * head_dim * esize + 16);  // the keys' rows, then the values' in the same place
     if (!values_in_keys && rows < (size_t)AS_THREADS * v_dim * esize) rows = (size_t)AS_THREADS * v_dim * esize;
     const size_t staged = small + rows;
     // rows of keys and of values that are whole 16-byte pieces at 16-byte places can be staged in shared memory
@@ -397,7 +446,7 @@ static int attention_split(int values_in_keys, int chunk, float softcap, const v
                        !(((uintptr_t)k_pool | (uintptr_t)v_pool) & 15);
     const size_t smem = stage ? staged : small;
     cudaStream_t s = (cudaStream_t)stream;
-    dim3 grid(n_tokens, n_kv_heads, p.n_parts), fold(n_tokens, n_heads);
+    dim3 grid(n_tokens, n_kv_heads, p.n_parts), fold(n_tokens, n_heads / maps);
 #define SPLIT_LAUNCH(T, STAGED, GMAX, ...)                                                                \
     do {                                                                                                  \
         if (smem + 4096 > 48 * 1024) { /* (the kernel's own 2 KB of static shared memory count too) */    \
@@ -426,6 +475,11 @@ static int attention_split(int values_in_keys, int chunk, float softcap, const v
 #undef SPLIT_LAUNCH
     int rc = ABK_LAUNCH_RESULT();
     if (rc) return rc;
+    if (maps == 2) {
+        if (bf) abk_launch(attention_fold_maps_kernel<__nv_bfloat16>, fold, dim3(AS_THREADS), 0, s, p);
+        else abk_launch(attention_fold_maps_kernel<float>, fold, dim3(AS_THREADS), 0, s, p);
+        return ABK_LAUNCH_RESULT();
+    }
     if (bf) abk_launch(attention_fold_kernel<__nv_bfloat16>, fold, dim3(AS_THREADS), 0, s, p);
     else abk_launch(attention_fold_kernel<float>, fold, dim3(AS_THREADS), 0, s, p);
     return ABK_LAUNCH_RESULT();
@@ -438,9 +492,24 @@ extern "C" int abk_attention_split(const void *q, long long q_row, void *out, in
                                    int ring_pages, int pinned_pages, int tokens_per_page, int max_keys, float *parts,
                                    long long parts_floats, int chunk, float softcap, const void *gate, long long ldg,
                                    void *stream) {
-    return attention_split(0, chunk, softcap, q, q_row, out, dtype, n_tokens, n_heads, n_kv_heads, head_dim, v_dim, scale, window, keep_first,
+    return attention_split(nullptr, 0, chunk, softcap, q, q_row, out, dtype, n_tokens, n_heads, n_kv_heads, head_dim, v_dim, scale, window, keep_first,
                            sink, token_seq, token_pos, seq_slot, k_pool, v_pool, page_table, table_width, ring_pages,
                            pinned_pages, tokens_per_page, max_keys, parts, parts_floats, gate, ldg, stream);
+}
+
+// The two maps of differential attention: n_heads counts every map of every head, a key row holds 2 * head_dim elements;
+// out [tokens, n_heads / 2 * v_dim] = keep * o / sqrt(mean(o^2) + eps), o = a1 - lambda * a2.
+extern "C" int abk_attention_split_maps(const void *q, long long q_row, void *out, int dtype, int n_tokens, int n_heads,
+                                        int n_kv_heads, int head_dim, int v_dim, float scale, int window, int keep_first,
+                                        const float *sink, const int *token_seq, const int *token_pos, const int *seq_slot,
+                                        const void *k_pool, const void *v_pool, const int *page_table, int table_width,
+                                        int ring_pages, int pinned_pages, int tokens_per_page, int max_keys, float *parts,
+                                        long long parts_floats, int chunk, float softcap, float lambda, float eps, float keep,
+                                        void *stream) {
+    const DifferentialHead diff = {lambda, eps, keep};
+    return attention_split(&diff, 0, chunk, softcap, q, q_row, out, dtype, n_tokens, n_heads, n_kv_heads, head_dim, v_dim, scale, window,
+                           keep_first, sink, token_seq, token_pos, seq_slot, k_pool, v_pool, page_table, table_width, ring_pages,
+                           pinned_pages, tokens_per_page, max_keys, parts, parts_floats, nullptr, 0, stream);
 }
 
 // Keys that carry their values (a value is the first v_dim elements of its key row; one pool): attention over shared
@@ -449,9 +518,9 @@ extern "C" int abk_attention_split_values_in_keys(const void *q, long long q_row
                                                   int n_heads, int n_kv_heads, int head_dim, int v_dim, float scale,
                                                   const float *sink, const int *token_seq, const int *token_pos,
                                                   const int *seq_slot, const void *k_pool, const int *page_table,
-                                                  int table_width, int tokens_per_page, int max_keys, float *parts,
-                                                  long long parts_floats, void *stream) {
-    return attention_split(1, 0, 0.0f, q, q_row, out, dtype, n_tokens, n_heads, n_kv_heads, head_dim, v_dim, scale, 0, 0, sink,
-                           token_seq, token_pos, seq_slot, k_pool, k_pool, page_table, table_width, 0, 0, tokens_per_page,
+                                                  int table_width, int ring_pages, int tokens_per_page, int window, int max_keys,
+                                                  float *parts, long long parts_floats, void *stream) {
+    return attention_split(nullptr, 1, 0, 0.0f, q, q_row, out, dtype, n_tokens, n_heads, n_kv_heads, head_dim, v_dim, scale, window, 0, sink,
+                           token_seq, token_pos, seq_slot, k_pool, k_pool, page_table, table_width, ring_pages, 0, tokens_per_page,
                            max_keys, parts, parts_floats, nullptr, 0, stream);
 }

@@ -15,24 +15,30 @@
 // Tiles come in by cp.async into rows padded by 16 bytes (ldmatrix without bank conflicts); with two stages the
 // next tile comes in while this one is multiplied.
 //
+// Differential attention (MAPS 2): a head has two maps, which read the two halves of its query and key rows and the same
+// values. A CTA then has eight warps, four for either map, over one copy of the tiles; at the end the second map's warps
+// leave their outputs in shared memory in float32 and the first map's make the head of the two (csrc/differential.cuh).
+//
 // The weights of the second product are float32: each is split into three bfloat16 parts (the value rounded,
 // the remainder rounded, the remainder of that), which together hold its 24 bits, and the product is taken
 // three times into the same float32 accumulators. Scores have bfloat16 operands and so are exact products
 // summed in float32.
 #define ABK_DEFINE_ERROR
 #include "common.cuh"
+#include "differential.cuh"
 #include "mma_tiles.cuh"
 
 #define AW_ROWS 64
 #define AW_KEYS 64
-#define AW_THREADS 128
+#define AW_THREADS 128  // a map
 #define AW_MAX_VT 16  // value columns / 8 a warp accumulates: values of up to 128
 
 struct AttnWindow {
     const __nv_bfloat16 *qkv;  // rows of `row` elements: q heads, then (at k_off) k heads, then (at v_off) v heads
     long long row;
     __nv_bfloat16 *out;        // [tokens, n_heads * v_dim]
-    int n_heads, n_kv_heads, head_dim, v_dim;
+    int n_heads, n_kv_heads, head_dim, v_dim;  // head_dim: of one map
+    DifferentialHead diff;     // MAPS 2: what makes a head of its two maps
     int k_off, v_off;
     float scale_log2;          // score scale times log2(e)
     float scale, softcap;      // softcap > 0: z <- softcap * tanh(scale * (q . k) / softcap), in float32, before the softmax
@@ -59,27 +65,30 @@ template <int N> __device__ __forceinline__ void cp_async_wait() { asm volatile(
 
 // 64 rows of `width` elements (a multiple of 8) from global rows `first ..` (rows from `limit` on are zeros) into
 // shared rows of `pitch` bytes whose first `padded` elements (a multiple of 16 >= width) are all written.
-__device__ __forceinline__ void load_tile(uint32_t dst, int pitch, int padded, const __nv_bfloat16 *src, long long row_pitch,
+template <int THREADS> __device__ __forceinline__ void load_tile(uint32_t dst, int pitch, int padded, const __nv_bfloat16 *src, long long row_pitch,
                                           int first, int limit, int width) {
     const int chunks = padded >> 3;
-    for (int e = threadIdx.x; e < 64 * chunks; e += AW_THREADS) {
+    for (int e = threadIdx.x; e < 64 * chunks; e += THREADS) {
         const int r = e / chunks, c = e - r * chunks;
         const bool real = first + r < limit && c * 8 < width;
         cp_async_16(dst + r * pitch + c * 16, real ? src + (long long)(first + r) * row_pitch + c * 8 : src, real);
     }
 }
 
-__global__ void __launch_bounds__(AW_THREADS) attention_window_kernel(AttnWindow p) {
+// (two maps: a head's halves start at column 0 and at head_dim, a multiple of 16, of a shared row)
+template <int MAPS> __device__ __forceinline__ void attention_window_cta(const AttnWindow &p) {
     extern __shared__ __align__(16) uint8_t aw_smem[];
-    const int D = p.head_dim, VD = p.v_dim;
+    constexpr int THREADS = AW_THREADS * MAPS;
+    const int D = MAPS * p.head_dim, VD = p.v_dim;  // a query or key row
     const int d16 = (D + 15) & ~15, v16 = (VD + 15) & ~15;
     const int pitch_k = d16 * 2 + 16, pitch_v = v16 * 2 + 16;
     const uint32_t q_s = (uint32_t)__cvta_generic_to_shared(aw_smem);
     const uint32_t k_s = q_s + AW_ROWS * pitch_k;                   // p.stages stages
     const uint32_t v_s = k_s + p.stages * AW_KEYS * pitch_k;        // p.stages stages
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, c2 = (lane & 3) * 2;
+    const int warp = (threadIdx.x >> 5) & 3, map = MAPS == 2 ? threadIdx.x >> 7 : 0, lane = threadIdx.x & 31, g = lane >> 2, c2 = (lane & 3) * 2;
+    const int slices = MAPS == 2 ? p.head_dim / 16 : d16 / 16, slice0 = map * slices * 32;  // 16-column steps of a map; its first byte of a row
     const int h = blockIdx.y, kvh = h / (p.n_heads / p.n_kv_heads);
-    const float sink2 = p.sink ? p.sink[h] * 1.4426950408889634f : -INFINITY;  // a weight: ahead of the wait
+    const float sink2 = p.sink ? p.sink[MAPS * h + map] * 1.4426950408889634f : -INFINITY;  // a weight: ahead of the wait
     pdl_wait();
     // which sequence and which of its tiles of 64 rows this CTA has
     int seq = -1, tile = blockIdx.x, start = 0, n = 0;
@@ -105,9 +114,9 @@ __global__ void __launch_bounds__(AW_THREADS) attention_window_kernel(AttnWindow
     const int n_tiles = kept_tiles + w_last - w_first + 1;
 #define TILE_AT(i) ((i) < kept_tiles ? (i) : w_first + (i) - kept_tiles)
 
-    load_tile(q_s, pitch_k, d16, base + (long long)h * D, p.row, r0, n, D);
-    load_tile(k_s, pitch_k, d16, kg, p.row, TILE_AT(0) * AW_KEYS, n, D);
-    load_tile(v_s, pitch_v, v16, vg, p.row, TILE_AT(0) * AW_KEYS, n, VD);
+    load_tile<THREADS>(q_s, pitch_k, d16, base + (long long)h * D, p.row, r0, n, D);
+    load_tile<THREADS>(k_s, pitch_k, d16, kg, p.row, TILE_AT(0) * AW_KEYS, n, D);
+    load_tile<THREADS>(v_s, pitch_v, v16, vg, p.row, TILE_AT(0) * AW_KEYS, n, VD);
     cp_async_commit();
 
     float o[AW_MAX_VT][4];
@@ -123,14 +132,14 @@ __global__ void __launch_bounds__(AW_THREADS) attention_window_kernel(AttnWindow
         const int stage = p.stages == 2 ? it & 1 : 0, key0 = TILE_AT(it) * AW_KEYS;
         if (p.stages == 2 && it + 1 < n_tiles) {  // the next tile into the other stage (its last readers passed the barrier below)
             const int next = TILE_AT(it + 1) * AW_KEYS;
-            load_tile(k_s + (stage ^ 1) * AW_KEYS * pitch_k, pitch_k, d16, kg, p.row, next, n, D);
-            load_tile(v_s + (stage ^ 1) * AW_KEYS * pitch_v, pitch_v, v16, vg, p.row, next, n, VD);
+            load_tile<THREADS>(k_s + (stage ^ 1) * AW_KEYS * pitch_k, pitch_k, d16, kg, p.row, next, n, D);
+            load_tile<THREADS>(v_s + (stage ^ 1) * AW_KEYS * pitch_v, pitch_v, v16, vg, p.row, next, n, VD);
             cp_async_commit();
             cp_async_wait<1>();
         } else {
             if (p.stages == 1 && it > 0) {  // one stage: this tile now (other CTAs of the SM work meanwhile)
-                load_tile(k_s, pitch_k, d16, kg, p.row, key0, n, D);
-                load_tile(v_s, pitch_v, v16, vg, p.row, key0, n, VD);
+                load_tile<THREADS>(k_s, pitch_k, d16, kg, p.row, key0, n, D);
+                load_tile<THREADS>(v_s, pitch_v, v16, vg, p.row, key0, n, VD);
                 cp_async_commit();
             }
             cp_async_wait<0>();
@@ -142,13 +151,13 @@ __global__ void __launch_bounds__(AW_THREADS) attention_window_kernel(AttnWindow
         float s[8][4];
 #pragma unroll
         for (int t = 0; t < 8; t++) s[t][0] = s[t][1] = s[t][2] = s[t][3] = 0.0f;
-        for (int ks = 0; ks < d16 / 16; ks++) {
+        for (int ks = 0; ks < slices; ks++) {
             uint32_t a[4];
-            ldsm_x4(q_s + (warp * 16 + (lane & 15)) * pitch_k + (ks * 16 + (lane >> 4) * 8) * 2, a[0], a[1], a[2], a[3]);
+            ldsm_x4(q_s + slice0 + (warp * 16 + (lane & 15)) * pitch_k + (ks * 16 + (lane >> 4) * 8) * 2, a[0], a[1], a[2], a[3]);
 #pragma unroll
             for (int tp = 0; tp < 4; tp++) {
                 uint32_t b0, b1, b2, b3;
-                ldsm_x4(kt + (tp * 16 + (lane & 7) + ((lane >> 4) << 3)) * pitch_k + (ks * 16 + ((lane >> 3) & 1) * 8) * 2,
+                ldsm_x4(kt + slice0 + (tp * 16 + (lane & 7) + ((lane >> 4) << 3)) * pitch_k + (ks * 16 + ((lane >> 3) & 1) * 8) * 2,
                         b0, b1, b2, b3);
                 mma_bf16(s[2 * tp], a, b0, b1);
                 mma_bf16(s[2 * tp + 1], a, b2, b3);
@@ -250,7 +259,32 @@ __global__ void __launch_bounds__(AW_THREADS) attention_window_kernel(AttnWindow
     }
 #undef TILE_AT
     // out = o / l
-    const float inv_a = 1.0f / l[0], inv_b = 1.0f / l[1];
+    float inv_a = 1.0f / l[0], inv_b = 1.0f / l[1];
+    if constexpr (MAPS == 2) {
+        // the second map's outputs to shared memory (the tiles are done with: the loop ended in a barrier), rows of VD + 8
+        // floats; the first map's warps take them off theirs and norm the rows, a row's columns lying in four lanes
+        float *other = (float *)aw_smem + (warp * 16 + g) * (VD + 8) + c2;
+        if (map == 1) {
+#pragma unroll
+            for (int t = 0; t < AW_MAX_VT; t++)
+                if (t < n_vt && t * 8 + c2 < VD) {
+                    *(float2 *)(other + t * 8) = make_float2(o[t][0] * inv_a, o[t][1] * inv_a);
+                    *(float2 *)(other + 8 * (VD + 8) + t * 8) = make_float2(o[t][2] * inv_b, o[t][3] * inv_b);
+                }
+        }
+        __syncthreads();
+        if (map == 1) return;
+        float sa = 0.0f, sb = 0.0f;
+#pragma unroll
+        for (int t = 0; t < AW_MAX_VT; t++)
+            if (t < n_vt && t * 8 + c2 < VD) {
+                const float2 ra = *(const float2 *)(other + t * 8), rb = *(const float2 *)(other + 8 * (VD + 8) + t * 8);
+                o[t][0] = differential_value(p.diff, o[t][0] * inv_a, ra.x), o[t][1] = differential_value(p.diff, o[t][1] * inv_a, ra.y);
+                o[t][2] = differential_value(p.diff, o[t][2] * inv_b, rb.x), o[t][3] = differential_value(p.diff, o[t][3] * inv_b, rb.y);
+                sa = fmaf(o[t][0], o[t][0], fmaf(o[t][1], o[t][1], sa)), sb = fmaf(o[t][2], o[t][2], fmaf(o[t][3], o[t][3], sb));
+            }
+        inv_a = differential_scale(p.diff, quad_sum(sa), VD), inv_b = differential_scale(p.diff, quad_sum(sb), VD);
+    }
 #pragma unroll
     for (int t = 0; t < AW_MAX_VT; t++) {
         const int col = t * 8 + c2;
@@ -267,13 +301,18 @@ __global__ void __launch_bounds__(AW_THREADS) attention_window_kernel(AttnWindow
     }
 }
 
+__global__ void __launch_bounds__(AW_THREADS) attention_window_kernel(AttnWindow p) { attention_window_cta<1>(p); }
+__global__ void __launch_bounds__(2 * AW_THREADS, 2) attention_window_maps_kernel(AttnWindow p) { attention_window_cta<2>(p); }
+
 // max_tiles: an upper bound of the step's tiles of 64 rows, sum over its sequences of ceil(rows / 64) (the host
 // knows the rows; CTAs beyond the real tiles return at once).
-extern "C" int abk_attention_window(const void *qkv, long long row, void *out, int n_heads, int n_kv_heads, int head_dim,
-                                    int v_dim, int k_off, int v_off, float scale, int window, int keep_first,
-                                    const float *sink, const int *seq_start, int n_seqs, int max_tiles, int chunk,
-                                    float softcap, void *stream) {
+static int attention_window(const DifferentialHead *diff, const void *qkv, long long row, void *out, int n_heads, int n_kv_heads, int head_dim,
+                            int v_dim, int k_off, int v_off, float scale, int window, int keep_first,
+                            const float *sink, const int *seq_start, int n_seqs, int max_tiles, int chunk,
+                            float softcap, void *stream) {
     if (n_seqs <= 0 || max_tiles <= 0) return 0;
+    const int maps = diff ? 2 : 1;
+    if (maps == 2 && (head_dim % 16 || head_dim > 128)) ABK_REFUSE("attention_window: maps of %d are not a multiple of 16 up to 128", head_dim);
     if (head_dim % 8 || head_dim < 8 || head_dim > 256) ABK_REFUSE("attention_window: head_dim %d is not a multiple of 8 up to 256", head_dim);
     if (v_dim % 8 || v_dim < 8 || v_dim > 8 * AW_MAX_VT) ABK_REFUSE("attention_window: value size %d is not a multiple of 8 up to %d", v_dim, 8 * AW_MAX_VT);
     if (row % 8 || k_off % 8 || v_off % 8 || ((uintptr_t)qkv & 15)) ABK_REFUSE("attention_window: rows of q, k and v are not 16-byte aligned");
@@ -285,7 +324,8 @@ extern "C" int abk_attention_window(const void *qkv, long long row, void *out, i
     p.head_dim = head_dim, p.v_dim = v_dim, p.k_off = k_off, p.v_off = v_off, p.scale_log2 = scale * 1.4426950408889634f;
     p.window = window > 0 ? window : 0, p.keep_first = keep_first, p.sink = sink, p.seq_start = seq_start, p.n_seqs = n_seqs;
     p.scale = scale, p.softcap = softcap > 0.0f ? softcap : 0.0f, p.chunk = chunk > 0 ? chunk : 0;
-    const int d16 = (head_dim + 15) & ~15, v16 = (v_dim + 15) & ~15;
+    p.diff = diff ? *diff : DifferentialHead();
+    const int d16 = (maps * head_dim + 15) & ~15, v16 = (v_dim + 15) & ~15;
     static int stages_env = -1;  // ABACUS_WINDOW_STAGES=1|2 pins the number of stages (for comparison)
     if (stages_env < 0) {
         const char *e = getenv("ABACUS_WINDOW_STAGES");
@@ -294,9 +334,36 @@ extern "C" int abk_attention_window(const void *qkv, long long row, void *out, i
     // one stage by default: measured on a B200 (16 heads of 128, window 1,024) a CTA that waits for its tile while the
     // SM's other CTAs work (four fit) beats two stages with three CTAs an SM: 1,100 against 1,376 us for 8 x 2,048 tokens
     p.stages = stages_env ? stages_env : 1;
-    const int smem = (1 + p.stages) * 64 * (d16 * 2 + 16) + p.stages * 64 * (v16 * 2 + 16);
+    int smem = (1 + p.stages) * 64 * (d16 * 2 + 16) + p.stages * 64 * (v16 * 2 + 16);
+    if (maps == 2) {
+        const int outputs = 64 * (v_dim + 8) * 4;  // the second map's, where the tiles were
+        if (smem < outputs) smem = outputs;
+        cudaError_t e = abk_allow_shared_memory((const void *)attention_window_maps_kernel, smem);
+        if (e != cudaSuccess) return (int)e;
+        abk_launch(attention_window_maps_kernel, dim3(max_tiles, n_heads), dim3(2 * AW_THREADS), (size_t)smem, (cudaStream_t)stream, p);
+        return ABK_LAUNCH_RESULT();
+    }
     cudaError_t e = abk_allow_shared_memory((const void *)attention_window_kernel, smem);
     if (e != cudaSuccess) return (int)e;
     abk_launch(attention_window_kernel, dim3(max_tiles, n_heads), dim3(AW_THREADS), (size_t)smem, (cudaStream_t)stream, p);
     return ABK_LAUNCH_RESULT();
+}
+
+extern "C" int abk_attention_window(const void *qkv, long long row, void *out, int n_heads, int n_kv_heads, int head_dim,
+                                    int v_dim, int k_off, int v_off, float scale, int window, int keep_first,
+                                    const float *sink, const int *seq_start, int n_seqs, int max_tiles, int chunk,
+                                    float softcap, void *stream) {
+    return attention_window(nullptr, qkv, row, out, n_heads, n_kv_heads, head_dim, v_dim, k_off, v_off, scale, window, keep_first, sink,
+                            seq_start, n_seqs, max_tiles, chunk, softcap, stream);
+}
+
+// Differential attention: n_heads and n_kv_heads count heads of two maps of head_dim each, laid out head by head as
+// [map 1 | map 2]; sink (null: none) has a number a map, [2 * n_heads].
+extern "C" int abk_attention_window_maps(const void *qkv, long long row, void *out, int n_heads, int n_kv_heads, int head_dim,
+                                         int v_dim, int k_off, int v_off, float scale, int window, int keep_first,
+                                         const float *sink, const int *seq_start, int n_seqs, int max_tiles, int chunk,
+                                         float softcap, float lambda, float eps, float keep, void *stream) {
+    const DifferentialHead diff = {lambda, eps, keep};
+    return attention_window(&diff, qkv, row, out, n_heads, n_kv_heads, head_dim, v_dim, k_off, v_off, scale, window, keep_first, sink,
+                            seq_start, n_seqs, max_tiles, chunk, softcap, stream);
 }

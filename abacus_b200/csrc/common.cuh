@@ -171,11 +171,32 @@ __device__ __forceinline__ float silu_mul_fast(float gate, float up) {
     return gate * r * up;
 }
 
-// The activation of a gated feed-forward times its up value, in the bfloat16 path: ABK_SILU (above) or ABK_RELU.
-enum { ABK_SILU = 0, ABK_RELU = 1 };
-__device__ __forceinline__ float gated_mul(int act, float gate, float up) {
-    return act == ABK_RELU ? fmaxf(gate, 0.0f) * up : silu_mul_fast(gate, up);
+// The activation of a gated feed-forward times its up value: ABK_SILU (above), ABK_RELU, or ABK_CLAMPED, which bounds both
+// first, g = min(gate, limit), u = clamp(up, -limit, limit), and gives g * sigmoid(1.702 g) * (u + 1).
+enum { ABK_SILU = 0, ABK_RELU = 1, ABK_CLAMPED = 2 };
+__device__ __forceinline__ float gated_mul(int act, float gate, float up, float limit) {  // in the bfloat16 path
+    if (act == ABK_RELU) return fmaxf(gate, 0.0f) * up;
+    if (act == ABK_CLAMPED) {
+        const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit) + 1.0f;
+        float e, r;
+        asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(g * (-1.702f * 1.4426950408889634f)));
+        asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.0f + e));
+        return g * r * u;
+    }
+    return silu_mul_fast(gate, up);
 }
+__device__ __forceinline__ float gated_mul_exact(int act, float gate, float up, float limit) {  // in the float32 path
+    if (act == ABK_RELU) return fmaxf(gate, 0.0f) * up;
+    if (act == ABK_CLAMPED) {
+        const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit) + 1.0f;
+        return g / (1.0f + expf(-1.702f * g)) * u;
+    }
+    return gate / (1.0f + expf(-gate)) * up;
+}
+
+// What may be applied to a product's sums where they are stored.
+enum { ABK_OUT_PLAIN = 0, ABK_OUT_RELU_SQUARED = 1 };
+__device__ __forceinline__ float out_act(int act, float v) { return act == ABK_OUT_RELU_SQUARED ? (v > 0.0f ? v * v : 0.0f) : v; }
 
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll

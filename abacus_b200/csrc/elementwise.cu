@@ -181,8 +181,8 @@ extern "C" int abk_add_rmsnorm(float *x, const float *y, const float *w, void *o
 
 // ------------------------------------------------------------------ a branch's output normed, added, and the stream normed
 // x += wy * (y / sqrt(mean(y^2) + eps_y)); out = w * (x / sqrt(mean(x^2) + eps)): the norm behind a branch, the residual
-// sum and the norm ahead of the next branch. y null: nothing is added. With `rows`, output row r is made from row rows[r]
-// and x is left as it is.
+// sum and the norm ahead of the next branch. y null: nothing is added. w null: the next branch reads the stream itself,
+// out = x. With `rows`, output row r is made from row rows[r] and x is left as it is.
 template <typename TO>
 __global__ void __launch_bounds__(256) normed_add_rmsnorm_kernel(float *__restrict__ x, const float *__restrict__ y, const float *__restrict__ wy,
                                                                  const float *__restrict__ w, TO *__restrict__ out, const int *__restrict__ rows,
@@ -204,8 +204,10 @@ __global__ void __launch_bounds__(256) normed_add_rmsnorm_kernel(float *__restri
         float v = xr[j];
         if (yr) v += wy[j] * (yr[j] * scale_y);
         if (yr && !rows) xr[j] = v;
+        if (!w) out[(long long)r * d + j] = from_float<TO>(v);
         ss += v * v;
     }
+    if (!w) return;
     ss = block_sum(ss, scratch);
     const float scale = 1.0f / sqrtf(ss / (float)d + eps);
     TO *o = out + (long long)r * d;
@@ -239,7 +241,7 @@ __global__ void __launch_bounds__(256) normed_add_rmsnorm_row_kernel(float *__re
 #pragma unroll
     for (int i = 0; i < V; i++) {
         const int j = 4 * (threadIdx.x + 256 * i);
-        wv[i] = j < d ? *(const float4 *)(w + j) : zero;
+        wv[i] = w && j < d ? *(const float4 *)(w + j) : zero;
         wb[i] = y && j < d ? *(const float4 *)(wy + j) : zero;
     }
     pdl_wait();
@@ -263,6 +265,14 @@ __global__ void __launch_bounds__(256) normed_add_rmsnorm_row_kernel(float *__re
             v[i].z += wb[i].z * (u[i].z * scale_y), v[i].w += wb[i].w * (u[i].w * scale_y);
             if (!rows && j < d) *(float4 *)(xr + j) = v[i];
         }
+    }
+    if (!w) {
+#pragma unroll
+        for (int i = 0; i < V; i++) {
+            const int j = 4 * (threadIdx.x + 256 * i);
+            if (j < d) store4(out + (long long)r * d + j, v[i].x, v[i].y, v[i].z, v[i].w);
+        }
+        return;
     }
     float ss = 0.0f;
 #pragma unroll
@@ -309,7 +319,8 @@ extern "C" int abk_normed_add_rmsnorm(float *x, const float *y, const float *wy,
 // gate of [block, 2 block), ... With block = inter that is all gates and then all ups (src/model.c:98).
 __device__ __forceinline__ long long gate_column(int j, int block) { return (long long)(j / block) * 2 * block + j % block; }
 template <typename T>
-__global__ void swiglu_kernel(const T *__restrict__ gate_up, T *__restrict__ act, long long total, int inter, int block, int kind) {
+__global__ void swiglu_kernel(const T *__restrict__ gate_up, T *__restrict__ act, long long total, int inter, int block, int kind,
+                              float limit) {
     pdl_wait();
     for (long long e = (long long)blockIdx.x * blockDim.x + threadIdx.x; e < total;
          e += (long long)gridDim.x * blockDim.x) {
@@ -317,13 +328,13 @@ __global__ void swiglu_kernel(const T *__restrict__ gate_up, T *__restrict__ act
         int j = (int)(e - t * inter);
         float g = to_float(gate_up[t * 2 * inter + gate_column(j, block)]);
         float u = to_float(gate_up[t * 2 * inter + gate_column(j, block) + block]);
-        act[e] = from_float<T>(sizeof(T) == 2 || kind != ABK_SILU ? gated_mul(kind, g, u) : g / (1.0f + expf(-g)) * u);
+        act[e] = from_float<T>(sizeof(T) == 2 ? gated_mul(kind, g, u, limit) : gated_mul_exact(kind, g, u, limit));
     }
 }
 
 // bfloat16 with inter and block multiples of 8: eight elements a thread, read and written as 16-byte vectors.
 __global__ void swiglu_bf16x8_kernel(const __nv_bfloat16 *__restrict__ gate_up, __nv_bfloat16 *__restrict__ act,
-                                     long long groups, int inter, int block, int kind) {
+                                     long long groups, int inter, int block, int kind, float limit) {
     pdl_wait();
     const int per_row = inter >> 3;
     for (long long g = (long long)blockIdx.x * blockDim.x + threadIdx.x; g < groups; g += (long long)gridDim.x * blockDim.x) {
@@ -337,14 +348,15 @@ __global__ void swiglu_bf16x8_kernel(const __nv_bfloat16 *__restrict__ gate_up, 
 #pragma unroll
         for (int e = 0; e < 4; e++) {
             float2 gv = __bfloat1622float2(gp[e]), uv = __bfloat1622float2(up[e]);
-            op[e] = __floats2bfloat162_rn(gated_mul(kind, gv.x, uv.x), gated_mul(kind, gv.y, uv.y));
+            op[e] = __floats2bfloat162_rn(gated_mul(kind, gv.x, uv.x, limit), gated_mul(kind, gv.y, uv.y, limit));
         }
         *(uint4 *)(act + t * inter + j) = out;
     }
 }
 
-// The same with the activation ABK_SILU or ABK_RELU (relu(gate) * up).
-extern "C" int abk_gated_act(const void *gate_up, void *act, int dtype, int n_tokens, int inter, int block, int kind, void *stream) {
+// The same with the activation ABK_SILU, ABK_RELU (relu(gate) * up) or ABK_CLAMPED (with its limit).
+extern "C" int abk_gated_act(const void *gate_up, void *act, int dtype, int n_tokens, int inter, int block, int kind, float limit,
+                             void *stream) {
     long long total = (long long)n_tokens * inter;
     if (total <= 0) return 0;
     if (block <= 0 || inter % block) ABK_REFUSE("swiglu: turns of %d columns do not divide %d", block, inter);
@@ -352,7 +364,7 @@ extern "C" int abk_gated_act(const void *gate_up, void *act, int dtype, int n_to
         long long groups = total >> 3, want = (groups + 255) / 256;
         int blocks = (int)(want > abk_sm_count() * 16 ? abk_sm_count() * 16 : want);
         abk_launch(swiglu_bf16x8_kernel, dim3(blocks), dim3(256), 0, (cudaStream_t)stream, (const __nv_bfloat16 *)gate_up,
-                   (__nv_bfloat16 *)act, groups, inter, block, kind);
+                   (__nv_bfloat16 *)act, groups, inter, block, kind, limit);
         return ABK_LAUNCH_RESULT();
     }
     int threads = 256;
@@ -360,14 +372,14 @@ extern "C" int abk_gated_act(const void *gate_up, void *act, int dtype, int n_to
     if (blocks > abk_sm_count() * 32) blocks = abk_sm_count() * 32;
     cudaStream_t s = (cudaStream_t)stream;
     if (dtype == ABK_BF16)
-        abk_launch(swiglu_kernel<__nv_bfloat16>, dim3((int)blocks), dim3(threads), 0, s, (const __nv_bfloat16 *)gate_up, (__nv_bfloat16 *)act, total, inter, block, kind);
+        abk_launch(swiglu_kernel<__nv_bfloat16>, dim3((int)blocks), dim3(threads), 0, s, (const __nv_bfloat16 *)gate_up, (__nv_bfloat16 *)act, total, inter, block, kind, limit);
     else
-        abk_launch(swiglu_kernel<float>, dim3((int)blocks), dim3(threads), 0, s, (const float *)gate_up, (float *)act, total, inter, block, kind);
+        abk_launch(swiglu_kernel<float>, dim3((int)blocks), dim3(threads), 0, s, (const float *)gate_up, (float *)act, total, inter, block, kind, limit);
     return ABK_LAUNCH_RESULT();
 }
 
 extern "C" int abk_swiglu(const void *gate_up, void *act, int dtype, int n_tokens, int inter, int block, void *stream) {
-    return abk_gated_act(gate_up, act, dtype, n_tokens, inter, block, ABK_SILU, stream);
+    return abk_gated_act(gate_up, act, dtype, n_tokens, inter, block, ABK_SILU, 0.0f, stream);
 }
 
 // ------------------------------------------------------------------ q/k/v preparation
@@ -381,6 +393,7 @@ struct QkvPrep {
     void *qkv;
     int n_heads, n_kv_heads, head_dim;
     int v_dim = 0;  // size of a value head where it is not head_dim (0: head_dim); the general kernel alone takes it
+    int maps = 1;   // k heads that share a value head and lie side by side in one cache row (the general kernel alone)
     long long row_size = 0;  // elements between rows of qkv where a row has padding behind its heads (0: none)
     int q_only;  // only the q heads are prepared (keys and values come from elsewhere)
     const int *token_seq, *token_pos, *seq_slot, *seq_len_after;
@@ -400,7 +413,7 @@ template <typename T> __global__ void qkv_prep_kernel(QkvPrep p) {
     pdl_wait();
     int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     int head = blockIdx.y * PREP_WARPS + warp;
-    int total_heads = p.n_heads + 2 * p.n_kv_heads;
+    int total_heads = p.n_heads + p.n_kv_heads + p.n_kv_heads / p.maps;
     if (head >= (p.q_only ? p.n_heads : total_heads)) return;
     int seq = p.token_seq[t];
     if (seq < 0) return;
@@ -411,7 +424,7 @@ template <typename T> __global__ void qkv_prep_kernel(QkvPrep p) {
     int kv_head = is_q ? 0 : is_k ? head - p.n_heads : head - p.n_heads - p.n_kv_heads;
     // a row of qkv: the q heads and the k heads of head_dim, then the v heads of vd
     const long long row_size =
-        p.row_size > 0 ? p.row_size : (long long)(p.n_heads + p.n_kv_heads) * hd + (long long)p.n_kv_heads * vd;
+        p.row_size > 0 ? p.row_size : (long long)(p.n_heads + p.n_kv_heads) * hd + (long long)(p.n_kv_heads / p.maps) * vd;
     T *row = (T *)p.qkv + (long long)t * row_size +
              (is_q || is_k ? (long long)head * hd : (long long)(p.n_heads + p.n_kv_heads) * hd + (long long)kv_head * vd);
     float *b = buf[warp];
@@ -447,7 +460,8 @@ template <typename T> __global__ void qkv_prep_kernel(QkvPrep p) {
     // A windowed cache keeps ring_pages pages; of the positions that share a place only the last is written.
     if (!cache_keeps(p.cache, pos, p.seq_len_after[seq])) return;
     int page = cache_page(p.cache, p.seq_slot[seq], pos);
-    T *dst = (T *)(is_k ? p.k_pool : p.v_pool) + cache_offset(p.cache, page, kv_head, p.n_kv_heads, pos, is_k ? hd : vd);
+    T *dst = is_k ? (T *)p.k_pool + cache_offset(p.cache, page, kv_head / p.maps, p.n_kv_heads / p.maps, pos, p.maps * hd) + kv_head % p.maps * hd
+                  : (T *)p.v_pool + cache_offset(p.cache, page, kv_head, p.n_kv_heads / p.maps, pos, vd);
     if (is_k)
         for (int j = lane; j < hd; j += 32) dst[j] = from_float<T>(b[j]);
     else
@@ -616,13 +630,15 @@ template <int HD> __global__ void __launch_bounds__(FAST_WARPS * 32) qkv_prep_pr
     }
 }
 
-// v_dim: the size of a value head (0: head_dim); pinned_pages: see PagedCache; row_size: elements between rows of qkv.
+// v_dim: the size of a value head (0: head_dim); pinned_pages: see PagedCache; row_size: elements between rows of qkv; maps: that
+// many of the n_kv_heads k heads in a row share a value head (there are n_kv_heads / maps of those) and one row of the cache,
+// side by side.
 extern "C" int abk_qkv_prep_general(void *qkv, int dtype, int n_tokens, int n_heads, int n_kv_heads, int head_dim,
                                     int q_only, const int *token_seq, const int *token_pos, const int *seq_slot,
                                     const int *seq_len_after, const float *q_norm, const float *k_norm, float eps,
                                     const float *cos, const float *sin, int rotary_dim, int interleaved, void *k_pool,
                                     void *v_pool, const int *page_table, int table_width, int ring_pages,
-                                    int tokens_per_page, int v_dim, int pinned_pages, long long row_size, void *stream) {
+                                    int tokens_per_page, int v_dim, int pinned_pages, long long row_size, int maps, void *stream) {
     if (n_tokens <= 0) return 0;
     if (head_dim > MAX_HEAD_DIM || head_dim < 1)
         ABK_REFUSE("qkv_prep: head_dim %d is not 1 to %d", head_dim, MAX_HEAD_DIM);
@@ -630,13 +646,14 @@ extern "C" int abk_qkv_prep_general(void *qkv, int dtype, int n_tokens, int n_he
         ABK_REFUSE("qkv_prep: rotary_dim %d does not fit head_dim %d", rotary_dim, head_dim);
     QkvPrep p;
     p.qkv = qkv, p.n_heads = n_heads, p.n_kv_heads = n_kv_heads, p.head_dim = head_dim, p.q_only = q_only;
-    p.v_dim = v_dim, p.row_size = row_size;
+    if (maps < 1 || n_kv_heads % maps) ABK_REFUSE("qkv_prep: %d k heads in runs of %d", n_kv_heads, maps);
+    p.v_dim = v_dim, p.row_size = row_size, p.maps = maps;
     p.token_seq = token_seq, p.token_pos = token_pos, p.seq_slot = seq_slot, p.seq_len_after = seq_len_after;
     p.q_norm = q_norm, p.k_norm = k_norm, p.eps = eps, p.cos = cos, p.sin = sin;
     p.rotary_dim = rotary_dim, p.interleaved = interleaved, p.k_pool = k_pool, p.v_pool = v_pool;
     p.cache.page_table = page_table, p.cache.table_width = table_width, p.cache.ring_pages = ring_pages;
     p.cache.tokens_per_page = tokens_per_page, p.cache.pinned_pages = pinned_pages;
-    int total_heads = n_heads + 2 * n_kv_heads;
+    int total_heads = n_heads + n_kv_heads + n_kv_heads / maps;
     dim3 grid(n_tokens, (total_heads + PREP_WARPS - 1) / PREP_WARPS);
     cudaStream_t s = (cudaStream_t)stream;
     if (dtype == ABK_BF16)

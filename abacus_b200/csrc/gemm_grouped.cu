@@ -12,7 +12,9 @@
 //                 of stages -> tcgen05.mma 128 x 128 x 16 into tensor memory -> tcgen05.ld epilogue, one warp that
 //                 loads, one that multiplies, four that store. The weights are one matrix [experts * N, K]; a tile's
 //                 weight rows start at expert * N + its column. Tiles beyond the last used one leave at once. Rows of
-//                 padding hold whatever the buffer held; their results are never read.
+//                 padding hold whatever the buffer held; their results are never read. Gated: an expert's matrix holds gate
+//                 and up rows in turns of 64, so that a tile of 128 columns has both of 64 features, and the activation
+//                 is applied where the tile is stored.
 //   moe_unsort    out[t] (+)= sum over k of sorted[place of pair t * top + k], in the order of k.
 // All waits on barriers are bounded (tc::mbar_wait); a wait that runs out sets status word 1.
 #define ABK_DEFINE_ERROR
@@ -25,7 +27,8 @@
 #define GG_K 64
 #define GG_STAGES 4
 #define GG_THREADS 192
-enum { GG_NONE = 0, GG_RELU_SQUARED = 1 };
+enum { GG_NONE = 0, GG_RELU_SQUARED = 1, GG_SILU_GATED = 2, GG_CLAMPED_GATED = 3 };
+#define GG_TURN (GG_BN / 2)  // rows of gate, then of up, of a gated matrix
 
 // ---------------------------------------------------------------- sorting pairs by expert
 __global__ void __launch_bounds__(256) moe_count_kernel(const int *pair_expert, int n_pairs, int *counts, int *rank) {
@@ -129,6 +132,7 @@ struct GemmGrouped {
     const int *tile_expert;
     int *status;
     int vec;  // every 16-column run of an output row starts on a 16-byte boundary
+    float limit;  // of the clamped activation
 };
 
 struct GroupedSmem {
@@ -233,7 +237,28 @@ __global__ void __launch_bounds__(GG_THREADS) gemm_grouped_kernel(const __grid_c
         if (!ok) flags[0] = 1;
         tc::fence_after_sync();
         TO *out = (TO *)g.out + (long long)(p0 + row) * g.ldo;
-        if (ok) {
+        if (ok && ACT >= GG_SILU_GATED) {
+            const int f0 = q0 / 2;  // the tile's first feature
+#pragma unroll 1
+            for (int c0 = 0; c0 < GG_TURN; c0 += 16) {
+                uint32_t v[16], u[16];
+                tc::tmem_ld16(tmem + ((uint32_t)(quarter * 32) << 16) + c0, v);
+                tc::tmem_ld16(tmem + ((uint32_t)(quarter * 32) << 16) + GG_TURN + c0, u);
+                tc::tmem_ld_wait();
+#pragma unroll
+                for (int j = 0; j < 16; j++) {  // gate and up pass through bfloat16, as they do where they are stored in between
+                    const float gate = __bfloat162float(__float2bfloat16_rn(__uint_as_float(v[j])));
+                    const float up = __bfloat162float(__float2bfloat16_rn(__uint_as_float(u[j])));
+                    v[j] = __float_as_uint(gated_mul(ACT == GG_CLAMPED_GATED ? ABK_CLAMPED : ABK_SILU, gate, up, g.limit));
+                }
+                if (g.vec) {
+                    gg_store16(out + f0 + c0, v);
+                } else {
+#pragma unroll
+                    for (int j = 0; j < 16; j++) out[f0 + c0 + j] = from_float<TO>(__uint_as_float(v[j]));
+                }
+            }
+        } else if (ok) {
 #pragma unroll 1
             for (int c0 = 0; c0 < GG_BN; c0 += 16) {
                 if (q0 + c0 >= g.N) break;
@@ -267,19 +292,22 @@ __global__ void __launch_bounds__(GG_THREADS) gemm_grouped_kernel(const __grid_c
 }
 
 // x bfloat16 [max_tiles * 128, K] (sorted rows); w bfloat16 [experts, N, K]; out [max_tiles * 128, ldo] bfloat16 or
-// (out_f32) float32; tile_expert int32 [max_tiles]; status int32 [>= 2].
+// (out_f32) float32; tile_expert int32 [max_tiles]; status int32 [>= 2]. Gated: N counts gate and up rows (a multiple of 128),
+// out has N / 2 columns.
 extern "C" int abk_gemm_grouped(const void *x, const void *w, void *out, long long ldo, int out_f32, int activation,
-                                int max_tiles, int experts, int N, int K, const int *tile_expert, int *status, void *stream) {
+                                int max_tiles, int experts, int N, int K, const int *tile_expert, float limit, int *status, void *stream) {
     if (max_tiles <= 0 || N <= 0) return 0;
     if (K <= 0 || K % 8) ABK_REFUSE("gemm_grouped: K = %d must be a multiple of 8", K);
-    if (activation != GG_NONE && activation != GG_RELU_SQUARED) ABK_REFUSE("gemm_grouped: activation %d is not built", activation);
+    const bool gated = activation == GG_SILU_GATED || activation == GG_CLAMPED_GATED;
+    if (gated && (N % GG_BN || out_f32)) ABK_REFUSE("gemm_grouped: gate and up rows in turns of %d do not fit %d rows", GG_TURN, N);
+    if (activation < GG_NONE || activation > GG_CLAMPED_GATED) ABK_REFUSE("gemm_grouped: activation %d is not built", activation);
     CUtensorMap mx, mw;
     int rc = tmap::bf16_rows_of_128_bytes(x, (long long)max_tiles * GG_ROWS, K, K, GG_ROWS, &mx);
     if (rc) return rc;
     rc = tmap::bf16_rows_of_128_bytes(w, (long long)experts * N, K, K, GG_BN, &mw);
     if (rc) return rc;
     GemmGrouped g;
-    g.out = out, g.ldo = ldo, g.N = N, g.K = K, g.k_blocks = (K + GG_K - 1) / GG_K, g.tile_expert = tile_expert, g.status = status;
+    g.out = out, g.ldo = ldo, g.N = N, g.K = K, g.k_blocks = (K + GG_K - 1) / GG_K, g.tile_expert = tile_expert, g.status = status, g.limit = limit;
     g.vec = ((uintptr_t)out % 16 == 0) && (ldo * (out_f32 ? 4 : 2)) % 16 == 0;
     dim3 grid(max_tiles, (N + GG_BN - 1) / GG_BN);
     if (grid.y > 65535) ABK_REFUSE("gemm_grouped: %d output features are more than a grid takes", N);
@@ -291,6 +319,8 @@ extern "C" int abk_gemm_grouped(const void *x, const void *w, void *out, long lo
         abk_launch(gemm_grouped_kernel<TO, ACT>, grid, dim3(GG_THREADS), (size_t)GroupedSmem::BYTES, s, mx, mw, g); \
     } while (0)
     if (out_f32) { if (activation) GG_LAUNCH(float, 1); else GG_LAUNCH(float, 0); }
+    else if (activation == GG_CLAMPED_GATED) GG_LAUNCH(__nv_bfloat16, GG_CLAMPED_GATED);
+    else if (activation == GG_SILU_GATED) GG_LAUNCH(__nv_bfloat16, GG_SILU_GATED);
     else { if (activation) GG_LAUNCH(__nv_bfloat16, 1); else GG_LAUNCH(__nv_bfloat16, 0); }
 #undef GG_LAUNCH
     return ABK_LAUNCH_RESULT();

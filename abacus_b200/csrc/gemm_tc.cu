@@ -49,7 +49,9 @@ struct GemmTc {
     int *status;
     int vec;  // stride_q == 1 and every 16-column run of a row starts on a 16-byte boundary
     int in_cluster;  // the splits of a tile are a thread-block cluster and add up through distributed shared memory
-    int gated_act = ABK_SILU;  // what EPI_GATED applies to the gate: ABK_SILU or ABK_RELU
+    int gated_act = ABK_SILU;  // what EPI_GATED applies to the gate: ABK_SILU, ABK_RELU or ABK_CLAMPED (with its limit)
+    float gated_limit = 0.0f;
+    int act = ABK_OUT_PLAIN;   // what the other epilogues apply to the sums they store (ABK_OUT_*)
     int weights_are_p;  // which operand is nobody's output (the weights): its first stages are asked for before pdl_wait()
 };
 
@@ -172,6 +174,10 @@ __global__ void __launch_bounds__(GEMM_THREADS) gemm_tc_kernel(const __grid_cons
                 uint32_t v[16];
                 tc::tmem_ld16(tmem + ((uint32_t)(quarter * 32) << 16) + c0, v);
                 tc::tmem_ld_wait();
+                if (direct && g.act) {
+#pragma unroll
+                    for (int j = 0; j < 16; j++) v[j] = __float_as_uint(out_act(g.act, __uint_as_float(v[j])));
+                }
                 if (g.in_cluster) {  // the operands' stages are free: every product has read them
                     float *at = (float *)smem + row * (BN + 4) + c0;
 #pragma unroll
@@ -226,7 +232,7 @@ __global__ void __launch_bounds__(GEMM_THREADS) gemm_tc_kernel(const __grid_cons
                         for (int j = 0; j < 8; j++)
                             if (c0 + j < cols)
                                 out[(long long)p * g.stride_p + (long long)(q0 + c0 + j) * g.stride_q] =
-                                    from_float<TO>(sum[j]);
+                                    from_float<TO>(out_act(g.act, sum[j]));
                     }
                 }
                 if (threadIdx.x == 64) g.tickets[tile] = 0;
@@ -256,7 +262,8 @@ __global__ void __launch_bounds__(GEMM_THREADS) gemm_tc_kernel(const __grid_cons
 #pragma unroll
                     for (int j = 0; j < 4; j++)
                         if (q0 + gi * 4 + j < g.Q)
-                            out[(long long)p * g.stride_p + (long long)(q0 + gi * 4 + j) * g.stride_q] = from_float<TO>(r4[j]);
+                            out[(long long)p * g.stride_p + (long long)(q0 + gi * 4 + j) * g.stride_q] =
+                                from_float<TO>(out_act(g.act, r4[j]));
                 }
             }
         }
@@ -532,7 +539,7 @@ __global__ void __launch_bounds__(EPI == EPI_QKV ? QKV_THREADS : GEMM_THREADS) g
                     for (int j = 0; j < 32; j++) {
                         const float gate = __bfloat162float(__float2bfloat16_rn(__uint_as_float(gv[j])));
                         const float up = __bfloat162float(__float2bfloat16_rn(__uint_as_float(uv[j])));
-                        gv[j] = __float_as_uint(gated_mul(g.gated_act, gate, up));
+                        gv[j] = __float_as_uint(gated_mul(g.gated_act, gate, up, g.gated_limit));
                     }
                     if (p < g.P && f0 + c0 + 32 <= g.Q) {
                         store16(out + (long long)p * g.stride_p + f0 + c0, gv);
@@ -549,6 +556,10 @@ __global__ void __launch_bounds__(EPI == EPI_QKV ? QKV_THREADS : GEMM_THREADS) g
                     tc::tmem_ld16(tmem + ((uint32_t)(quarter * 32) << 16) + b * BN + c0, v);
                     tc::tmem_ld16(tmem + ((uint32_t)(quarter * 32) << 16) + b * BN + c0 + 16, v + 16);
                     tc::tmem_ld_wait();
+                    if (g.act) {
+#pragma unroll
+                        for (int j = 0; j < 32; j++) v[j] = __float_as_uint(out_act(g.act, __uint_as_float(v[j])));
+                    }
 #pragma unroll
                     for (int h = 0; h < 32; h += 16) {
                         if (g.vec && p < g.P && q0 + c0 + h + 16 <= g.Q) {
@@ -722,7 +733,7 @@ __global__ void __launch_bounds__(EPI == EPI_QKV ? QKV_THREADS : GEMM_THREADS) g
                     for (int j = 0; j < 32; j++) {
                         const float gate = __bfloat162float(__float2bfloat16_rn(__uint_as_float(gv[j])));
                         const float up = __bfloat162float(__float2bfloat16_rn(__uint_as_float(uv[j])));
-                        gv[j] = __float_as_uint(gated_mul(g.gated_act, gate, up));
+                        gv[j] = __float_as_uint(gated_mul(g.gated_act, gate, up, g.gated_limit));
                     }
                     if (p < g.P && f0 + c0 + 32 <= g.Q) {
                         store16(out + (long long)p * g.stride_p + f0 + c0, gv);
@@ -739,6 +750,10 @@ __global__ void __launch_bounds__(EPI == EPI_QKV ? QKV_THREADS : GEMM_THREADS) g
                     tc::tmem_ld16(tmem + ((uint32_t)(quarter * 32) << 16) + b * BN + c0, v);
                     tc::tmem_ld16(tmem + ((uint32_t)(quarter * 32) << 16) + b * BN + c0 + 16, v + 16);
                     tc::tmem_ld_wait();
+                    if (g.act) {
+#pragma unroll
+                        for (int j = 0; j < 32; j++) v[j] = __float_as_uint(out_act(g.act, __uint_as_float(v[j])));
+                    }
 #pragma unroll
                     for (int h = 0; h < 32; h += 16) {
                         if (g.vec && p < g.P && q0 + c0 + h + 16 <= g.Q) {
@@ -878,9 +893,9 @@ static int launch_persistent(const CUtensorMap &mp, const CUtensorMap &mq, const
 // act[M, N] = silu(x . gate^T) * (x . up^T), w [2 N, K] holding gate and up rows in turns of 128: the persistent
 // kernel with the activation in its epilogue. Many rows only (more than 256), N a multiple of 128, act bfloat16
 // with 16-byte aligned rows; other shapes are refused (the caller multiplies and activates in two steps).
-// kind: the activation, ABK_SILU or ABK_RELU (relu(gate) * up).
+// kind: the activation, ABK_SILU, ABK_RELU (relu(gate) * up) or ABK_CLAMPED (with its limit).
 extern "C" int abk_gemm_tc_gated(const void *x, const void *w, void *act, int M, int N, int K, long long ldx,
-                                 long long ldw, long long ldo, int kind, int *status, void *stream) {
+                                 long long ldw, long long ldo, int kind, float limit, int *status, void *stream) {
     if (M <= 0 || N <= 0) return 0;
     if (M <= 256 || N % 128 || K <= 0 || K % 8 || ldx % 8 || ldw % 8 || ldo % 8 || (((uintptr_t)x | (uintptr_t)w | (uintptr_t)act) & 15))
         ABK_REFUSE("gemm_tc_swiglu: %d rows, %d features, K = %d are not what the fused kernel takes", M, N, K);
@@ -889,7 +904,7 @@ extern "C" int abk_gemm_tc_gated(const void *x, const void *w, void *act, int M,
     if (!rc) rc = tensor_map(w, 2LL * N, K, ldw, 256, &mw);
     if (rc) return rc;
     GemmTc g;
-    g.out = act, g.P = M, g.Q = N, g.K = K, g.stride_p = ldo, g.stride_q = 1, g.gated_act = kind;
+    g.out = act, g.P = M, g.Q = N, g.K = K, g.stride_p = ldo, g.stride_q = 1, g.gated_act = kind, g.gated_limit = limit;
     g.k_blocks = (K + TILE_K - 1) / TILE_K, g.k_blocks_per_split = g.k_blocks, g.splits = 1;
     g.partials = nullptr, g.tickets = nullptr, g.status = status, g.vec = 1, g.in_cluster = 0, g.weights_are_p = 0;
     if (pairs_win(M, 2 * N) && !abk_pairs_off()) {
@@ -905,7 +920,7 @@ extern "C" int abk_gemm_tc_gated(const void *x, const void *w, void *act, int M,
 
 extern "C" int abk_gemm_tc_swiglu(const void *x, const void *w, void *act, int M, int N, int K, long long ldx,
                                   long long ldw, long long ldo, int *status, void *stream) {
-    return abk_gemm_tc_gated(x, w, act, M, N, K, ldx, ldw, ldo, ABK_SILU, status, stream);
+    return abk_gemm_tc_gated(x, w, act, M, N, K, ldx, ldw, ldo, ABK_SILU, 0.0f, status, stream);
 }
 
 // qkv[M, :n_heads * 128] = the prepared q heads of x . w^T, and the prepared k and the v heads of every token that
@@ -970,10 +985,12 @@ extern "C" int abk_gemm_tc_scratch_tickets() { return 1 << 16; }
 // float32 with row pitch ldo. scratch: float32 [abk_gemm_tc_scratch_floats()]; tickets: int32
 // [abk_gemm_tc_scratch_tickets()], all zero; status: int32 [>= 2], word 1 is set if a wait ran out.
 // force_bn / force_swap / force_splits / force_persistent (0 / -1 / 0 / -1: choose) pin the configuration, for tests.
-extern "C" int abk_gemm_tc(const void *x, const void *w, void *out, int out_dtype, int M, int N, int K, long long ldx,
-                           long long ldw, long long ldo, float *scratch, int *tickets, int *status, int force_bn,
-                           int force_swap, int force_splits, int force_persistent, void *stream) {
+// act (ABK_OUT_*): an activation of the sums where they are stored.
+extern "C" int abk_gemm_tc_act(const void *x, const void *w, void *out, int out_dtype, int M, int N, int K, long long ldx,
+                               long long ldw, long long ldo, float *scratch, int *tickets, int *status, int force_bn,
+                               int force_swap, int force_splits, int force_persistent, int act, void *stream) {
     if (M <= 0 || N <= 0) return 0;
+    if (act != ABK_OUT_PLAIN && act != ABK_OUT_RELU_SQUARED) ABK_REFUSE("gemm_tc: activation %d is not built", act);
     if (K <= 0 || K % 8 || ldx % 8 || ldw % 8)
         ABK_REFUSE("gemm_tc: K = %d and the row pitches %lld, %lld must be multiples of 8", K, ldx, ldw);
     if (((uintptr_t)x | (uintptr_t)w) & 15) ABK_REFUSE("gemm_tc: operands must be 16-byte aligned");
@@ -999,7 +1016,7 @@ extern "C" int abk_gemm_tc(const void *x, const void *w, void *out, int out_dtyp
         if (!rc2) rc2 = tensor_map(w, N, K, ldw, 128, &mw2);
         if (rc2) return rc2;
         GemmTc g2;
-        g2.out = out, g2.P = M, g2.Q = N, g2.K = K, g2.stride_p = ldo, g2.stride_q = 1;
+        g2.act = act, g2.out = out, g2.P = M, g2.Q = N, g2.K = K, g2.stride_p = ldo, g2.stride_q = 1;
         g2.k_blocks = (K + TILE_K - 1) / TILE_K, g2.k_blocks_per_split = g2.k_blocks, g2.splits = 1;
         g2.partials = nullptr, g2.tickets = nullptr, g2.status = status, g2.in_cluster = 0, g2.weights_are_p = 0;
         g2.vec = ((uintptr_t)out % 16 == 0) && (ldo * (out_dtype == ABK_BF16 ? 2 : 4)) % 16 == 0;
@@ -1055,7 +1072,7 @@ extern "C" int abk_gemm_tc(const void *x, const void *w, void *out, int out_dtyp
     rc = tensor_map(w, N, K, ldw, swap ? TILE_P : bn, &mw);
     if (rc) return rc;
     GemmTc g;
-    g.out = out, g.P = P, g.Q = Q, g.K = K;
+    g.act = act, g.out = out, g.P = P, g.Q = Q, g.K = K;
     g.stride_p = swap ? 1 : ldo, g.stride_q = swap ? ldo : 1;
     g.k_blocks = k_blocks, g.k_blocks_per_split = per, g.splits = splits;
     g.partials = scratch, g.tickets = tickets, g.status = status;
@@ -1077,4 +1094,11 @@ extern "C" int abk_gemm_tc(const void *x, const void *w, void *out, int out_dtyp
     else rc = launch_bn<float>(bn, mp, mq, g, grid, s);
     if (rc == ABK_REFUSED) ABK_REFUSE("gemm_tc: no kernel for a column tile of %d", bn);
     return rc;
+}
+
+extern "C" int abk_gemm_tc(const void *x, const void *w, void *out, int out_dtype, int M, int N, int K, long long ldx,
+                           long long ldw, long long ldo, float *scratch, int *tickets, int *status, int force_bn,
+                           int force_swap, int force_splits, int force_persistent, void *stream) {
+    return abk_gemm_tc_act(x, w, out, out_dtype, M, N, K, ldx, ldw, ldo, scratch, tickets, status, force_bn, force_swap,
+                           force_splits, force_persistent, ABK_OUT_PLAIN, stream);
 }

@@ -9,12 +9,14 @@
 //
 //   latent_prep   per token: c = w * x / sqrt(mean(x^2) + eps) over the first `rank` columns of the down-projection,
 //                 the rotation of the shared key part and of every query head's rotated part (pairs (2i, 2i+1) or (i, i + rot_dims / 2),
-//                 angle table [position][rot_dims / 2]; elements beyond rot_dims pass unchanged), the cache write,
-//                 and the query parts put where the attention kernel wants them.
+//                 angle table [position][rot_dims / 2]; elements beyond rot_dims pass unchanged), the cache write (a
+//                 windowed layer's ring of pages: only what is still there after the step), the same row among the step's
+//                 own where a prompt's attention reads it from there, and the query parts put where the attention
+//                 kernel wants them.
 //   head_product  out[t, h, :] = W[h] x[t, h, :] for every head: a product per head with a matrix of its own
 //                 (U_h^T on the plain query part, V_h on the weighted latents), float32 sums in a fixed order.
 //   latent_rows   the cache rows of the step's own tokens, gathered into consecutive rows (for a prompt whose keys
-//                 and values are made in full size from the latents).
+//                 and values are made in full size from another entry's latents).
 //   spread_shared a step's shared rotated key part copied behind every head's plain key part.
 #define ABK_DEFINE_ERROR
 #include "common.cuh"
@@ -34,7 +36,9 @@ struct LatentPrep {
     void *pool;           // cache rows [pages][1][tokens_per_page][row]; null: nothing is written (another entry's cache)
     int row;
     PagedCache cache;
-    const int *token_seq, *token_pos, *seq_slot;
+    void *rows;           // the step's own rows [tokens][ld_rows], the same contents; null: not wanted
+    long long ld_rows;
+    const int *token_seq, *token_pos, *seq_slot, *seq_len_after;
 };
 
 template <typename T> __global__ void __launch_bounds__(128) latent_prep_kernel(LatentPrep p) {
@@ -42,11 +46,15 @@ template <typename T> __global__ void __launch_bounds__(128) latent_prep_kernel(
     const int t = blockIdx.x, tid = threadIdx.x;
     pdl_wait();
     const int seq = p.token_seq[t];
-    if (seq < 0) return;
+    if (seq < 0) {
+        if (p.rows)
+            for (int i = tid; i < p.row; i += 128) ((T *)p.rows)[(long long)t * p.ld_rows + i] = from_float<T>(0.0f);
+        return;
+    }
     const int pos = p.token_pos[t], half = p.rot_dims / 2;
     const T *src = (const T *)p.proj + (long long)t * p.ldp;
     const float *cs = p.cos + (long long)pos * half, *sn = p.sin + (long long)pos * half;
-    if (p.pool) {
+    if (p.pool || p.rows) {
         const T *down = src + p.down_at;
         float ss = 0.0f;
         for (int i = tid; i < p.rank; i += 128) {
@@ -55,17 +63,22 @@ template <typename T> __global__ void __launch_bounds__(128) latent_prep_kernel(
         }
         ss = block_sum(ss, scratch);
         const float inv = 1.0f / sqrtf(ss / (float)p.rank + p.eps);
-        const int page = cache_page(p.cache, p.seq_slot[seq], pos);
-        T *dst = (T *)p.pool + cache_offset(p.cache, page, 0, 1, pos, p.row);
-        for (int i = tid; i < p.rank; i += 128) dst[i] = from_float<T>(to_float(down[i]) * inv * p.norm_w[i]);
+        T *kept = nullptr, *own = p.rows ? (T *)p.rows + (long long)t * p.ld_rows : nullptr;
+        if (p.pool && cache_keeps(p.cache, pos, p.seq_len_after[seq]))
+            kept = (T *)p.pool + cache_offset(p.cache, cache_page(p.cache, p.seq_slot[seq], pos), 0, 1, pos, p.row);
+        auto put = [&](int i, T v) {
+            if (kept) kept[i] = v;
+            if (own) own[i] = v;
+        };
+        for (int i = tid; i < p.rank; i += 128) put(i, from_float<T>(to_float(down[i]) * inv * p.norm_w[i]));
         for (int i = tid; i < half; i += 128) {
             const int ia = p.interleaved ? 2 * i : i, ib = p.interleaved ? 2 * i + 1 : i + half;
             const float u = to_float(down[p.rank + ia]), v = to_float(down[p.rank + ib]);
-            dst[p.rank + ia] = from_float<T>(u * cs[i] - v * sn[i]);
-            dst[p.rank + ib] = from_float<T>(v * cs[i] + u * sn[i]);
+            put(p.rank + ia, from_float<T>(u * cs[i] - v * sn[i]));
+            put(p.rank + ib, from_float<T>(v * cs[i] + u * sn[i]));
         }
-        for (int i = p.rot_dims + tid; i < p.rot; i += 128) dst[p.rank + i] = down[p.rank + i];
-        for (int i = p.rank + p.rot + tid; i < p.row; i += 128) dst[i] = from_float<T>(0.0f);
+        for (int i = p.rot_dims + tid; i < p.rot; i += 128) put(p.rank + i, down[p.rank + i]);
+        for (int i = p.rank + p.rot + tid; i < p.row; i += 128) put(i, from_float<T>(0.0f));
     }
     T *q_out = (T *)p.q_dst + (long long)t * p.ldq;
     const int per_head = p.dim + p.rot;
@@ -97,19 +110,20 @@ template <typename T> __global__ void __launch_bounds__(128) latent_prep_kernel(
 extern "C" int abk_latent_prep(const void *proj, long long ldp, int dtype, int n_tokens, int down_at, int n_heads, int dim,
                                int rot, int rank, int rot_dims, int interleaved, const float *norm_w, float eps, const float *cos,
                                const float *sin, void *q_dst, long long ldq, int q_head, int q_rot_at, int copy_plain,
-                               void *pool, int row, const int *page_table, int table_width, int tokens_per_page,
-                               const int *token_seq, const int *token_pos, const int *seq_slot, void *stream) {
+                               void *pool, int row, const int *page_table, int table_width, int ring_pages, int tokens_per_page,
+                               void *rows, long long ld_rows, const int *token_seq, const int *token_pos, const int *seq_slot,
+                               const int *seq_len_after, void *stream) {
     if (n_tokens <= 0) return 0;
     if (rot_dims < 0 || rot_dims % 2 || rot_dims > rot) ABK_REFUSE("latent_prep: %d rotated dimensions of %d", rot_dims, rot);
-    if (q_head < q_rot_at + rot || (pool && row < rank + rot))
+    if (q_head < q_rot_at + rot || ((pool || rows) && row < rank + rot) || (rows && ld_rows < row))
         ABK_REFUSE("latent_prep: a head of %d or a cache row of %d does not hold %d + %d elements", q_head, row, rank, rot);
     LatentPrep p;
     p.proj = proj, p.ldp = ldp, p.down_at = down_at, p.n_heads = n_heads, p.dim = dim, p.rot = rot, p.rank = rank;
     p.rot_dims = rot_dims, p.interleaved = interleaved, p.norm_w = norm_w, p.eps = eps, p.cos = cos, p.sin = sin, p.q_dst = q_dst, p.ldq = ldq;
     p.q_head = q_head, p.q_rot_at = q_rot_at, p.copy_plain = copy_plain, p.pool = pool, p.row = row;
-    p.cache.page_table = page_table, p.cache.table_width = table_width, p.cache.ring_pages = 0;
-    p.cache.tokens_per_page = tokens_per_page, p.cache.pinned_pages = 0;
-    p.token_seq = token_seq, p.token_pos = token_pos, p.seq_slot = seq_slot;
+    p.cache.page_table = page_table, p.cache.table_width = table_width, p.cache.ring_pages = ring_pages;
+    p.cache.tokens_per_page = tokens_per_page, p.cache.pinned_pages = 0, p.rows = rows, p.ld_rows = ld_rows;
+    p.token_seq = token_seq, p.token_pos = token_pos, p.seq_slot = seq_slot, p.seq_len_after = seq_len_after;
     cudaStream_t s = (cudaStream_t)stream;
     if (dtype == ABK_BF16) abk_launch(latent_prep_kernel<__nv_bfloat16>, dim3(n_tokens), dim3(128), 0, s, p);
     else abk_launch(latent_prep_kernel<float>, dim3(n_tokens), dim3(128), 0, s, p);

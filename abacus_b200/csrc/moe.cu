@@ -7,8 +7,10 @@
 //                   (a learned shift per output that the weights do not see), the weight s * scale. A pair is
 //                   (token, k-th choice), numbered token * top + k; pairs of padding rows carry expert -1. Router
 //                   outputs from `n_real` on stand for experts without matrices that return their input: such a
-//                   pair carries -2 - (output - n_real), which the products skip and moe_combine_weighted knows. With `always` >= 0 every token has one more pair, its last: that expert with
-//                   weight 1 (a shared expert that lies stacked behind the routed ones).
+//                   pair carries -2 - (output - n_real), which the products skip and moe_combine_weighted knows. With
+//                   `always` >= 0 every token has one more pair, its last: that expert with weight 1 (a shared expert that
+//                   lies stacked behind the routed ones). With `bias` z = R x + bias. With `shared_weight` R has one row
+//                   more, and sigmoid of its product is the token's weight of a shared expert.
 //   routed_product  out[pair] = act(W[expert of pair] (scale of pair * x[row of pair])): a product whose matrix is
 //                   chosen per row. With a scale the input is multiplied by it and rounded to its stored type first
 //                   (the weight acts on the expert's input). A CTA stages the pair's row in shared memory; a warp makes
@@ -17,8 +19,10 @@
 //   moe_combine     out[t] (+)= sum over k of pairs[t * top + k], in the order of k.
 //   moe_combine_weighted  out[t] = sum over k of weight[t, k] * (pairs[t * top + k], or x[t] for an expert that returns
 //                   its input), in the order of k: the weight on the experts' outputs, in float32. The pairs' rows lie in
-//                   the pairs' order, or (with `place`) sorted by expert, pair p at row place[p].
-//   routed_product also has the gated form: W holds gate rows then up rows, out = silu(gate . x) * (up . x).
+//                   the pairs' order, or (with `place`) sorted by expert, pair p at row place[p]. With `shared`, what a
+//                   shared expert left in out joins first, times its weight for the token (1 where there is none).
+//   routed_product also has the gated forms: W holds gate and up rows in turns of `block` (all gates then all ups where block
+//                   is their number), out = silu(gate . x) * (up . x), or the clamped form (common.cuh: gated_mul).
 //   relu_squared    x = max(x, 0)^2 in place.
 #define ABK_DEFINE_ERROR
 #include "common.cuh"
@@ -28,10 +32,11 @@ template <typename T>
 __global__ void __launch_bounds__(MR_THREADS) moe_route_kernel(const T *x, long long ldx, const float *router, int d, int experts,
                                                         int top, int score, int always, const int *token_seq,
                                                         int *pair_expert, float *pair_weight, const float *correction,
-                                                        float weight_scale, int n_real) {
-    extern __shared__ __align__(16) float mr_smem[];  // [d, rounded up to 4] the row, [experts] logits, [experts] taken flags,
+                                                        float weight_scale, int n_real, const float *bias, float *shared_weight) {
+    extern __shared__ __align__(16) float mr_smem[];  // [d, rounded up to 4] the row, [experts + 1] logits, [experts] taken flags,
     float *xs = mr_smem, *z = xs + ((d + 3) & ~3);    // [experts] what the choice goes by
-    int *taken = (int *)(z + experts);
+    const int outputs = experts + (shared_weight ? 1 : 0);  // router rows: the last may be the shared expert's
+    int *taken = (int *)(z + experts + 1);
     float *key = (float *)(taken + experts);
     const int softmax_chosen = score == 1;
     const int t = blockIdx.x, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -40,6 +45,7 @@ __global__ void __launch_bounds__(MR_THREADS) moe_route_kernel(const T *x, long 
     pdl_wait();
     if (token_seq[t] < 0) {
         for (int k = tid; k < per; k += MR_THREADS) pair_expert[k] = -1, pair_weight[k] = 0.0f;
+        if (shared_weight && tid == 0) shared_weight[t] = 0.0f;
         return;
     }
     if (always >= 0 && tid == 0) pair_expert[top] = always, pair_weight[top] = 1.0f;
@@ -48,8 +54,8 @@ __global__ void __launch_bounds__(MR_THREADS) moe_route_kernel(const T *x, long 
     __syncthreads();
     const bool vec = d % 4 == 0 && ((uintptr_t)router & 15) == 0;
     constexpr int W = MR_THREADS / 32;
-    for (int e = warp; e < experts;) {  // a warp's router rows, up to four at a time so that their loads are in flight together
-        const int left = (experts - e + W - 1) / W, rows = left < 4 ? left : 4;
+    for (int e = warp; e < outputs;) {  // a warp's router rows, up to four at a time so that their loads are in flight together
+        const int left = (outputs - e + W - 1) / W, rows = left < 4 ? left : 4;
         float acc[4] = {0.0f, 0.0f, 0.0f, 0.0f};
         const float *w = router + (long long)e * d;
         if (rows == 4) lane_dots<4>(w, (long long)W * d, xs, d, lane, vec, acc);
@@ -58,12 +64,13 @@ __global__ void __launch_bounds__(MR_THREADS) moe_route_kernel(const T *x, long 
         else lane_dots<1>(w, 0, xs, d, lane, vec, acc);
         for (int u = 0; u < rows; u++) {
             const float sum = warp_sum(acc[u]);
-            if (lane == 0) z[e + u * W] = sum;
+            if (lane == 0) z[e + u * W] = bias && e + u * W < experts ? sum + bias[e + u * W] : sum;
         }
         e += rows * W;
     }
     __syncthreads();
     if (warp != 0) return;
+    if (shared_weight && lane == 0) shared_weight[t] = 1.0f / (1.0f + expf(-z[experts]));
     if (score == 2) {  // z becomes softmax(z) over all outputs; the choice goes by it plus the correction
         float mx = -INFINITY, sum = 0.0f;
         for (int e = lane; e < experts; e += 32) mx = fmaxf(mx, z[e]);
@@ -107,12 +114,13 @@ __global__ void __launch_bounds__(MR_THREADS) moe_route_kernel(const T *x, long 
 
 extern "C" int abk_moe_route(const void *x, long long ldx, int dtype, const float *router, int n_tokens, int d, int experts,
                              int top, int score, int always, const int *token_seq, int *pair_expert,
-                             float *pair_weight, const float *correction, float weight_scale, int n_real, void *stream) {
+                             float *pair_weight, const float *correction, float weight_scale, int n_real, const float *bias,
+                             float *shared_weight, void *stream) {
     if (n_tokens <= 0) return 0;
     if (top < 1 || top > experts) ABK_REFUSE("moe_route: %d of %d experts", top, experts);
     if (score < 0 || score > 2) ABK_REFUSE("moe_route: score %d is not built", score);
     if (n_real < 0 || n_real > experts) n_real = experts;
-    const size_t smem = (size_t)(((d + 3) & ~3) + 3 * experts) * 4;
+    const size_t smem = (size_t)(((d + 3) & ~3) + 3 * experts + 1) * 4;
     if (smem > 200 * 1024) ABK_REFUSE("moe_route: a row of %d and %d experts do not fit shared memory", d, experts);
     cudaStream_t s = (cudaStream_t)stream;
     if (dtype == ABK_BF16) {
@@ -121,26 +129,29 @@ extern "C" int abk_moe_route(const void *x, long long ldx, int dtype, const floa
             if (e != cudaSuccess) return (int)e;
         }
         abk_launch(moe_route_kernel<__nv_bfloat16>, dim3(n_tokens), dim3(MR_THREADS), smem, s, (const __nv_bfloat16 *)x, ldx, router,
-                   d, experts, top, score, always, token_seq, pair_expert, pair_weight, correction, weight_scale, n_real);
+                   d, experts, top, score, always, token_seq, pair_expert, pair_weight, correction, weight_scale, n_real, bias, shared_weight);
     } else {
         if (smem > 48 * 1024) {
             cudaError_t e = abk_allow_shared_memory((const void *)moe_route_kernel<float>, (int)smem);
             if (e != cudaSuccess) return (int)e;
         }
         abk_launch(moe_route_kernel<float>, dim3(n_tokens), dim3(MR_THREADS), smem, s, (const float *)x, ldx, router, d, experts, top,
-                   score, always, token_seq, pair_expert, pair_weight, correction, weight_scale, n_real);
+                   score, always, token_seq, pair_expert, pair_weight, correction, weight_scale, n_real,
+                   bias, shared_weight);
     }
     return ABK_LAUNCH_RESULT();
 }
 
 #define RP_PER_WARP 4
-enum { RP_NONE = 0, RP_RELU_SQUARED = 1, RP_SILU_GATED = 2 };  // gated: w has 2 * outs rows a matrix, gate rows then up rows
+// gated: w has 2 * outs rows a matrix, gate and up rows in turns of `block`
+enum { RP_NONE = 0, RP_RELU_SQUARED = 1, RP_SILU_GATED = 2, RP_CLAMPED_GATED = 3 };
 
 template <typename T, typename TO, int ACT>
 __global__ void __launch_bounds__(128) routed_product_kernel(const T *__restrict__ x, long long ldx, int pairs_per_row,
                                                              const T *__restrict__ w, const int *pair_expert,
                                                              const float *pair_scale, TO *__restrict__ out, long long ldo,
-                                                             int in, int outs) {
+                                                             int in, int outs, int block, float limit) {
+    constexpr bool GATED = ACT == RP_SILU_GATED || ACT == RP_CLAMPED_GATED;
     extern __shared__ __align__(16) float rp_x[];  // [in]
     const int pair = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     pdl_wait();
@@ -159,12 +170,13 @@ __global__ void __launch_bounds__(128) routed_product_kernel(const T *__restrict
     }
     __syncthreads();
     if (o0 >= outs) return;
-    const T *wr = w + ((long long)e * (ACT == RP_SILU_GATED ? 2 * outs : outs) + o0) * in;
+    // (a turn is a multiple of RP_PER_WARP rows, or all of them, so that a warp's gate rows lie together, and so its up rows)
+    const T *wr = w + ((long long)e * (GATED ? 2 * outs : outs) + (GATED ? o0 / block * 2 * block + o0 % block : o0)) * in;
     const bool vec = in % (16 / (int)sizeof(T)) == 0 && ((uintptr_t)w & 15) == 0;
     float acc[RP_PER_WARP] = {0.0f, 0.0f, 0.0f, 0.0f};
     float up[RP_PER_WARP] = {0.0f, 0.0f, 0.0f, 0.0f};
-    if (ACT == RP_SILU_GATED) {
-        const T *wu = wr + (long long)outs * in;
+    if (GATED) {
+        const T *wu = wr + (long long)block * in;
         if (o0 + RP_PER_WARP <= outs) lane_dots<RP_PER_WARP>(wu, in, rp_x, in, lane, vec, up);
         else
             for (int u = 0; o0 + u < outs; u++) lane_dots<1>(wu + (long long)u * in, 0, rp_x, in, lane, vec, up + u);
@@ -180,15 +192,20 @@ __global__ void __launch_bounds__(128) routed_product_kernel(const T *__restrict
             const float g = to_float(from_float<T>(v)), w_up = to_float(from_float<T>(warp_sum(up[u])));
             v = g / (1.0f + expf(-g)) * w_up;
         }
+        if (ACT == RP_CLAMPED_GATED) {
+            const float g = to_float(from_float<T>(v)), w_up = to_float(from_float<T>(warp_sum(up[u])));
+            v = sizeof(T) == 2 ? gated_mul(ABK_CLAMPED, g, w_up, limit) : gated_mul_exact(ABK_CLAMPED, g, w_up, limit);
+        }
         if (lane == 0 && o0 + u < outs) out[(long long)pair * ldo + o0 + u] = from_float<TO>(v);
     }
 }
 
 // x: the row of pair p is x + (p / pairs_per_row) * ldx (pairs_per_row 1: a row per pair; `top`: a row per token);
-// w [experts][outs][in] of x's type; out [pairs][ldo] of x's type or (out_f32) float32.
+// w [experts][outs][in] of x's type (gated: [experts][2 * outs][in], gate and up rows in turns of `block`, a multiple of 4
+// that divides outs, or outs itself); out [pairs][ldo] of x's type or (out_f32) float32. limit: of the clamped form.
 extern "C" int abk_routed_product(const void *x, long long ldx, int pairs_per_row, int dtype, const void *w,
                                   const int *pair_expert, const float *pair_scale, void *out, long long ldo, int out_f32,
-                                  int activation, int n_pairs, int in, int outs, void *stream) {
+                                  int activation, int n_pairs, int in, int outs, int block, float limit, void *stream) {
     if (n_pairs <= 0 || outs <= 0) return 0;
     if (in < 1 || (size_t)in * 4 > 200 * 1024) ABK_REFUSE("routed_product: an inner size of %d does not fit shared memory", in);
     if (pairs_per_row < 1) pairs_per_row = 1;
@@ -204,13 +221,23 @@ extern "C" int abk_routed_product(const void *x, long long ldx, int pairs_per_ro
             if (e != cudaSuccess) return (int)e;                                                                    \
         }                                                                                                           \
         abk_launch(routed_product_kernel<T, TO, ACT>, grid, dim3(128), smem, s, (const T *)x, ldx, pairs_per_row,   \
-                   (const T *)w, pair_expert, pair_scale, (TO *)out, ldo, in, outs);                                \
+                   (const T *)w, pair_expert, pair_scale, (TO *)out, ldo, in, outs, block, limit);                                \
     } while (0)
-    const bool relu2 = activation == RP_RELU_SQUARED, gated = activation == RP_SILU_GATED;
-    if (activation != RP_NONE && !relu2 && !gated) ABK_REFUSE("routed_product: activation %d is not built", activation);
-    if (dtype == ABK_BF16 && out_f32) { if (gated) RP_LAUNCH(bf, float, 2); else if (relu2) RP_LAUNCH(bf, float, 1); else RP_LAUNCH(bf, float, 0); }
-    else if (dtype == ABK_BF16) { if (gated) RP_LAUNCH(bf, bf, 2); else if (relu2) RP_LAUNCH(bf, bf, 1); else RP_LAUNCH(bf, bf, 0); }
-    else { if (gated) RP_LAUNCH(float, float, 2); else if (relu2) RP_LAUNCH(float, float, 1); else RP_LAUNCH(float, float, 0); }
+    const bool gated = activation == RP_SILU_GATED || activation == RP_CLAMPED_GATED;
+    if (activation < RP_NONE || activation > RP_CLAMPED_GATED) ABK_REFUSE("routed_product: activation %d is not built", activation);
+    if (gated && (block <= 0 || outs % block || (block % RP_PER_WARP && block != outs)))
+        ABK_REFUSE("routed_product: turns of %d rows do not fit %d features", block, outs);
+#define RP_BY_ACT(T, TO)                                                                                             \
+    do {                                                                                                            \
+        if (activation == RP_CLAMPED_GATED) RP_LAUNCH(T, TO, RP_CLAMPED_GATED);                                     \
+        else if (activation == RP_SILU_GATED) RP_LAUNCH(T, TO, RP_SILU_GATED);                                      \
+        else if (activation == RP_RELU_SQUARED) RP_LAUNCH(T, TO, RP_RELU_SQUARED);                                  \
+        else RP_LAUNCH(T, TO, RP_NONE);                                                                             \
+    } while (0)
+    if (dtype == ABK_BF16 && out_f32) RP_BY_ACT(bf, float);
+    else if (dtype == ABK_BF16) RP_BY_ACT(bf, bf);
+    else RP_BY_ACT(float, float);
+#undef RP_BY_ACT
 #undef RP_LAUNCH
     return ABK_LAUNCH_RESULT();
 }
@@ -235,37 +262,62 @@ extern "C" int abk_moe_combine(const float *pairs, float *out, int n_tokens, int
     return ABK_LAUNCH_RESULT();
 }
 
-template <typename T>
+// VEC: four columns a thread as one 16-byte piece (d a multiple of 4).
+template <typename T, bool VEC>
 __global__ void __launch_bounds__(256) moe_combine_weighted_kernel(const float *pairs, const float *weight, const int *expert,
                                                                    const T *x, long long ldx, float *out, long long total, int d,
-                                                                   int top, const int *place) {
+                                                                   int top, const int *place, int shared, const float *shared_weight) {
+    constexpr int W = VEC ? 4 : 1;
     pdl_wait();
-    const long long i = (long long)blockIdx.x * 256 + threadIdx.x;
+    const long long i = ((long long)blockIdx.x * 256 + threadIdx.x) * W;
     if (i >= total) return;
     const long long t = i / d, j = i - t * d;
-    float acc = 0.0f;
+    float acc[W];
+#pragma unroll
+    for (int u = 0; u < W; u++) acc[u] = 0.0f;
+    if (shared) {  // what a shared expert left in out
+        const float sw = shared_weight ? shared_weight[t] : 1.0f;
+        if (VEC) {
+            const float4 r = *(const float4 *)(out + i);
+            acc[0] = sw * r.x, acc[W > 1 ? 1 : 0] = sw * r.y, acc[W > 2 ? 2 : 0] = sw * r.z, acc[W > 3 ? 3 : 0] = sw * r.w;
+        } else {
+            acc[0] = sw * out[i];
+        }
+    }
     for (int k = 0; k < top; k++) {
         const int e = expert[t * top + k];
         if (e == -1) continue;  // a padding row
         const long long at = place && e >= 0 ? place[t * top + k] : t * top + k;  // rows sorted by expert: the pair's place
-        acc = fmaf(weight[t * top + k], e >= 0 ? pairs[at * d + j] : to_float(x[t * ldx + j]), acc);
+        const float w = weight[t * top + k];
+        if (VEC && e >= 0) {
+            const float4 r = *(const float4 *)(pairs + at * d + j);
+            acc[0] = fmaf(w, r.x, acc[0]), acc[W > 1 ? 1 : 0] = fmaf(w, r.y, acc[W > 1 ? 1 : 0]);
+            acc[W > 2 ? 2 : 0] = fmaf(w, r.z, acc[W > 2 ? 2 : 0]), acc[W > 3 ? 3 : 0] = fmaf(w, r.w, acc[W > 3 ? 3 : 0]);
+        } else {
+#pragma unroll
+            for (int u = 0; u < W; u++) acc[u] = fmaf(w, e >= 0 ? pairs[at * d + j + u] : to_float(x[t * ldx + j + u]), acc[u]);
+        }
     }
-    out[i] = acc;
+    if (VEC) *(float4 *)(out + i) = make_float4(acc[0], acc[W > 1 ? 1 : 0], acc[W > 2 ? 2 : 0], acc[W > 3 ? 3 : 0]);
+    else out[i] = acc[0];
 }
 
 // out float32 [tokens][d] = sum_k weight[t, k] * (pairs[t * top + k], or x[t] where expert[t, k] <= -2). place (or null):
-// pair p's row in `pairs` is place[p] (rows sorted by expert), not p.
+// pair p's row in `pairs` is place[p] (rows sorted by expert), not p. shared: out holds a shared expert's output, which
+// joins the sum times shared_weight[t] (null: as it is).
 extern "C" int abk_moe_combine_weighted(const float *pairs, const float *weight, const int *expert, const void *x, long long ldx,
-                                        int dtype, float *out, int n_tokens, int d, int top, const int *place, void *stream) {
+                                        int dtype, float *out, int n_tokens, int d, int top, const int *place, int shared,
+                                        const float *shared_weight, void *stream) {
     const long long total = (long long)n_tokens * d;
     if (total <= 0) return 0;
-    const unsigned blocks = (unsigned)((total + 255) / 256);
-    if (dtype == ABK_BF16)
-        abk_launch(moe_combine_weighted_kernel<__nv_bfloat16>, dim3(blocks), dim3(256), 0, (cudaStream_t)stream, pairs, weight,
-                   expert, (const __nv_bfloat16 *)x, ldx, out, total, d, top, place);
-    else
-        abk_launch(moe_combine_weighted_kernel<float>, dim3(blocks), dim3(256), 0, (cudaStream_t)stream, pairs, weight, expert,
-                   (const float *)x, ldx, out, total, d, top, place);
+    const bool vec = d % 4 == 0 && (((uintptr_t)pairs | (uintptr_t)out) & 15) == 0;
+    const unsigned blocks = (unsigned)((total / (vec ? 4 : 1) + 255) / 256);
+#define MC_LAUNCH(T, VEC)                                                                                                       \
+    abk_launch(moe_combine_weighted_kernel<T, VEC>, dim3(blocks), dim3(256), 0, (cudaStream_t)stream, pairs, weight, expert, \
+               (const T *)x, ldx, out, total, d, top, place, shared, shared_weight)
+    if (dtype == ABK_BF16) { if (vec) MC_LAUNCH(__nv_bfloat16, true); else MC_LAUNCH(__nv_bfloat16, false); }
+    else { if (vec) MC_LAUNCH(float, true); else MC_LAUNCH(float, false); }
+#undef MC_LAUNCH
     return ABK_LAUNCH_RESULT();
 }
 

@@ -122,7 +122,7 @@ class CStep:
         for b in model.blocks:
             if type(b) is not PreNormBlock or type(b.mixer) is not Attention or type(b.ffn) is not GatedMLP:
                 return False
-            if b.mixer.whole or b.mixer.spec.head_gate or b.ffn.spec.activation != "silu":  # (options the walker's entries do not carry)
+            if b.mixer.whole or b.mixer.maps > 1 or b.mixer.spec.head_gate or b.ffn.spec.activation != "silu":  # (options the walker's entries do not carry)
                 return False
             if type(b.mixer_norm) is not RMSNorm or type(b.ffn_norm) is not RMSNorm:
                 return False

@@ -102,13 +102,14 @@ def add_rmsnorm(x, y, weight, out, eps, rows=None, n_rows=None):
 
 def normed_add_rmsnorm(x, y, weight_y, eps_y, weight, out, eps, rows=None, n_rows=None):
     """x += weight_y * y / sqrt(mean(y^2) + eps_y) (y None: nothing); out = weight * x / sqrt(mean(x^2) + eps): the norm
-    behind a branch, the residual sum and the norm ahead of the next branch. x, y float32 [tokens, d]. rows (int32): only
-    those rows are made, into out[0:len(rows)], and x is left as it is."""
+    behind a branch, the residual sum and the norm ahead of the next branch. x, y float32 [tokens, d]. weight None: no norm
+    ahead of the next branch, out = x (in out's type). rows (int32): only those rows are made, into out[0:len(rows)], and x
+    is left as it is."""
     _need_cuda(x, y, weight_y, weight, out, rows)
     lib = load_module("elementwise")
     d = x.shape[-1]
     n = n_rows if n_rows is not None else (rows.numel() if rows is not None else x.shape[0])
-    assert x.dtype == weight.dtype == torch.float32 and weight.numel() == d and x.is_contiguous()
+    assert x.dtype == torch.float32 and x.is_contiguous() and (weight is None or (weight.dtype == x.dtype and weight.numel() == d))
     assert y is None or (y.dtype == weight_y.dtype == torch.float32 and y.is_contiguous() and y.shape[-1] == d == weight_y.numel())
     assert out.is_contiguous() and out.shape[-1] == d and out.shape[0] >= n and (rows is not None or x.shape[0] >= n)
     _check(lib, lib.abk_normed_add_rmsnorm(_p(x), _p(y), _p(weight_y if y is not None else None), _p(weight), _p(out), _i(_dt(out)),
@@ -130,11 +131,14 @@ def embed_sinusoids(batch, table, coarse, fine, n_positions, x, status):
                                         _p(status), _stream()), "embed_sinusoids")
 
 
-ACTIVATIONS = {"silu": 0, "relu": 1}  # what a gated feed-forward applies to its gate (csrc/common.cuh)
+# what a gated feed-forward makes of its gate and up (csrc/common.cuh; "clamped_silu" bounds both at `limit` first)
+ACTIVATIONS = {"silu": 0, "relu": 1, "clamped_silu": 2}
+OUT_ACTIVATIONS = {None: 0, "relu_squared": 1}  # what may be applied to a product's sums where they are stored
 
 
-def swiglu(gate_up, act, block=None, activation="silu"):
-    """act = silu(gate) * up (src/model.c:274-282), or relu(gate) * up. A row of gate_up holds gate and up in turns of
+def swiglu(gate_up, act, block=None, activation="silu", limit=0.0):
+    """act = silu(gate) * up (src/model.c:274-282), or relu(gate) * up, or with "clamped_silu" g sigmoid(1.702 g) (u + 1),
+    g = min(gate, limit), u = clamp(up, -limit, limit). A row of gate_up holds gate and up in turns of
     `block` columns (gate of features [0, block), up of the same, gate of the next block, ...); by default all gates
     and then all ups."""
     _need_cuda(gate_up, act)
@@ -143,12 +147,15 @@ def swiglu(gate_up, act, block=None, activation="silu"):
     assert act.shape == (n, two_i // 2) and act.dtype == gate_up.dtype
     assert gate_up.is_contiguous() and act.is_contiguous()
     _check(lib, lib.abk_gated_act(_p(gate_up), _p(act), _i(_dt(act)), _i(n), _i(two_i // 2), _i(block or two_i // 2),
-                                  _i(ACTIVATIONS[activation]), _stream()), "swiglu")
+                                  _i(ACTIVATIONS[activation]), _f(limit), _stream()), "swiglu")
 
 
 def qkv_prep(qkv, n_heads, n_kv_heads, head_dim, batch, q_norm, k_norm, eps, cos, sin, rotary_dim, interleaved,
-             cache, q_only=False, v_dim=None, row=None):
+             cache, q_only=False, v_dim=None, row=None, maps=1):
     """Per-head norm of q and k, rotary encoding, and the cache write of k and v (src/model.c:247-259).
+
+    maps: runs of that many of the n_kv_heads k heads share a value head and a row of the cache, side by side (the row of
+    qkv then has n_kv_heads / maps value heads).
 
     qkv [T, (Hq + 2 Hkv) * hd] is changed in place. batch: engine.batch.StepBatch. cache: a
     cache.LayerKV or None (nothing written). q_only: only the q heads are prepared.
@@ -157,7 +164,8 @@ def qkv_prep(qkv, n_heads, n_kv_heads, head_dim, batch, q_norm, k_norm, eps, cos
     lib = load_module("elementwise")
     n = batch.n_rows
     vd = v_dim or head_dim
-    heads_size = (n_heads + n_kv_heads) * head_dim + n_kv_heads * vd
+    n_values = n_kv_heads // maps
+    heads_size = (n_heads + n_kv_heads) * head_dim + n_values * vd
     row = row or heads_size  # a row may have padding behind its heads
     assert qkv.is_contiguous() and qkv.shape[1] == row >= heads_size and qkv.shape[0] >= n
     if cos is not None:
@@ -165,10 +173,10 @@ def qkv_prep(qkv, n_heads, n_kv_heads, head_dim, batch, q_norm, k_norm, eps, cos
         if batch.max_position >= cos.shape[0]:
             raise KernelError(f"position {batch.max_position} is beyond the rotary table of {cos.shape[0]} positions")
     if cache is not None:
-        assert cache.k.dtype == qkv.dtype and cache.k.shape[1:] == (n_kv_heads, cache.tokens_per_page, head_dim)
-        assert cache.v.shape[1:] == (n_kv_heads, cache.tokens_per_page, vd)
+        assert cache.k.dtype == qkv.dtype and cache.k.shape[1:] == (n_values, cache.tokens_per_page, maps * head_dim)
+        assert cache.v.shape[1:] == (n_values, cache.tokens_per_page, vd)
     pinned = cache.pinned_pages if cache is not None else 0
-    if vd != head_dim or pinned or row != heads_size:  # the general kernel alone takes values of another size,
+    if vd != head_dim or pinned or row != heads_size or maps > 1:  # the general kernel alone takes values of another size,
         # pinned first pages and padded rows
         _check(lib, lib.abk_qkv_prep_general(
             _p(qkv), _i(_dt(qkv)), _i(n), _i(n_heads), _i(n_kv_heads), _i(head_dim), _i(1 if q_only else 0),
@@ -177,7 +185,7 @@ def qkv_prep(qkv, n_heads, n_kv_heads, head_dim, batch, q_norm, k_norm, eps, cos
             _p(cache.k if cache is not None else None), _p(cache.v if cache is not None else None),
             _p(cache.page_table if cache is not None else None), _i(cache.table_width if cache is not None else 0),
             _i(cache.ring_pages if cache is not None else 0), _i(cache.tokens_per_page if cache is not None else 1),
-            _i(vd), _i(pinned), _ll(row), _stream()), "qkv_prep")
+            _i(vd), _i(pinned), _ll(row), _i(maps), _stream()), "qkv_prep")
         return
     _check(lib, lib.abk_qkv_prep(
         _p(qkv), _i(_dt(qkv)), _i(n), _i(n_heads), _i(n_kv_heads), _i(head_dim), _i(1 if q_only else 0),
@@ -253,16 +261,16 @@ def gemm_rows_takes(x, w, out, m):
             and x.stride(1) == 1 and w.stride(1) == 1 and out.stride(1) == 1)
 
 
-def gemm_rows(x, w, out, m=None):
+def gemm_rows(x, w, out, m=None, activation=None):
     """out[:m] = x[:m] . w^T for m <= 16 rows: the weights stream once through warp-level tensor-core
-    products, no scratch memory (src/model.c:299 and the like)."""
+    products, no scratch memory (src/model.c:299 and the like). activation: applied to the sums (OUT_ACTIVATIONS)."""
     _need_cuda(x, w, out)
     lib = load_module("gemm_rows")
     m = x.shape[0] if m is None else m
     n, k = w.shape
     assert x.shape[1] == k and out.shape[1] == n and x.shape[0] >= m and out.shape[0] >= m
-    _check(lib, lib.abk_gemm_rows(_p(x), _p(w), _p(out), _i(_dt(out)), _i(m), _i(n), _i(k), _ll(x.stride(0)),
-                                  _ll(w.stride(0)), _ll(out.stride(0)), _stream()), "gemm_rows")
+    _check(lib, lib.abk_gemm_rows_act(_p(x), _p(w), _p(out), _i(_dt(out)), _i(m), _i(n), _i(k), _ll(x.stride(0)),
+                                      _ll(w.stride(0)), _ll(out.stride(0)), _i(OUT_ACTIVATIONS[activation]), _stream()), "gemm_rows")
 
 
 def gemm_rows_planes(x, w, out, block, m=None, tanh_from=None):
@@ -283,8 +291,8 @@ def gemm_rows_planes(x, w, out, block, m=None, tanh_from=None):
            "gemm_rows_planes")
 
 
-def gemm_rows_swiglu(x, w_gate_up, act, m=None, block=None, activation="silu"):
-    """act[:m] = silu(x . gate^T) * (x . up^T) (or relu, by activation) for m <= 64 rows, w_gate_up [2 I, K] holding gate and up rows in
+def gemm_rows_swiglu(x, w_gate_up, act, m=None, block=None, activation="silu", limit=0.0):
+    """act[:m] = silu(x . gate^T) * (x . up^T) (or another of ACTIVATIONS) for m <= 64 rows, w_gate_up [2 I, K] holding gate and up rows in
     turns of `block` rows (by default all gates, then all ups): the feed-forward's first product and its
     activation in one kernel (src/model.c:307-308)."""
     _need_cuda(x, w_gate_up, act)
@@ -294,7 +302,7 @@ def gemm_rows_swiglu(x, w_gate_up, act, m=None, block=None, activation="silu"):
     assert x.shape[1] == k and act.shape[1] == two_i // 2 and act.dtype == torch.bfloat16 and act.stride(1) == 1
     _check(lib, lib.abk_gemm_rows_gated(_p(x), _p(w_gate_up), _p(act), _i(m), _i(two_i // 2), _i(k), _ll(x.stride(0)),
                                         _ll(w_gate_up.stride(0)), _ll(act.stride(0)), _i(block or two_i // 2),
-                                        _i(ACTIVATIONS[activation]), _stream()), "gemm_rows_swiglu")
+                                        _i(ACTIVATIONS[activation]), _f(limit), _stream()), "gemm_rows_swiglu")
 
 
 def gemm_tc_swiglu_takes(x, w_gate_up, act, m, block):
@@ -304,8 +312,8 @@ def gemm_tc_swiglu_takes(x, w_gate_up, act, m, block):
             and act.stride(0) % 8 == 0 and act.data_ptr() % 16 == 0 and gemm_tc_takes(x, w_gate_up, act))
 
 
-def gemm_tc_swiglu(x, w_gate_up, act, m=None, activation="silu"):
-    """act[:m] = silu(x . gate^T) * (x . up^T) (or relu, by activation) on the tcgen05 tensor cores for more than 256 rows, w_gate_up
+def gemm_tc_swiglu(x, w_gate_up, act, m=None, activation="silu", limit=0.0):
+    """act[:m] = silu(x . gate^T) * (x . up^T) (or another of ACTIVATIONS) on the tcgen05 tensor cores for more than 256 rows, w_gate_up
     [2 I, K] holding gate and up rows in turns of 128: the activation runs in the product's epilogue, under the
     next tile's multiplication (src/model.c:307-308)."""
     _need_cuda(x, w_gate_up, act)
@@ -315,7 +323,7 @@ def gemm_tc_swiglu(x, w_gate_up, act, m=None, activation="silu"):
     assert x.dtype == torch.bfloat16 and w_gate_up.dtype == torch.bfloat16 and act.dtype == torch.bfloat16
     assert x.shape[1] == k and act.shape[1] == two_i // 2 and x.stride(1) == 1 and w_gate_up.stride(1) == 1 and act.stride(1) == 1
     _check(lib, lib.abk_gemm_tc_gated(_p(x), _p(w_gate_up), _p(act), _i(m), _i(two_i // 2), _i(k), _ll(x.stride(0)),
-                                      _ll(w_gate_up.stride(0)), _ll(act.stride(0)), _i(ACTIVATIONS[activation]),
+                                      _ll(w_gate_up.stride(0)), _ll(act.stride(0)), _i(ACTIVATIONS[activation]), _f(limit),
                                       _p(_Scratch.of(x.device).status), _stream()), "gemm_tc_swiglu")
 
 
@@ -781,11 +789,11 @@ def gemm_tc_takes(x, w, out):
             and x.stride(1) == 1 and w.stride(1) == 1 and out.stride(1) == 1)
 
 
-def gemm_tc(x, w, out, m=None, tile_n=0, swap=-1, splits=0, persistent=-1):
+def gemm_tc(x, w, out, m=None, tile_n=0, swap=-1, splits=0, persistent=-1, activation=None):
     """out[:m] = x[:m] . w^T in bfloat16 on the tcgen05 tensor cores, float32 accumulation.
 
     tile_n, swap, splits and persistent pin the tile configuration (tests); 0 / -1 / 0 / -1 let the
-    kernel choose.
+    kernel choose. activation: applied to the sums (OUT_ACTIVATIONS).
     """
     _need_cuda(x, w, out)
     lib = load_module("gemm_tc")
@@ -795,9 +803,10 @@ def gemm_tc(x, w, out, m=None, tile_n=0, swap=-1, splits=0, persistent=-1):
     assert x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16
     assert x.shape[1] == k and out.shape[1] == n and x.shape[0] >= m and out.shape[0] >= m
     assert x.stride(1) == 1 and w.stride(1) == 1 and out.stride(1) == 1
-    _check(lib, lib.abk_gemm_tc(_p(x), _p(w), _p(out), _i(_dt(out)), _i(m), _i(n), _i(k), _ll(x.stride(0)),
-                                _ll(w.stride(0)), _ll(out.stride(0)), _p(sc.gemm_floats), _p(sc.gemm_tickets),
-                                _p(sc.status), _i(tile_n), _i(swap), _i(splits), _i(persistent), _stream()), "gemm_tc")
+    _check(lib, lib.abk_gemm_tc_act(_p(x), _p(w), _p(out), _i(_dt(out)), _i(m), _i(n), _i(k), _ll(x.stride(0)),
+                                    _ll(w.stride(0)), _ll(out.stride(0)), _p(sc.gemm_floats), _p(sc.gemm_tickets),
+                                    _p(sc.status), _i(tile_n), _i(swap), _i(splits), _i(persistent),
+                                    _i(OUT_ACTIVATIONS[activation]), _stream()), "gemm_tc")
 
 
 # ------------------------------------------------------------------ streams (csrc/streams.cu)
@@ -977,13 +986,14 @@ def gated_head_norm(o, gate, weight, out, n_tokens, n_heads, value_dim, eps, sil
 
 # ------------------------------------------------------------------ latent attention (csrc/latent.cu)
 def latent_prep(proj, down_at, n_heads, dim, rot, rank, rot_dims, norm_w, eps, cos, sin, q_dst, q_head, q_rot_at, copy_plain,
-                cache, batch, interleaved=True):
+                cache, batch, interleaved=True, rows=None):
     """What stands between the projections of a latent-attention layer and its attention kernel, per token: the
     latent c = norm_w * z / sqrt(mean(z^2) + eps) over the first `rank` columns of the down-projection (proj[:,
     down_at:]), the rotation (pairs (2i, 2i+1), or with interleaved False (i, i + rot_dims / 2), of the first rot_dims
     elements) of the shared key part behind it and of
     every query head's rotated part (proj[:, h * (dim + rot) + dim:]), the row [c | r | zeros] written to the cache
-    (cache: a cache.LayerKV whose rows hold at least rank + rot elements; None: the entry reads another's cache), and
+    (cache: a cache.LayerKV whose rows hold at least rank + rot elements; of a window's ring of pages only what is still
+    there after the step; None: the entry reads another's cache) and, with `rows`, to rows[token] (the step's own), and
     the query parts put into q_dst: head h of a row at h * q_head, its rotated part at + q_rot_at (zeros behind it up
     to the head's end), its plain part (copy_plain) at + 0."""
     _need_cuda(proj, norm_w, cos, sin, q_dst)
@@ -996,16 +1006,20 @@ def latent_prep(proj, down_at, n_heads, dim, rot, rank, rot_dims, norm_w, eps, c
     if cos is None:
         rot_dims = 0
     if cache is not None:
-        assert cache.k.dtype == proj.dtype and cache.k.shape[1] == 1 and cache.ring_pages == 0 and cache.k.is_contiguous()
+        assert cache.k.dtype == proj.dtype and cache.k.shape[1] == 1 and cache.k.is_contiguous()
         assert norm_w.dtype == torch.float32 and norm_w.numel() == rank
+        assert rows is None or rows.shape[1] == cache.k.shape[-1]
+    assert rows is None or (rows.dtype == proj.dtype and rows.stride(1) == 1 and rows.shape[0] >= n and norm_w is not None)
     _check(lib, lib.abk_latent_prep(
         _p(proj), _ll(proj.stride(0)), _i(_dt(proj)), _i(n), _i(down_at), _i(n_heads), _i(dim), _i(rot), _i(rank),
         _i(rot_dims), _i(1 if interleaved else 0), _p(norm_w), _f(eps), _p(cos), _p(sin), _p(q_dst), _ll(q_dst.stride(0)),
         _i(q_head), _i(q_rot_at),
         _i(1 if copy_plain else 0), _p(cache.k if cache is not None else None),
-        _i(cache.k.shape[-1] if cache is not None else 0), _p(cache.page_table if cache is not None else None),
-        _i(cache.table_width if cache is not None else 0), _i(cache.tokens_per_page if cache is not None else 1),
-        _p(batch.token_seq), _p(batch.token_pos), _p(batch.seq_slot), _stream()), "latent_prep")
+        _i(cache.k.shape[-1] if cache is not None else rows.shape[1] if rows is not None else 0),
+        _p(cache.page_table if cache is not None else None), _i(cache.table_width if cache is not None else 0),
+        _i(cache.ring_pages if cache is not None else 0), _i(cache.tokens_per_page if cache is not None else 1),
+        _p(rows), _ll(rows.stride(0) if rows is not None else 0), _p(batch.token_seq), _p(batch.token_pos), _p(batch.seq_slot),
+        _p(batch.seq_len_after), _stream()), "latent_prep")
 
 
 def head_product(x, x_head, w, out, o_head, n, gate=None):
@@ -1047,36 +1061,99 @@ def spread_shared(shared, keys, k_head, at, count, heads, n):
                                       _i(count), _i(heads), _i(_dt(keys)), _i(n), _stream()), "spread_shared")
 
 
-def attention_values_in_keys(q, out, n_heads, head_dim, v_dim, scale, batch, cache, sink=None, ws=None):
+def attention_values_in_keys(q, out, n_heads, head_dim, v_dim, scale, batch, cache, sink=None, ws=None, window=None, rows=None):
     """Causal attention of every token of the step over a cache with one kv head whose values are the first v_dim
     elements of its keys (latent rows), float32 softmax weights, an optional sink. q [tokens, n_heads * head_dim], out
     [tokens, n_heads * v_dim]. A step of one token a sequence in bfloat16 with rows of up to 256
-    runs split along the keys (csrc/attention_split.cu), everything else on the general kernel."""
-    _need_cuda(q, out, sink)
+    runs split along the keys (csrc/attention_split.cu), everything else on the general kernel. window: only the last
+    `window` keys are seen. rows [tokens, head_dim]: keys come from the step's own rows (whole prompts), not the cache."""
+    _need_cuda(q, out, sink, rows)
     n = batch.n_rows
     assert q.is_contiguous() and q.shape[1] == n_heads * head_dim and out.is_contiguous() and out.dtype == q.dtype
     assert out.shape[1] == n_heads * v_dim and cache.k.dtype == q.dtype and cache.k.shape[1:] == (1, cache.tokens_per_page, head_dim)
-    assert cache.values_in_keys and cache.ring_pages == 0 and v_dim <= head_dim
+    assert cache.values_in_keys and v_dim <= head_dim and (rows is None or (rows.is_contiguous() and rows.dtype == q.dtype
+                                                                            and rows.shape[1] == head_dim and rows.shape[0] >= n))
+    if rows is not None and batch.any_continuation:
+        raise KernelRefused("keys from the step's own rows: every sequence must start at position 0")
+    if rows is None and cache.ring_pages and not batch.is_decode:
+        raise KernelRefused("a window's ring of pages does not hold the keys of every token of a longer step")
     assert sink is None or (sink.dtype == torch.float32 and sink.numel() == n_heads)
-    if batch.is_decode and ws is not None and q.dtype == torch.bfloat16 and head_dim % 8 == 0 and head_dim <= 256:
+    if batch.is_decode and rows is None and ws is not None and q.dtype == torch.bfloat16 and head_dim % 8 == 0 and head_dim <= 256:
         lib = load_module("attention_split")
         top = getattr(batch, "position_bound", None) or batch.max_len_after
         if batch.max_len_after > top:
             raise KernelError(f"a row at position {batch.max_len_after - 1} is beyond the bound {top}")
+        top = min(top, window) if window else top
         n_parts = -(-top // 128)
         parts = ws.get("attention_parts", (n * n_heads * n_parts * (v_dim + 2),), torch.float32)
         _check(lib, lib.abk_attention_split_values_in_keys(
             _p(q), _ll(q.shape[1]), _p(out), _i(_dt(q)), _i(n), _i(n_heads), _i(1), _i(head_dim), _i(v_dim), _f(scale),
             _p(sink), _p(batch.token_seq), _p(batch.token_pos), _p(batch.seq_slot), _p(cache.k), _p(cache.page_table),
-            _i(cache.table_width), _i(cache.tokens_per_page), _i(top), _p(parts), _ll(parts.numel()), _stream()),
-            "attention_split", kernels=2)
+            _i(cache.table_width), _i(cache.ring_pages), _i(cache.tokens_per_page), _i(window or 0), _i(top), _p(parts),
+            _ll(parts.numel()), _stream()), "attention_split", kernels=2)
         return
     lib = load_module("attention_generic")
     _check(lib, lib.abk_attention_values_in_keys(
         _p(q), _ll(q.shape[1]), _p(out), _i(_dt(q)), _i(n), _i(n_heads), _i(1), _i(head_dim), _f(scale),
         _p(batch.token_seq), _p(batch.token_pos), _p(batch.seq_slot), _p(batch.seq_start), _p(batch.seq_pos0), _p(cache.k),
-        _p(cache.page_table), _i(cache.table_width), _i(cache.tokens_per_page), _i(v_dim), _p(sink), _i(1), _stream()),
-        "attention")
+        _p(cache.page_table), _i(cache.table_width), _i(cache.ring_pages), _i(cache.tokens_per_page), _p(rows),
+        _ll(rows.stride(0) if rows is not None else 0), _i(v_dim), _i(window or 0), _p(sink), _i(1), _stream()), "attention")
+
+
+def attention_differential(qkv, out, n_heads, n_kv_heads, head_dim, scale, window, batch, cache, lam, eps, keep, from_step=False,
+                           ws=None, v_dim=None, sink=None, row=None, chunk=None, softcap=None):
+    """Differential attention of a step: every head has two maps, each an attention of its own over the same values, laid
+    out head by head as [map 1 | map 2] (head_dim elements each) in q, in k and in the cache's key rows. Per head
+    o = a1 - lam * a2, then out = keep * o / sqrt(mean(o^2) + eps), all float32. n_heads, n_kv_heads count heads, not maps.
+    Picks the kernel for the phase and sizes, as attention() does, with its options."""
+    _need_cuda(qkv, out, sink)
+    n, vd = batch.n_rows, v_dim or head_dim
+    q_size, k_size = 2 * n_heads * head_dim, 2 * n_kv_heads * head_dim
+    row = row or q_size + k_size + n_kv_heads * vd
+    assert qkv.is_contiguous() and qkv.shape[1] == row >= q_size + k_size + n_kv_heads * vd and qkv.shape[0] >= n
+    assert out.is_contiguous() and out.dtype == qkv.dtype and out.shape[1] == n_heads * vd and out.shape[0] >= n
+    assert sink is None or (sink.dtype == torch.float32 and sink.numel() == 2 * n_heads)
+    assert cache is None or (cache.k.dtype == qkv.dtype and cache.k.shape[-1] == 2 * head_dim and cache.v.shape[-1] == vd)
+    bf16 = qkv.dtype == torch.bfloat16
+    if batch.is_decode and not from_step and ws is not None and bf16 and head_dim % 8 == 0 and head_dim <= 256 and vd <= 256:
+        lib = load_module("attention_split")
+        top = getattr(batch, "position_bound", None) or batch.max_len_after
+        if batch.max_len_after > top:
+            raise KernelError(f"a row at position {batch.max_len_after - 1} is beyond the bound {top}")
+        max_keys = min([top] + [limit for limit in (window, chunk) if limit])
+        parts = ws.get("attention_parts", (n * 2 * n_heads * -(-max_keys // 128) * (vd + 2),), torch.float32)
+        _check(lib, lib.abk_attention_split_maps(
+            _p(qkv), _ll(row), _p(out), _i(_dt(qkv)), _i(n), _i(2 * n_heads), _i(n_kv_heads), _i(head_dim), _i(vd), _f(scale),
+            _i(window or 0), _i(0), _p(sink), _p(batch.token_seq), _p(batch.token_pos), _p(batch.seq_slot), _p(cache.k),
+            _p(cache.v), _p(cache.page_table), _i(cache.table_width), _i(cache.ring_pages), _i(cache.pinned_pages),
+            _i(cache.tokens_per_page), _i(max_keys), _p(parts), _ll(parts.numel()), _i(chunk or 0), _f(softcap or 0.0), _f(lam),
+            _f(eps), _f(keep), _stream()), "attention_split", kernels=2)
+        return
+    if (not batch.is_decode and not batch.any_continuation and bf16 and head_dim % 16 == 0 and head_dim <= 128 and vd % 8 == 0
+            and 8 <= vd <= 128 and row % 8 == 0 and qkv.data_ptr() % 16 == 0):
+        lib = load_module("attention_window")
+        n_seqs = batch.seq_slot.numel()
+        _check(lib, lib.abk_attention_window_maps(
+            _p(qkv), _ll(row), _p(out), _i(n_heads), _i(n_kv_heads), _i(head_dim), _i(vd), _i(q_size), _i(q_size + k_size), _f(scale),
+            _i(window or 0), _i(0), _p(sink), _p(batch.seq_start), _i(n_seqs), _i((n + 63) // 64 + n_seqs), _i(chunk or 0),
+            _f(softcap or 0.0), _f(lam), _f(eps), _f(keep), _stream()), "attention_window")
+        return
+    lib = load_module("attention_generic")
+    maps = (ws.get("attention_maps", (n, 2 * n_heads * vd), torch.float32) if ws is not None
+            else torch.empty((n, 2 * n_heads * vd), dtype=torch.float32, device=qkv.device))
+    esize = qkv.element_size()
+    k_step = ctypes.c_void_p(qkv.data_ptr() + q_size * esize) if from_step else ctypes.c_void_p(0)
+    v_step = ctypes.c_void_p(qkv.data_ptr() + (q_size + k_size) * esize) if from_step else ctypes.c_void_p(0)
+    _check(lib, lib.abk_attention_maps(
+        _p(qkv), _ll(row), _p(maps), _i(_dt(qkv)), _i(n), _i(2 * n_heads), _i(n_kv_heads), _i(head_dim), _i(2), _f(scale),
+        _i(window or 0), _p(batch.token_seq), _p(batch.token_pos), _p(batch.seq_slot), _p(batch.seq_start), _p(batch.seq_pos0),
+        _p(cache.k if cache is not None else None), _p(cache.v if cache is not None else None),
+        _p(cache.page_table if cache is not None else None), _i(cache.table_width if cache is not None else 0),
+        _i(cache.ring_pages if cache is not None else 0), _i(cache.tokens_per_page if cache is not None else 1), k_step, v_step,
+        _ll(row), _i(vd), _i(0), _i(cache.pinned_pages if cache is not None else 0), _p(sink), _i(chunk or 0),
+        _f(softcap or 0.0), _stream()), "attention")
+    _check(lib, lib.abk_differential_heads(_p(maps), _p(out), _i(_dt(out)), _i(n), _i(n_heads), _i(vd), _f(lam), _f(eps), _f(keep),
+                                           _stream()), "differential_heads")
 
 
 # ------------------------------------------------------------------ linear attention with a decay (csrc/lightning.cu)
@@ -1180,21 +1257,27 @@ def matrix_memory(proj, q_at, k_at, v_at, gates, bias_i, bias_f, cap, denom_eps,
 
 # ------------------------------------------------------------------ routed experts (csrc/moe.cu)
 RELU_SQUARED = 1
-SILU_GATED = 2  # the matrix holds gate rows, then up rows: silu(gate . x) * (up . x)
+SILU_GATED = 2  # the matrix holds gate and up rows in turns: silu(gate . x) * (up . x)
+CLAMPED_GATED = 3  # the same with the activation "clamped_silu" of ACTIVATIONS
+GATED = (SILU_GATED, CLAMPED_GATED)
 
 
 def moe_route(x, router, top, batch, pair_expert, pair_weight, softmax_chosen=False, always=None, softmax_all=False,
-              correction=None, weight_scale=1.0, n_real=None):
+              correction=None, weight_scale=1.0, n_real=None, bias=None, shared_weight=None):
     """Per token the `top` experts with the largest router logits (router float32 [experts, d], x as stored) and their
     weights, sigmoid(logit) or the softmax over the chosen; pair token * top + k is the token's k-th choice
     (pair_expert int32, -1 for padding rows; pair_weight float32). always (an expert's index): every token has top + 1
     pairs, the last that expert with weight 1. softmax_all: s = softmax over all router outputs, the choice goes by
     s + correction (float32 [outputs] or None), the weight is s * weight_scale. n_real: router outputs from there on stand
-    for experts that return their input; such a pair carries -2 - (output - n_real)."""
-    _need_cuda(x, router, pair_expert, pair_weight, correction)
-    assert correction is None or (correction.dtype == torch.float32 and correction.numel() == router.shape[0])
+    for experts that return their input; such a pair carries -2 - (output - n_real). bias (float32 [outputs]): added to the
+    logits. shared_weight (float32 [tokens]): the router has one row more, the last; sigmoid of its product goes there."""
+    _need_cuda(x, router, pair_expert, pair_weight, correction, bias, shared_weight)
     lib = load_module("moe")
     n, (experts, d) = batch.n_rows, router.shape
+    experts -= 0 if shared_weight is None else 1
+    assert correction is None or (correction.dtype == torch.float32 and correction.numel() == experts)
+    assert bias is None or (bias.dtype == torch.float32 and bias.numel() == experts)
+    assert shared_weight is None or (shared_weight.dtype == torch.float32 and shared_weight.numel() >= n)
     assert router.dtype == torch.float32 and router.is_contiguous() and x.stride(1) == 1 and x.shape[1] == d
     assert pair_expert.dtype == torch.int32 and pair_weight.dtype == torch.float32
     per = top + (0 if always is None else 1)
@@ -1202,18 +1285,19 @@ def moe_route(x, router, top, batch, pair_expert, pair_weight, softmax_chosen=Fa
     _check(lib, lib.abk_moe_route(_p(x), _ll(x.stride(0)), _i(_dt(x)), _p(router), _i(n), _i(d), _i(experts), _i(top),
                                   _i(2 if softmax_all else 1 if softmax_chosen else 0), _i(-1 if always is None else always),
                                   _p(batch.token_seq), _p(pair_expert), _p(pair_weight), _p(correction), _f(weight_scale),
-                                  _i(experts if n_real is None else n_real), _stream()), "moe_route")
+                                  _i(experts if n_real is None else n_real), _p(bias), _p(shared_weight), _stream()), "moe_route")
 
 
-def routed_product(x, pairs_per_row, w, pair_expert, pair_scale, out, n_pairs, activation=0):
+def routed_product(x, pairs_per_row, w, pair_expert, pair_scale, out, n_pairs, activation=0, block=None, limit=0.0):
     """out[p] = act(w[pair_expert[p]] (pair_scale[p] * x[p // pairs_per_row])) for p < n_pairs: a product whose matrix,
     w [experts, outs, in], is chosen per row. pair_scale None: no scale; with one the scaled input is rounded to x's
-    type first. out of x's type or float32. activation: 0 none, RELU_SQUARED, or SILU_GATED (w [experts, 2 * outs, in]: gate
-    rows, then up rows). Pairs whose expert is negative give zeros."""
+    type first. out of x's type or float32. activation: 0 none, RELU_SQUARED, or one of GATED (w [experts, 2 * outs, in]: gate
+    and up rows in turns of `block`, by default all gates, then all ups; limit: of CLAMPED_GATED). Pairs whose expert is
+    negative give zeros."""
     _need_cuda(x, w, pair_expert, pair_scale, out)
     lib = load_module("moe")
     experts, outs, inner = w.shape
-    if activation == SILU_GATED:
+    if activation in GATED:
         assert outs % 2 == 0
         outs //= 2
     assert x.dtype == w.dtype and w.is_contiguous() and x.stride(1) == 1 and x.shape[1] == inner
@@ -1221,7 +1305,8 @@ def routed_product(x, pairs_per_row, w, pair_expert, pair_scale, out, n_pairs, a
     _check(lib, lib.abk_routed_product(_p(x), _ll(x.stride(0)), _i(pairs_per_row), _i(_dt(x)), _p(w), _p(pair_expert),
                                        _p(pair_scale), _p(out), _ll(out.stride(0)),
                                        _i(1 if out.dtype == torch.float32 and x.dtype != torch.float32 else 0),
-                                       _i(activation), _i(n_pairs), _i(inner), _i(outs), _stream()), "routed_product")
+                                       _i(activation), _i(n_pairs), _i(inner), _i(outs), _i(block or outs), _f(limit), _stream()),
+           "routed_product")
 
 
 def moe_combine(pairs, out, n, top, add):
@@ -1234,11 +1319,13 @@ def moe_combine(pairs, out, n, top, add):
     _check(lib, lib.abk_moe_combine(_p(pairs), _p(out), _i(n), _i(d), _i(top), _i(1 if add else 0), _stream()), "moe_combine")
 
 
-def moe_combine_weighted(pairs, weight, expert, x, out, n, top, place=None):
+def moe_combine_weighted(pairs, weight, expert, x, out, n, top, place=None, shared=False, shared_weight=None):
     """out[t] = sum over k of weight[t * top + k] * (pairs[t * top + k], or x[t] where expert[t * top + k] <= -2: an expert
     that returns its input), in the order of k; pairs, weight and out float32, x as stored. place int32: the rows of
-    `pairs` lie sorted by expert, pair p's at place[p]."""
-    _need_cuda(pairs, weight, expert, x, out)
+    `pairs` lie sorted by expert, pair p's at place[p]. shared: out holds what a shared expert made, which joins the sum
+    times shared_weight[t] (float32; None: as it is)."""
+    _need_cuda(pairs, weight, expert, x, out, shared_weight)
+    assert shared_weight is None or (shared and shared_weight.dtype == torch.float32 and shared_weight.numel() >= n)
     lib = load_module("moe")
     d = out.shape[1]
     assert pairs.dtype == out.dtype == weight.dtype == torch.float32 and pairs.is_contiguous() and out.is_contiguous()
@@ -1250,7 +1337,7 @@ def moe_combine_weighted(pairs, weight, expert, x, out, n, top, place=None):
         _need_cuda(place)
         assert place.dtype == torch.int32 and place.numel() >= n * top
     _check(lib, lib.abk_moe_combine_weighted(_p(pairs), _p(weight), _p(expert), _p(x), _ll(x.stride(0)), _i(_dt(x)), _p(out),
-                                             _i(n), _i(d), _i(top), _p(place) if place is not None else ctypes.c_void_p(0),
+                                             _i(n), _i(d), _i(top), _p(place), _i(1 if shared else 0), _p(shared_weight),
                                              _stream()), "moe_combine_weighted")
 
 
@@ -1263,6 +1350,7 @@ def relu_squared(x, n):
 
 
 # ------------------------------------------------------------------ routed experts over many rows (csrc/gemm_grouped.cu)
+GROUPED_TURN = 64   # rows of gate, then of up, in a gated expert's matrix where the grouped product applies the activation
 GROUPED_ROWS = 128  # rows of a tile of the grouped product: an expert's run of sorted rows is padded to whole tiles
 
 
@@ -1294,18 +1382,21 @@ def moe_sort(x, pairs_per_row, pair_expert, pair_scale, n_pairs, experts, scratc
                                  _i(max_tiles), _p(sorted_rows), _stream()), "moe_sort", kernels=3)
 
 
-def gemm_grouped(x, w, out, tile_expert, activation=0):
+def gemm_grouped(x, w, out, tile_expert, activation=0, limit=0.0):
     """out[p] = act(w[tile_expert[p // 128]] x[p]) for the sorted rows x bfloat16 [tiles * 128, K] on the tcgen05 tensor
-    cores; w bfloat16 [experts, N, K]; out bfloat16 or float32 [tiles * 128, N]. Tiles whose expert is -1 are left alone."""
+    cores; w bfloat16 [experts, N, K]; out bfloat16 or float32 [tiles * 128, N]. Tiles whose expert is -1 are left alone.
+    activation: 0 none, RELU_SQUARED, or one of GATED (w holds gate and up rows in turns of GROUPED_TURN, N a multiple of 128,
+    out bfloat16 [tiles * 128, N / 2]; limit: of CLAMPED_GATED)."""
     _need_cuda(x, w, out, tile_expert)
     lib = load_module("gemm_grouped")
     experts, n, k = w.shape
     tiles = tile_expert.numel()
     assert x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and x.is_contiguous() and w.is_contiguous()
-    assert x.shape == (tiles * GROUPED_ROWS, k) and out.shape == (tiles * GROUPED_ROWS, n) and out.stride(1) == 1
+    columns = n // 2 if activation in GATED else n
+    assert x.shape == (tiles * GROUPED_ROWS, k) and out.shape == (tiles * GROUPED_ROWS, columns) and out.stride(1) == 1
     assert out.dtype in (torch.bfloat16, torch.float32)
     _check(lib, lib.abk_gemm_grouped(_p(x), _p(w), _p(out), _ll(out.stride(0)), _i(1 if out.dtype == torch.float32 else 0),
-                                     _i(activation), _i(tiles), _i(experts), _i(n), _i(k), _p(tile_expert),
+                                     _i(activation), _i(tiles), _i(experts), _i(n), _i(k), _p(tile_expert), _f(limit),
                                      _p(kernel_status(x.device)), _stream()), "gemm_grouped")
 
 

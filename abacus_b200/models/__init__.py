@@ -1,4 +1,4 @@
-from . import lilovik, linonex, movarax, qwen3, temetar, tilulorn  # noqa: F401  (register Qwen3ForCausalLM, Temetar, Movarax, Linonex, Tilulorn and Lilovik)
+from . import kimilix, lilovik, linonex, movarax, qwen3, temetar, tilulorn  # noqa: F401  (register Qwen3ForCausalLM, Temetar, Movarax, Linonex, Tilulorn, Lilovik and Kimilix)
 from .layout import ModelLayout
 from .model import Model, expected_tensors
 

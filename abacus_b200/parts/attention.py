@@ -9,7 +9,9 @@ kept behind a window, a sink, float32 weights, a short causal convolution over t
 right after their projection (its last inputs are part of the sequence's state, beside the keys and values), keys
 seen only within the token's own chunk of positions, and capped scores. A layer may do without a softmax altogether
 (weights "sigmoid": each key for itself, with a distance bias and a shift per head, the heads' weights mixed before
-they meet the values): the projection, its preparation and the cache are the same, the attention kernels its own.
+they meet the values): the projection, its preparation and the cache are the same, the attention kernels its own. Or it is
+differential (diff): every head has two maps over the same values. q and k then have twice the heads of head_dim for norm
+and rotation, a key row of the cache holds both maps side by side, and the attention kernels make one head of the two.
 """
 import os
 
@@ -64,7 +66,11 @@ class Attention:
             raise ValueError("slopes, a shift per head and mixed heads go with sigmoid weights")
         if s.slopes is not None and len(s.slopes) != s.n_heads:
             raise ValueError(f"{len(s.slopes)} slopes for {s.n_heads} heads")
-        self.general = (self.v_dim != s.head_dim or bool(s.keep_first) or s.sink or s.exact_weights or s.conv_taps > 0
+        self.maps = 1 if s.diff is None else 2
+        if s.diff is not None and (self.whole or self.sigmoid or s.head_gate or s.keep_first or s.conv_taps or not s.exact_weights):
+            raise ValueError("differential attention has softmax weights in float32 and a norm per head, and takes no gate, kept first "
+                             "keys, convolution, biases or values that are its keys")
+        self.general = (self.maps > 1 or self.v_dim != s.head_dim or bool(s.keep_first) or s.sink or s.exact_weights or s.conv_taps > 0
                         or bool(s.chunk) or bool(s.softcap) or self.whole or s.head_gate or self.sigmoid)
         if s.conv_taps < 0 or s.conv_taps > 8:
             raise ValueError(f"conv_taps {s.conv_taps}: the convolution takes 1 to 8 taps")
@@ -77,7 +83,7 @@ class Attention:
                              "kernel, which a layer with a sink, kept first keys or values of their own size runs on, "
                              "any size up to 256)")
         self.position = POSITIONS.build(s.position) if s.position is not None else None
-        self.q_size, self.kv_size = s.n_heads * s.head_dim, s.n_kv_heads * s.head_dim
+        self.q_size, self.kv_size = s.n_heads * self.maps * s.head_dim, s.n_kv_heads * self.maps * s.head_dim
         self.v_size = s.n_kv_heads * self.v_dim
         # a row of q, k and v is padded to a multiple of 8 elements, so that every row starts 16-byte aligned whatever
         # the values' size (nothing to pad where values are as large as keys: head_dim is a multiple of 8)
@@ -96,7 +102,7 @@ class Attention:
 
     def step_plans(self):
         """What this mixer wants made on the host for every step and sent with the step's indices."""
-        return [] if self.sigmoid else [self.lists]  # (attention without a softmax needs none)
+        return [] if self.sigmoid or self.maps > 1 else [self.lists]  # (attention without a softmax and differential attention need none)
 
     def step_weights(self):
         """The tensors a step reads once whatever its size (for the bytes a decode step must move)."""
@@ -115,7 +121,9 @@ class Attention:
         elif s.qk_norm_eps is not None:
             shapes.update(q_norm=(s.head_dim,), k_norm=(s.head_dim,))
         if s.sink:
-            shapes["sink"] = (s.n_heads,)
+            shapes["sink"] = (s.n_heads * self.maps,)
+        if s.diff is not None:
+            shapes.update({n: (s.head_dim,) for n in ("lq1", "lk1", "lq2", "lk2")})
         if s.bias:
             shapes.update(bq=(self.q_size,), bk=(self.kv_size,), bv=(self.v_size,))
         if s.shift:
@@ -146,6 +154,10 @@ class Attention:
         self.mix = to_device(params["mix"], ctx, torch.float32) if self.spec.mix else None
         self.slopes = (torch.tensor(self.spec.slopes, dtype=torch.float64).to(torch.float32).to(ctx.device)
                        if self.spec.slopes is not None else None)
+        self.lam = None
+        if self.spec.diff is not None:  # the second map's factor, one number a layer
+            l = {n: params[n].detach().to("cpu", torch.float64) for n in ("lq1", "lk1", "lq2", "lk2")}
+            self.lam = float(torch.exp((l["lq1"] * l["lk1"]).sum()) - torch.exp((l["lq2"] * l["lk2"]).sum())) + self.spec.diff
         self.conv = None
         if self.spec.conv_taps:  # one table for the whole row of q, k and v; the row's padding has taps of zero
             taps = torch.cat([params["conv_q"], params["conv_k"], params["conv_v"]], dim=0).to(torch.float32)
@@ -156,7 +168,7 @@ class Attention:
     def cache_need(self):
         s = self.spec
         states = (("conv_tail", (s.conv_taps - 1, self.row), "float32"),) if s.conv_taps > 1 else ()
-        return CacheNeed(n_kv_heads=s.n_kv_heads, head_dim=s.head_dim, window=s.window, v_head_dim=self.v_dim,
+        return CacheNeed(n_kv_heads=s.n_kv_heads, head_dim=self.maps * s.head_dim, window=s.window, v_head_dim=self.v_dim,
                          keep_first=s.keep_first if s.window is not None else 0, states=states)
 
     def prepare(self, max_positions, device):
@@ -221,15 +233,21 @@ class Attention:
                                                   self.k_norm, self.cos, self.sin, rotary_dim, interleaved)):
             prepare = dict(q_norm=self.q_norm, k_norm=self.k_norm, eps=s.qk_norm_eps, cos=self.cos, sin=self.sin, keep=writes)
         else:
-            ops.qkv_prep(qkv, s.n_heads, s.n_kv_heads, s.head_dim, batch, self.q_norm, self.k_norm, s.qk_norm_eps,
+            ops.qkv_prep(qkv, self.maps * s.n_heads, self.maps * s.n_kv_heads, s.head_dim, batch, self.q_norm, self.k_norm, s.qk_norm_eps,
                          self.cos, self.sin, rotary_dim, interleaved, cache.kv if writes else None, q_only=not writes,
-                         v_dim=self.v_dim, row=self.row if self.general else None)
+                         v_dim=self.v_dim, row=self.row if self.general else None, maps=self.maps)
         if from_step and (batch.any_continuation or not writes):
             raise ops.KernelRefused("windowed attention takes several tokens of a sequence only at its start, "
                                     "and only with keys of its own")
         if self.sigmoid:
             ops.attention_sigmoid(qkv, att, s.n_heads, s.n_kv_heads, s.head_dim, s.scale, batch, cache.kv, v_dim=self.v_dim,
                                   softcap=s.softcap, slopes=self.slopes, shift=self.shift, mix=self.mix, row=self.row, ws=ws)
+            self.o_proj.forward(att, out, n)
+            return out
+        if self.maps > 1:
+            ops.attention_differential(qkv, att, s.n_heads, s.n_kv_heads, s.head_dim, s.scale, s.window, batch, cache.kv, self.lam,
+                                       s.diff_eps, 1.0 - s.diff, from_step=from_step, ws=ws, v_dim=self.v_dim, sink=self.sink,
+                                       row=self.row, chunk=s.chunk, softcap=s.softcap)
             self.o_proj.forward(att, out, n)
             return out
         mine = batch.plan.get(self.lists.name)

@@ -247,8 +247,37 @@ class LoopInputFrame:
         return out
 
 
+class NormedEndFrame(PlainFrame):
+    """The plain frame of blocks that hand on a branch's output with its norm (parts/block.py: sandwich_norm, post_norm): the
+    pending branch with its norm, the last norm, the output matrix on the wanted rows."""
+
+    def __init__(self, spec):
+        super().__init__(spec)
+        self.options = spec.frame_spec
+
+    def logits(self, x, pending, batch, ws):
+        r = batch.n_logit_rows
+        out = ws.get("logits", (max(r, 1), self.vocab), torch.float32)[:r]
+        if r:
+            xn = ws.get("xn_final", (r, self.hidden), self.ctx.dtype)
+            self.final_norm.forward_normed(x, pending, xn, rows=batch.logit_rows, n_rows=r)
+            self.head.forward(xn, out, r)
+        return out
+
+
+@FRAMES.register("scaled")
+class ScaledFrame(NormedEndFrame):
+    """x = table[token] * scale (config.specs.ScaledEmbeddingSpec); a tied output matrix is the table without its scale."""
+
+    def embed(self, batch, ws, status):
+        n = batch.n_rows
+        x = ws.get("x", (n, self.hidden), torch.float32)
+        ops.embed_pairs(batch, self.table, None, None, x.view(n, 1, self.hidden), self.options.scale, 0, 0, 0, status)
+        return x
+
+
 @FRAMES.register("sinusoids")
-class SinusoidsFrame(PlainFrame):
+class SinusoidsFrame(NormedEndFrame):
     """x = table[token] + a fixed sinusoid per position (config.specs.SinusoidEmbeddingSpec, parts/position.py); the stream
     is one row per token. The end: the pending branch with its norm (parts/block.py, sandwich_norm), the last norm, the
     output matrix on the wanted rows, the logits times logit_scale (which is in the last norm's weight, so it costs nothing
@@ -256,7 +285,6 @@ class SinusoidsFrame(PlainFrame):
 
     def __init__(self, spec):
         super().__init__(spec)
-        self.options = spec.frame_spec
         self.sinusoids = Sinusoids(spec.hidden, self.options.base)
         self.coarse = self.fine = None
 
@@ -272,12 +300,3 @@ class SinusoidsFrame(PlainFrame):
         x = ws.get("x", (batch.n_rows, self.hidden), torch.float32)
         ops.embed_sinusoids(batch, self.table, self.coarse, self.fine, self.n_positions, x, status)
         return x
-
-    def logits(self, x, pending, batch, ws):
-        r = batch.n_logit_rows
-        out = ws.get("logits", (max(r, 1), self.vocab), torch.float32)[:r]
-        if r:
-            xn = ws.get("xn_final", (r, self.hidden), self.ctx.dtype)
-            self.final_norm.forward_normed(x, pending, xn, rows=batch.logit_rows, n_rows=r)
-            self.head.forward(xn, out, r)
-        return out

@@ -12,6 +12,9 @@ Per token the cache holds [c | r]: c, the normed down-projection (rank elements)
       latents by one product, the shared part copied behind each head's keys, and the prompt kernels for ordinary heads
       run on them.
 
+With a window the cache keeps a ring of pages; a step of several tokens then has its sequences start at their first token
+and reads the latents it needs from the step's own rows.
+
 Scores, softmax weights, the norm of the latent and the rotation are float32 in both number formats.
 """
 import torch
@@ -53,6 +56,8 @@ class LatentAttention:
         self.gate_at = self.q_latent_at + self.q_rank8
         self.proj_width = self.gate_at + (_up8(s.n_heads) if s.head_gate else 0)
         self.cos = self.sin = None
+        if s.window is not None and (s.window < 1 or s.shares_latents):
+            raise ValueError(f"window {s.window}: a windowed layer sees at least its own token and has latents of its own")
         if self.row > 640:
             raise ValueError(f"rank {s.rank} + rot_dim {s.rot_dim}: the attention kernels take rows of up to 640")
 
@@ -109,7 +114,7 @@ class LatentAttention:
 
     def cache_need(self):
         s = self.spec
-        return CacheNeed(n_kv_heads=1, head_dim=self.row, v_head_dim=s.rank, values_in_keys=True)
+        return CacheNeed(n_kv_heads=1, head_dim=self.row, v_head_dim=s.rank, values_in_keys=True, window=s.window)
 
     def prepare(self, max_positions, device):
         if self.position is not None:
@@ -141,26 +146,34 @@ class LatentAttention:
         att = ws.get("att", (n, s.n_heads * s.v_head_dim), dt)
         kv = cache.kv
         gated = False
+        if s.window is not None and not batch.is_decode and batch.any_continuation:
+            raise ops.KernelRefused("windowed latent attention takes several tokens of a sequence only at its start")
+        own = None  # the step's own latent rows, where a prompt reads them (else they are the cache's)
+        if cache.owns_storage and not batch.is_decode and (s.window is not None or self.full_size_takes(batch)):
+            own = ws.get("latent_rows", (n, self.row), dt)
         if self.full_size_takes(batch):
             heads_size = 2 * self.q_size + s.n_heads * s.v_head_dim
             qkv = ws.get("latent_qkv", (n, _up8(heads_size)), dt)
             ops.latent_prep(proj, self.down_at, s.n_heads, s.head_dim, s.rot_dim, s.rank, rot_dims, self.down_norm,
                             s.norm_eps, self.cos, self.sin, qkv, self.per_head, s.head_dim, True,
-                            kv if cache.owns_storage else None, batch, interleaved=self.interleaved)
-            rows = ws.get("latent_rows", (n, self.row), dt)
-            ops.latent_rows(kv, rows, self.row, batch)
+                            kv if cache.owns_storage else None, batch, interleaved=self.interleaved, rows=own)
+            rows = own
+            if rows is None:
+                rows = ws.get("latent_rows", (n, self.row), dt)
+                ops.latent_rows(kv, rows, self.row, batch)
             self.up_full.forward(rows[:, :_up8(s.rank)], qkv[:, self.q_size:heads_size], n)
             ops.spread_shared(rows[:, s.rank:], qkv[:, self.q_size:], self.per_head, s.head_dim, s.rot_dim, s.n_heads, n)
-            ops.attention(qkv, att, s.n_heads, s.n_heads, self.per_head, s.scale, None, batch, None, from_step=True, ws=ws,
+            ops.attention(qkv, att, s.n_heads, s.n_heads, self.per_head, s.scale, s.window, batch, None, from_step=True, ws=ws,
                           v_dim=s.v_head_dim, sink=self.sink, exact_weights=True, row=qkv.shape[1])
         else:
             q_lat = ws.get("latent_q", (n, s.n_heads * self.row), dt)
             ops.latent_prep(proj, self.down_at, s.n_heads, s.head_dim, s.rot_dim, s.rank, rot_dims, self.down_norm,
                             s.norm_eps, self.cos, self.sin, q_lat, self.row, s.rank, False,
-                            kv if cache.owns_storage else None, batch, interleaved=self.interleaved)
+                            kv if cache.owns_storage else None, batch, interleaved=self.interleaved, rows=own)
             ops.head_product(proj, self.per_head, self.uk_t, q_lat, self.row, n)
             mixed = ws.get("latent_mixed", (n, s.n_heads * s.rank), dt)
-            ops.attention_values_in_keys(q_lat, mixed, s.n_heads, self.row, s.rank, s.scale, batch, kv, self.sink, ws)
+            ops.attention_values_in_keys(q_lat, mixed, s.n_heads, self.row, s.rank, s.scale, batch, kv, self.sink, ws,
+                                         window=s.window, rows=own)
             # (head h's output times sigmoid(g_h . x) where the values leave the latent space)
             ops.head_product(mixed, s.rank, self.uv, att, s.v_head_dim, n, gate=proj[:, self.gate_at:] if s.head_gate else None)
             gated = True

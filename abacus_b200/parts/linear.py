@@ -35,13 +35,16 @@ class Linear:
         self.weight = weight
         self.out_features, self.in_features = weight.shape
 
-    def forward(self, x, out, m=None):
+    def forward(self, x, out, m=None, activation=None):
+        """out[:m] = act(x[:m] . W^T); activation (ops.OUT_ACTIVATIONS): in the product's epilogue where it has one."""
         rows = x.shape[0] if m is None else m
         if (self.weight.dtype == torch.bfloat16 and rows_kernel_wins(rows, self.weight)
                 and ops.gemm_rows_takes(x, self.weight, out, rows)):
-            ops.gemm_rows(x, self.weight, out, rows)
+            ops.gemm_rows(x, self.weight, out, rows, activation=activation)
         elif self.weight.dtype == torch.bfloat16 and ops.gemm_tc_takes(x, self.weight, out):
-            ops.gemm_tc(x, self.weight, out, m)
+            ops.gemm_tc(x, self.weight, out, m, activation=activation)
         else:
             ops.gemm_simt(x, self.weight, out, m)
+            if activation == "relu_squared":
+                ops.relu_squared(out, rows)
         return out

@@ -21,8 +21,11 @@ class Rotary:
             raise ValueError(f"rotary pairing {spec.pairing!r} is neither half nor interleaved")
         if spec.rotary_dim < 2 or spec.rotary_dim % 2:
             raise ValueError(f"rotary_dim {spec.rotary_dim} must be even")
-        if (getattr(spec, "linear_factor", 1.0) != 1.0 or getattr(spec, "blend", None)) and not spec.exact_angles:
+        scalings = (getattr(spec, "linear_factor", 1.0) != 1.0, bool(getattr(spec, "blend", None)), bool(getattr(spec, "bands", None)))
+        if any(scalings) and not spec.exact_angles:
             raise ValueError("scaled frequencies are made with exact_angles")
+        if scalings[2] and (scalings[1] or not spec.bands[3] > spec.bands[2]):
+            raise ValueError("frequencies are scaled in bands or blended, not both, and the bands' high is above their low")
         self.spec = spec
         self.rotary_dim = spec.rotary_dim
         self.interleaved = spec.pairing == "interleaved"
@@ -33,7 +36,13 @@ class Rotary:
         s, dims = self.spec, self.rotary_dim
         i = np.arange(dims // 2, dtype=np.float64)
         freq = np.power(float(s.theta), -2.0 * i / dims) / float(getattr(s, "linear_factor", 1.0))
-        blend = getattr(s, "blend", None)
+        blend, bands = getattr(s, "blend", None), getattr(s, "bands", None)
+        if bands is not None:
+            factor, original, low, high = (float(v) for v in bands)
+            turns = original * freq / (2.0 * math.pi)  # a pair's turns over the original context
+            share = (turns - low) / (high - low)
+            between = (1.0 - share) * freq / factor + share * freq
+            return np.where(turns > high, freq, np.where(turns < low, freq / factor, between)), 1.0
         if blend is None:
             return freq, 1.0
         factor, original, fast, slow = (float(v) for v in blend)
