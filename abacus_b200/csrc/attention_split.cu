@@ -17,6 +17,7 @@
 #define ABK_DEFINE_ERROR
 #include "common.cuh"
 #include "differential.cuh"
+#include "mma_tiles.cuh"
 
 #define AS_THREADS 128
 #define AS_MAX_GROUP 16
@@ -38,7 +39,7 @@ struct AttnSplit {
     const int *token_seq, *token_pos, *seq_slot;
     const void *k_pool, *v_pool;
     PagedCache cache, v_cache;
-    int n_parts;
+    int n_parts, part_keys;  // a row's parts have part_keys keys each (128, or 64 in the kernel for latent rows)
     int values_in_keys;  // a value is the first v_dim elements of its key row (one pool)
     int runs;            // runs of query heads, a CTA each, that share a kv head of the cache; n_kv_heads counts the runs
     const void *gate;    // null, or a gate per token and head (of q's type, at gate + t * ldg + h): the head's output is
@@ -91,10 +92,6 @@ template <> __device__ __forceinline__ float dot_q<__nv_bfloat16>(const float *q
 // reading its own row meets no bank conflict), and once the scores are made the 128 value rows into the same memory,
 // under the softmax; else each thread reads global memory.
 // GMAX: the group's size rounded up to 1, 2, 4, 8 or 16 (what the loops over its heads are unrolled to).
-__device__ __forceinline__ void as_mma_bf16(float *c, uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
-    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
-                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
-}
 // A float32 number as three bfloat16 numbers that add up to it (its 24 bits), each pair packed for one operand register.
 __device__ __forceinline__ void as_split3(float x, float y, uint32_t &hi, uint32_t &mid, uint32_t &lo) {
     const __nv_bfloat16 xh = __float2bfloat16_rn(x), yh = __float2bfloat16_rn(y);
@@ -106,12 +103,7 @@ __device__ __forceinline__ void as_split3(float x, float y, uint32_t &hi, uint32
     lo = (uint32_t)__bfloat16_as_ushort(xl) | ((uint32_t)__bfloat16_as_ushort(yl) << 16);
 }
 
-// TC (bfloat16, STAGED, keys that carry their values, head_dim a multiple of 16, values a multiple of 8 up to 256): both
-// products on the warp-level tensor cores, the group's heads as the 16 rows of a tile. Scores: q from global memory
-// as the row operand, the staged key rows as the column operand, float32 sums. Weighted values: the float32 weights
-// as three bfloat16 parts that hold their 24 bits, each multiplied with the same value fragment, so that the weights
-// stay float32 in effect.
-template <typename T, bool STAGED, int GMAX, bool TC = false> __global__ void __launch_bounds__(AS_THREADS) attention_split_kernel(AttnSplit p) {
+template <typename T, bool STAGED, int GMAX> __global__ void __launch_bounds__(AS_THREADS) attention_split_kernel(AttnSplit p) {
     extern __shared__ __align__(16) float as_smem[];
     const int group = p.n_heads / p.n_kv_heads, hd = p.head_dim, vd = p.v_dim, kd = p.maps * hd;  // kd: a key row
     float *q_s = as_smem;                      // [group][hd]
@@ -122,14 +114,16 @@ template <typename T, bool STAGED, int GMAX, bool TC = false> __global__ void __
     uint8_t *v_s = k_s;                                        // [128][vd], once the keys are done with
     __shared__ long long k_off[AS_THREADS], v_off[AS_THREADS];
     const int t = blockIdx.x, kvh = blockIdx.y, part = blockIdx.z, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    pdl_wait();
+    // the step's indices and the page table were written by kernels further back than the one just before
     const int seq = p.token_seq[t];
-    if (seq < 0) return;
-    const int pos = p.token_pos[t], slot = p.seq_slot[seq];
-    int lo, kept, total;
-    visible_keys(p, pos, lo, kept, total);
-    if (part * AS_THREADS >= total) return;  // the fold knows how many parts a row has
-    const int n_valid = total - part * AS_THREADS < AS_THREADS ? total - part * AS_THREADS : AS_THREADS;
+    const int pos = p.token_pos[t];
+    int lo = 0, kept = 0, total = 0;
+    if (seq >= 0) visible_keys(p, pos, lo, kept, total);
+    if (part * AS_THREADS >= total) {  // (the fold knows how many parts a row has)
+        pdl_wait();
+        return;
+    }
+    const int slot = p.seq_slot[seq], n_valid = total - part * AS_THREADS < AS_THREADS ? total - part * AS_THREADS : AS_THREADS;
     const int number = part * AS_THREADS + tid;
     const bool valid = number < total;
     if (valid) {
@@ -139,6 +133,7 @@ template <typename T, bool STAGED, int GMAX, bool TC = false> __global__ void __
         v_off[tid] = cache_offset(p.v_cache, page, ckv, cn, j, p.values_in_keys ? kd : vd);
         k_off[tid] = cache_offset(p.cache, page, ckv, cn, j, kd);
     }
+    pdl_wait();
     const T *q = (const T *)p.q + (long long)t * p.q_row + (long long)kvh * group * hd;
     for (int e = tid; e < group * hd; e += AS_THREADS) q_s[e] = to_float(q[e]);
     __syncthreads();
@@ -155,36 +150,7 @@ template <typename T, bool STAGED, int GMAX, bool TC = false> __global__ void __
         __syncthreads();
     }
     float sc[GMAX];
-    if (TC) {
-        const int row = lane >> 2, k0 = (lane & 3) * 2;
-        const __nv_bfloat16 *qg = (const __nv_bfloat16 *)p.q + (long long)t * p.q_row + (long long)kvh * group * hd;
-        const bool lower = row < group, upper = row + 8 < group;
-        float acc[4][4];
-#pragma unroll
-        for (int nt = 0; nt < 4; nt++) acc[nt][0] = acc[nt][1] = acc[nt][2] = acc[nt][3] = 0.0f;
-        for (int kk = 0; kk < hd; kk += 16) {
-            const uint32_t a0 = lower ? *(const uint32_t *)(qg + (long long)row * hd + kk + k0) : 0u;
-            const uint32_t a1 = upper ? *(const uint32_t *)(qg + (long long)(row + 8) * hd + kk + k0) : 0u;
-            const uint32_t a2 = lower ? *(const uint32_t *)(qg + (long long)row * hd + kk + k0 + 8) : 0u;
-            const uint32_t a3 = upper ? *(const uint32_t *)(qg + (long long)(row + 8) * hd + kk + k0 + 8) : 0u;
-#pragma unroll
-            for (int nt = 0; nt < 4; nt++) {
-                const uint8_t *kr = k_s + (warp * 32 + nt * 8 + row) * k_pitch + (kk + k0) * 2;
-                as_mma_bf16(acc[nt], a0, a1, a2, a3, *(const uint32_t *)kr, *(const uint32_t *)(kr + 16));
-            }
-        }
-        // the scores to where the weights will stand, [head][key]; every thread then takes its own key's
-#pragma unroll
-        for (int nt = 0; nt < 4; nt++) {
-            const int key = warp * 32 + nt * 8 + k0;
-            if (lower) p_s[row * AS_THREADS + key] = score_of(p, acc[nt][0]), p_s[row * AS_THREADS + key + 1] = score_of(p, acc[nt][1]);
-            if (upper) p_s[(row + 8) * AS_THREADS + key] = score_of(p, acc[nt][2]), p_s[(row + 8) * AS_THREADS + key + 1] = score_of(p, acc[nt][3]);
-        }
-        __syncthreads();
-#pragma unroll
-        for (int g = 0; g < GMAX; g++)
-            if (g < group) sc[g] = valid ? p_s[g * AS_THREADS + tid] : -INFINITY;
-    } else if (valid) {
+    if (valid) {
         const T *k = STAGED ? (const T *)(k_s + tid * k_pitch) : (const T *)p.k_pool + k_off[tid];
 #pragma unroll
         for (int g = 0; g < GMAX; g++)
@@ -231,62 +197,6 @@ template <typename T, bool STAGED, int GMAX, bool TC = false> __global__ void __
     }
     if (STAGED && !p.values_in_keys) asm volatile("cp.async.wait_group 0;" ::: "memory");  // the values are here
     __syncthreads();
-    if (TC) {
-        // out[head][column] = sum over the part's keys of weight[head][key] * value[key][column]: a warp has every fourth
-        // tile of 8 columns; a key step's weights are split once and meet all of the warp's tiles
-        const int row = lane >> 2, k0 = (lane & 3) * 2;
-        const bool lower = row < group, upper = row + 8 < group;
-        const int n_tiles = vd / 8;
-        float c[8][4];
-#pragma unroll
-        for (int i = 0; i < 8; i++) c[i][0] = c[i][1] = c[i][2] = c[i][3] = 0.0f;
-        for (int ks = 0; ks < AS_THREADS; ks += 16) {
-            if (ks >= n_valid) break;
-            uint32_t ah[4], am[4], al[4];
-            const float *pl = p_s + row * AS_THREADS + ks + k0, *pu = p_s + (row + 8) * AS_THREADS + ks + k0;
-            as_split3(lower ? pl[0] : 0.0f, lower ? pl[1] : 0.0f, ah[0], am[0], al[0]);
-            as_split3(upper ? pu[0] : 0.0f, upper ? pu[1] : 0.0f, ah[1], am[1], al[1]);
-            as_split3(lower ? pl[8] : 0.0f, lower ? pl[9] : 0.0f, ah[2], am[2], al[2]);
-            as_split3(upper ? pu[8] : 0.0f, upper ? pu[9] : 0.0f, ah[3], am[3], al[3]);
-            // keys beyond the part's last hold whatever the memory held: their values are taken as zeros
-            const bool in0 = ks + k0 < n_valid, in1 = ks + k0 + 1 < n_valid, in8 = ks + k0 + 8 < n_valid, in9 = ks + k0 + 9 < n_valid;
-            const uint8_t *vr = k_s + (ks + k0) * k_pitch + row * 2;
-#pragma unroll
-            for (int i = 0; i < 8; i++) {
-                const int nt = warp + 4 * i;
-                if (nt >= n_tiles) break;
-                const uint8_t *v = vr + nt * 16;
-                const uint32_t v0 = in0 ? *(const uint16_t *)v : 0u, v1 = in1 ? *(const uint16_t *)(v + k_pitch) : 0u;
-                const uint32_t v8 = in8 ? *(const uint16_t *)(v + 8 * k_pitch) : 0u, v9 = in9 ? *(const uint16_t *)(v + 9 * k_pitch) : 0u;
-                const uint32_t b0 = v0 | (v1 << 16), b1 = v8 | (v9 << 16);
-                as_mma_bf16(c[i], ah[0], ah[1], ah[2], ah[3], b0, b1);
-                as_mma_bf16(c[i], am[0], am[1], am[2], am[3], b0, b1);
-                as_mma_bf16(c[i], al[0], al[1], al[2], al[3], b0, b1);
-            }
-        }
-#pragma unroll
-        for (int i = 0; i < 8; i++) {
-            const int nt = warp + 4 * i;
-            if (nt >= n_tiles) break;
-            const int col = nt * 8 + k0;
-            if (lower) {
-                float *dst = p.parts + (((long long)t * p.n_heads + kvh * group + row) * p.n_parts + part) * (vd + 2);
-                dst[col] = c[i][0], dst[col + 1] = c[i][1];
-            }
-            if (upper) {
-                float *dst = p.parts + (((long long)t * p.n_heads + kvh * group + row + 8) * p.n_parts + part) * (vd + 2);
-                dst[col] = c[i][2], dst[col + 1] = c[i][3];
-            }
-        }
-        if (tid < group) {
-            float *dst = p.parts + (((long long)t * p.n_heads + kvh * group + tid) * p.n_parts + part) * (vd + 2);
-#pragma unroll
-            for (int g = 0; g < GMAX; g++)
-                if (g == tid) dst[vd] = top[g];
-            dst[vd + 1] = (red[tid] + red[group + tid]) + (red[2 * group + tid] + red[3 * group + tid]);
-        }
-        return;
-    }
     // weighted values: a thread a value column (two for values beyond 128), every head of the group per value read
     float acc0[GMAX], acc1[GMAX];
 #pragma unroll
@@ -322,6 +232,273 @@ template <typename T, bool STAGED, int GMAX, bool TC = false> __global__ void __
     }
 }
 
+// The same for bfloat16 keys that carry their values (latent rows: one kv head, head_dim a multiple of 16, values a multiple of
+// 8 up to 256), both products on the warp-level tensor cores with the group's heads as the 16 rows of a tile. A CTA takes
+// PART keys; they and the queries come into shared memory by cp.async, zeros in the places of keys and heads there are none
+// of. A warp makes the scores of PART / 4 keys and has them in registers: maxima and sums meet over the warps through
+// shared memory. The weighted values: the float32 weights as three bfloat16 parts that hold their 24 bits, each multiplied
+// with the same value fragments, so that the weights stay float32 in effect.
+template <int PART> __global__ void __launch_bounds__(AS_THREADS) attention_split_latent_kernel(AttnSplit p) {
+    extern __shared__ __align__(16) float as_smem[];
+    constexpr int KEYS = PART / 4, NT = KEYS / 8, P_PITCH = PART + 8;  // a warp's keys, its tiles of 8
+    const int group = p.n_heads / p.n_kv_heads, hd = p.head_dim, vd = p.v_dim, pitch = hd * 2 + 16;
+    float *p_s = as_smem;                           // [16][P_PITCH] weights
+    float *red = p_s + 16 * P_PITCH;                // [2][4][16] the warps' maxima, then their sums
+    uint8_t *q_s = (uint8_t *)(red + 128);          // [16][pitch]
+    uint8_t *k_s = q_s + 16 * pitch;                // [PART][pitch]
+    __shared__ long long k_off[PART];
+    const int t = blockIdx.x, run = blockIdx.y, part = blockIdx.z, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int g = lane >> 2, c2 = (lane & 3) * 2;
+    // the step's indices, the page table and the keys of earlier steps were written by kernels further back than the one just
+    // before (which makes the queries and the token's own key): they are read before the wait
+    const int seq = p.token_seq[t];
+    const int pos = p.token_pos[t];
+    int lo = 0, kept = 0, total = 0;
+    if (seq >= 0) visible_keys(p, pos, lo, kept, total);
+    if (part * PART >= total) {  // (the fold knows how many parts a row has)
+        pdl_wait();
+        return;
+    }
+    const int slot = p.seq_slot[seq], n_valid = min(total - part * PART, PART);
+    if (tid < PART) {
+        const int number = part * PART + min(tid, n_valid - 1), j = number < kept ? number : lo + number - kept;
+        const int cn = p.n_kv_heads / p.runs;
+        k_off[tid] = cache_offset(p.cache, cache_page(p.cache, slot, j), run / p.runs, cn, j, hd);
+    }
+    const uint32_t q_at = (uint32_t)__cvta_generic_to_shared(q_s), k_at = (uint32_t)__cvta_generic_to_shared(k_s);
+    const int chunks = hd / 8;
+    const __nv_bfloat16 *q = (const __nv_bfloat16 *)p.q + (long long)t * p.q_row + (long long)run * group * hd;
+    // where the token's own key lies among the part's (it is the last that is seen)
+    const int own = part * PART + n_valid == total ? n_valid - 1 : PART;
+    __syncthreads();
+    for (int e = tid; e < PART * chunks; e += AS_THREADS) {
+        const int r = e / chunks, c = e - r * chunks;
+        if (r == own) continue;
+        asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(k_at + r * pitch + c * 16),
+                     "l"((const __nv_bfloat16 *)p.k_pool + k_off[r] + c * 8), "r"(r < n_valid ? 16 : 0) : "memory");
+    }
+    pdl_wait();
+    if (own < PART)
+        for (int c = tid; c < chunks; c += AS_THREADS)
+            asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(k_at + own * pitch + c * 16),
+                         "l"((const __nv_bfloat16 *)p.k_pool + k_off[own] + c * 8) : "memory");
+    for (int e = tid; e < 16 * chunks; e += AS_THREADS) {
+        const int r = e / chunks, c = e - r * chunks;
+        asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(q_at + r * pitch + c * 16),
+                     "l"(q + (long long)min(r, group - 1) * hd + c * 8), "r"(r < group ? 16 : 0) : "memory");
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();
+
+    float s[NT][4];
+#pragma unroll
+    for (int nt = 0; nt < NT; nt++) s[nt][0] = s[nt][1] = s[nt][2] = s[nt][3] = 0.0f;
+    const uint32_t qa = q_at + (lane & 15) * pitch + (lane >> 4) * 16;
+    const uint32_t ka = k_at + (warp * KEYS + (lane & 7) + ((lane >> 4) << 3)) * pitch + ((lane >> 3) & 1) * 16;
+#pragma unroll 4
+    for (int kk = 0; kk < hd / 16; kk++) {
+        uint32_t a[4];
+        ldsm_x4(qa + kk * 32, a[0], a[1], a[2], a[3]);
+#pragma unroll
+        for (int tp = 0; tp < NT / 2; tp++) {
+            uint32_t b0, b1, b2, b3;
+            ldsm_x4(ka + tp * 16 * pitch + kk * 32, b0, b1, b2, b3);
+            mma_bf16(s[2 * tp], a, b0, b1);
+            mma_bf16(s[2 * tp + 1], a, b2, b3);
+        }
+    }
+    // rows g and g + 8 (heads), keys warp * KEYS + 8 nt + c2 + {0, 1}
+    float top[2] = {-INFINITY, -INFINITY}, sum[2] = {0.0f, 0.0f};
+#pragma unroll
+    for (int nt = 0; nt < NT; nt++)
+#pragma unroll
+        for (int e = 0; e < 4; e++) {
+            s[nt][e] = warp * KEYS + nt * 8 + c2 + (e & 1) < n_valid ? score_of(p, s[nt][e]) : -INFINITY;
+            top[e >> 1] = fmaxf(top[e >> 1], s[nt][e]);
+        }
+#pragma unroll
+    for (int r = 0; r < 2; r++) {
+        top[r] = quad_max(top[r]);
+        if (c2 == 0) red[warp * 16 + g + 8 * r] = top[r];
+    }
+    __syncthreads();
+#pragma unroll
+    for (int r = 0; r < 2; r++) {
+        const float *m = red + g + 8 * r;
+        top[r] = fmaxf(fmaxf(m[0], m[16]), fmaxf(m[32], m[48]));  // (the part's first key is a real one)
+    }
+#pragma unroll
+    for (int nt = 0; nt < NT; nt++) {
+#pragma unroll
+        for (int e = 0; e < 4; e++) s[nt][e] = expf(s[nt][e] - top[e >> 1]), sum[e >> 1] += s[nt][e];
+        float *w = p_s + g * P_PITCH + warp * KEYS + nt * 8 + c2;
+        *(float2 *)w = make_float2(s[nt][0], s[nt][1]);
+        *(float2 *)(w + 8 * P_PITCH) = make_float2(s[nt][2], s[nt][3]);
+    }
+#pragma unroll
+    for (int r = 0; r < 2; r++) {
+        sum[r] = quad_sum(sum[r]);
+        if (c2 == 0) red[64 + warp * 16 + g + 8 * r] = sum[r];
+    }
+    __syncthreads();
+    // out[head][column]: a warp has every fourth pair of tiles of 8 columns; a key step's weights are split once for all of them
+    float o[4][8];
+#pragma unroll
+    for (int i = 0; i < 4; i++)
+#pragma unroll
+        for (int e = 0; e < 8; e++) o[i][e] = 0.0f;
+    const int n_pairs = (vd + 15) / 16;
+    const uint32_t va = k_at + ((lane & 7) + ((lane >> 3) & 1) * 8) * pitch + (lane >> 4) * 16;
+#pragma unroll
+    for (int ks = 0; ks < PART / 16; ks++) {
+        if (ks * 16 >= n_valid) break;
+        uint32_t hi[4], mid[4], low[4];
+#pragma unroll
+        for (int f = 0; f < 4; f++) {  // fragment register f: rows g + 8 (f & 1), keys 16 ks + 8 (f >> 1) + c2
+            const float2 w = *(const float2 *)(p_s + (g + 8 * (f & 1)) * P_PITCH + ks * 16 + 8 * (f >> 1) + c2);
+            as_split3(w.x, w.y, hi[f], mid[f], low[f]);
+        }
+#pragma unroll
+        for (int i = 0; i < 4; i++) {
+            const int pair = warp + 4 * i;
+            if (pair >= n_pairs) break;
+            uint32_t b0, b1, b2, b3;
+            ldsm_x4_t(va + ks * 16 * pitch + pair * 32, b0, b1, b2, b3);
+            mma_bf16(o[i], hi, b0, b1), mma_bf16(o[i] + 4, hi, b2, b3);
+            mma_bf16(o[i], mid, b0, b1), mma_bf16(o[i] + 4, mid, b2, b3);
+            mma_bf16(o[i], low, b0, b1), mma_bf16(o[i] + 4, low, b2, b3);
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < 4; i++) {
+        const int pair = warp + 4 * i;
+        if (pair >= n_pairs) break;
+#pragma unroll
+        for (int r = 0; r < 2; r++) {
+            if (g + 8 * r >= group) continue;
+            float *dst = p.parts + (((long long)t * p.n_heads + run * group + g + 8 * r) * p.n_parts + part) * (vd + 2) + pair * 16 + c2;
+            *(float2 *)dst = make_float2(o[i][2 * r], o[i][2 * r + 1]);
+            if (pair * 16 + 8 < vd) *(float2 *)(dst + 8) = make_float2(o[i][4 + 2 * r], o[i][4 + 2 * r + 1]);
+        }
+    }
+    if (tid < group) {
+        float *dst = p.parts + (((long long)t * p.n_heads + run * group + tid) * p.n_parts + part) * (vd + 2);
+        const float *m = red + tid;
+        dst[vd] = fmaxf(fmaxf(m[0], m[16]), fmaxf(m[32], m[48]));
+        dst[vd + 1] = (m[64] + m[80]) + (m[96] + m[112]);
+    }
+}
+
+// Folds a row's parts over latents and carries the heads' results out of the latent space in one kernel:
+//   out[t, h, :] = W[h] (sum over the parts of their weighted latents, over the sum of their sums) (times a gate per head).
+// A CTA has 32 output features of one head for up to 8 rows: its weights are asked for before the wait, a warp folds one
+// row (lanes along the latent's columns, two a lane) and leaves it in shared memory in bfloat16, and the product runs on
+// the warp-level tensor cores, two warps with 16 features each. rank a multiple of 8.
+#define AL_ROWS 8
+#define AL_THREADS (32 * AL_ROWS)
+#define AL_OUTS 32
+#define AL_TURN 8   // blocks of 32 columns whose weights a warp has in flight
+#define AL_PARTS 4  // parts whose loads a warp has in flight
+struct LatentOut {
+    const __nv_bfloat16 *w;  // [heads][outs][rank]
+    __nv_bfloat16 *out;      // row t, head h at out + t * ldo + h * outs
+    long long ldo;
+    int outs, n_rows;
+};
+__device__ __forceinline__ uint4 al_load16(const __nv_bfloat16 *p, bool ok) { return ok ? __ldg((const uint4 *)p) : make_uint4(0, 0, 0, 0); }
+
+__global__ void __launch_bounds__(AL_THREADS) latent_fold_out_kernel(AttnSplit p, LatentOut l) {
+    extern __shared__ __align__(16) uint8_t al_smem[];  // [AL_ROWS][pitch] bfloat16
+    const int rank = p.v_dim, blocks = (rank + 31) / 32, pitch = blocks * 32 + 8;
+    __nv_bfloat16 *mixed = (__nv_bfloat16 *)al_smem;
+    const int tiles = (l.outs + AL_OUTS - 1) / AL_OUTS, h = blockIdx.x / tiles, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int r = lane >> 2, c = lane & 3, o0 = blockIdx.x % tiles * AL_OUTS + warp * 16, t0 = blockIdx.y * AL_ROWS;
+    const __nv_bfloat16 *w_lo = l.w + ((long long)h * l.outs + o0 + r) * rank + 8 * c, *w_hi = w_lo + 8LL * rank;
+    const bool multiplies = warp < AL_OUTS / 16;
+    const bool has_lo = multiplies && o0 + r < l.outs, has_hi = multiplies && o0 + r + 8 < l.outs;
+    uint4 a_lo[AL_TURN], a_hi[AL_TURN];
+    auto load_weights = [&](int kb) {
+#pragma unroll
+        for (int u = 0; u < AL_TURN; u++) {
+            const bool in = kb + u < blocks && (kb + u) * 32 + 8 * c < rank;
+            a_lo[u] = al_load16(w_lo + (kb + u) * 32, in && has_lo), a_hi[u] = al_load16(w_hi + (kb + u) * 32, in && has_hi);
+        }
+    };
+    load_weights(0);
+    const float sink = p.sink ? p.sink[h] : -INFINITY;
+    const int t = t0 + warp, seq = t < l.n_rows ? p.token_seq[t] : -1, pos = seq >= 0 ? p.token_pos[t] : 0;  // (older than the kernel just before)
+    pdl_wait();
+    {
+        __nv_bfloat16 *dst = mixed + warp * pitch;
+        int lo, kept, total;
+        visible_keys(p, pos, lo, kept, total);
+        const int n = seq >= 0 ? (total + p.part_keys - 1) / p.part_keys : 0;
+        const float *src = p.parts + ((long long)t * p.n_heads + h) * p.n_parts * (rank + 2);
+        float top = sink, sum = 0.0f;
+        float2 acc[4];  // a lane's columns 2 lane + 64 u and the next (rank up to 256)
+#pragma unroll
+        for (int u = 0; u < 4; u++) acc[u] = make_float2(0.0f, 0.0f);
+        if (n > 32) {  // (up to 32 parts a lane's own maximum is the one it has below)
+            for (int k = lane; k < n; k += 32) top = fmaxf(top, src[(long long)k * (rank + 2) + rank]);
+            top = warp_max(top);
+        }
+        for (int k0 = 0; k0 < n; k0 += 32) {
+            const int left = min(32, n - k0);
+            const float2 own = lane < left ? *(const float2 *)(src + (long long)(k0 + lane) * (rank + 2) + rank) : make_float2(-INFINITY, 0.0f);
+            if (n <= 32) top = warp_max(fmaxf(top, own.x));
+            const float w = expf(own.x - top);  // (0 in lanes without a part)
+            sum = fmaf(own.y, w, sum);
+            for (int k = 0; k < left; k += AL_PARTS) {
+                float2 v[AL_PARTS][4];
+#pragma unroll
+                for (int i = 0; i < AL_PARTS; i++)
+#pragma unroll
+                    for (int u = 0; u < 4; u++)
+                        v[i][u] = k + i < left && 2 * lane + 64 * u < rank ? *(const float2 *)(src + (long long)(k0 + k + i) * (rank + 2) + 2 * lane + 64 * u)
+                                                                          : make_float2(0.0f, 0.0f);
+#pragma unroll
+                for (int i = 0; i < AL_PARTS; i++) {
+                    const float wk = __shfl_sync(0xffffffffu, w, (k + i) & 31);
+#pragma unroll
+                    for (int u = 0; u < 4; u++) acc[u].x = fmaf(v[i][u].x, wk, acc[u].x), acc[u].y = fmaf(v[i][u].y, wk, acc[u].y);
+                }
+            }
+        }
+        sum = warp_sum(sum) + (p.sink ? expf(sink - top) : 0.0f);
+        const float inv = n > 0 ? 1.0f / sum : 0.0f;
+#pragma unroll
+        for (int u = 0; u < 4; u++)
+            if (2 * lane + 64 * u < blocks * 32)
+                *(__nv_bfloat162 *)(dst + 2 * lane + 64 * u) = __floats2bfloat162_rn(acc[u].x * inv, acc[u].y * inv);
+    }
+    __syncthreads();
+    if (!multiplies) return;
+    float acc[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+    const __nv_bfloat16 *x = mixed + r * pitch + 8 * c;
+    for (int kb = 0; kb < blocks; kb += AL_TURN) {
+        if (kb) load_weights(kb);
+#pragma unroll
+        for (int u = 0; u < AL_TURN; u++) {
+            if (kb + u >= blocks) break;
+            const uint4 b = *(const uint4 *)(x + (kb + u) * 32);
+            // (16 consecutive bytes of both operands' rows: the columns sit in the product's slots in the same way)
+            const uint32_t a0[4] = {a_lo[u].x, a_hi[u].x, a_lo[u].y, a_hi[u].y}, a1[4] = {a_lo[u].z, a_hi[u].z, a_lo[u].w, a_hi[u].w};
+            mma_bf16(acc, a0, b.x, b.y);
+            mma_bf16(acc, a1, b.z, b.w);
+        }
+    }
+    // accumulator: features o0 + r and o0 + r + 8, rows 2 c and 2 c + 1
+#pragma unroll
+    for (int e = 0; e < 4; e++) {
+        const int t = t0 + 2 * c + (e & 1), o = o0 + r + 8 * (e >> 1);
+        if (t >= l.n_rows || o >= l.outs) continue;
+        float v = acc[e];
+        if (p.gate) v *= 1.0f / (1.0f + expf(-to_float(((const __nv_bfloat16 *)p.gate)[(long long)t * p.ldg + h])));
+        l.out[(long long)t * l.ldo + (long long)h * l.outs + o] = __float2bfloat16_rn(v);
+    }
+}
+
 // out[t, h] = sum over the row's parts (and the sink) of their weighted values, over the sum of their sums, all
 // against the largest maximum. One CTA per (token, head), parts in order.
 template <typename T> __global__ void __launch_bounds__(AS_THREADS) attention_fold_kernel(AttnSplit p) {
@@ -336,7 +513,7 @@ template <typename T> __global__ void __launch_bounds__(AS_THREADS) attention_fo
     }
     int lo, kept, total;
     visible_keys(p, p.token_pos[t], lo, kept, total);
-    const int n = (total + AS_THREADS - 1) / AS_THREADS;
+    const int n = (total + p.part_keys - 1) / p.part_keys;
     const float *src = p.parts + ((long long)t * p.n_heads + h) * p.n_parts * (vd + 2);
     float top = sink;
     for (int i = 0; i < n; i++) top = fmaxf(top, src[(long long)i * (vd + 2) + vd]);
@@ -358,16 +535,16 @@ template <typename T> __global__ void __launch_bounds__(AS_THREADS) attention_fo
     __shared__ float scratch[33];
     const int t = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, vd = p.v_dim, heads = p.n_heads / 2;
     const float sinks[2] = {p.sink ? p.sink[2 * h] : -INFINITY, p.sink ? p.sink[2 * h + 1] : -INFINITY};
+    const int seq = p.token_seq[t], pos = p.token_pos[t];
     pdl_wait();
     T *out = (T *)p.out + ((long long)t * heads + h) * vd;
-    const int seq = p.token_seq[t];
     if (seq < 0) {
         for (int d = tid; d < vd; d += AS_THREADS) out[d] = from_float<T>(0.0f);
         return;
     }
     int lo, kept, total;
-    visible_keys(p, p.token_pos[t], lo, kept, total);
-    const int n = (total + AS_THREADS - 1) / AS_THREADS;
+    visible_keys(p, pos, lo, kept, total);
+    const int n = (total + p.part_keys - 1) / p.part_keys;
     float a[2], b[2];
 #pragma unroll
     for (int m = 0; m < 2; m++) {
@@ -392,8 +569,9 @@ template <typename T> __global__ void __launch_bounds__(AS_THREADS) attention_fo
 }
 
 // max_keys: an upper bound of the keys any row of the step sees (its position + 1, or window + keep_first);
-// parts: float32 scratch of at least tokens * heads * ceil(max_keys / 128) * (v_dim + 2).
-static int attention_split(const DifferentialHead *diff, int values_in_keys, int chunk, float softcap, const void *q, long long q_row, void *out, int dtype, int n_tokens, int n_heads,
+// parts: float32 scratch of at least tokens * heads * ceil(max_keys / 128) * (v_dim + 2) (for keys that carry their values
+// twice that: their parts may have 64 keys). to (null: none): the fold carries the heads' results out of the latent space.
+static int attention_split(const LatentOut *to, const DifferentialHead *diff, int values_in_keys, int chunk, float softcap, const void *q, long long q_row, void *out, int dtype, int n_tokens, int n_heads,
                                    int n_kv_heads, int head_dim, int v_dim, float scale, int window, int keep_first,
                                    const float *sink, const int *token_seq, const int *token_pos, const int *seq_slot,
                                    const void *k_pool, const void *v_pool, const int *page_table, int table_width,
@@ -426,7 +604,12 @@ static int attention_split(const DifferentialHead *diff, int values_in_keys, int
     p.cache.page_table = page_table, p.cache.table_width = table_width, p.cache.ring_pages = ring_pages;
     p.cache.tokens_per_page = tokens_per_page, p.cache.pinned_pages = pinned_pages;
     p.v_cache = p.cache;
-    p.n_parts = (max_keys + AS_THREADS - 1) / AS_THREADS;
+    const bool tensor = dtype == ABK_BF16 && values_in_keys && head_dim % 16 == 0 && v_dim % 8 == 0 && q_row % 8 == 0 &&
+                        !(((uintptr_t)k_pool | (uintptr_t)q) & 15);
+    if (to && (!tensor || ((uintptr_t)to->w & 15))) ABK_REFUSE("attention_split: latents of %d in rows of %d are not what the fused fold takes", v_dim, head_dim);
+    // parts of 64 keys where parts of 128 would not fill the GPU
+    p.part_keys = tensor && (long long)n_tokens * n_kv_heads * ((max_keys + 127) / 128) < 2 * abk_sm_count() ? 64 : 128;
+    p.n_parts = (max_keys + p.part_keys - 1) / p.part_keys;
     p.values_in_keys = values_in_keys, p.runs = runs, p.gate = gate, p.ldg = ldg;
     p.maps = maps, p.diff = diff ? *diff : DifferentialHead();
     if (values_in_keys && v_dim > head_dim) ABK_REFUSE("attention_split: values of %d inside keys of %d", v_dim, head_dim);
@@ -463,10 +646,25 @@ static int attention_split(const DifferentialHead *diff, int values_in_keys, int
         else if (group <= 8) SPLIT_LAUNCH(T, STAGED, 8); \
         else SPLIT_LAUNCH(T, STAGED, 16);           \
     } while (0)
-    const bool tensor = bf && stage && values_in_keys && head_dim % 16 == 0 && v_dim % 8 == 0 && v_dim <= 256;
     if (tensor) {
-        if (group <= 8) SPLIT_LAUNCH(__nv_bfloat16, true, 8, true);
-        else SPLIT_LAUNCH(__nv_bfloat16, true, 16, true);
+        const size_t bytes = (16 * (p.part_keys + 8) + 128) * 4 + (size_t)(16 + p.part_keys) * (head_dim * 2 + 16);
+        const void *kernel = p.part_keys == 64 ? (const void *)attention_split_latent_kernel<64> : (const void *)attention_split_latent_kernel<128>;
+        if (bytes + 4096 > 48 * 1024) {
+            cudaError_t e = abk_allow_shared_memory(kernel, (int)bytes);
+            if (e != cudaSuccess) return (int)e;
+        }
+        if (p.part_keys == 64) abk_launch(attention_split_latent_kernel<64>, grid, dim3(AS_THREADS), bytes, s, p);
+        else abk_launch(attention_split_latent_kernel<128>, grid, dim3(AS_THREADS), bytes, s, p);
+        if (to) {
+            LatentOut l = *to;
+            l.n_rows = n_tokens;
+            const size_t mixed = (size_t)AL_ROWS * ((v_dim + 31) / 32 * 32 + 8) * 2;
+            int rc = ABK_LAUNCH_RESULT();
+            if (rc) return rc;
+            abk_launch(latent_fold_out_kernel, dim3(n_heads * ((l.outs + AL_OUTS - 1) / AL_OUTS), (n_tokens + AL_ROWS - 1) / AL_ROWS),
+                       dim3(AL_THREADS), mixed, s, p, l);
+            return ABK_LAUNCH_RESULT();
+        }
     } else if (bf && stage) SPLIT_BY_GROUP(__nv_bfloat16, true);
     else if (bf) SPLIT_BY_GROUP(__nv_bfloat16, false);
     else if (stage) SPLIT_BY_GROUP(float, true);
@@ -492,7 +690,7 @@ extern "C" int abk_attention_split(const void *q, long long q_row, void *out, in
                                    int ring_pages, int pinned_pages, int tokens_per_page, int max_keys, float *parts,
                                    long long parts_floats, int chunk, float softcap, const void *gate, long long ldg,
                                    void *stream) {
-    return attention_split(nullptr, 0, chunk, softcap, q, q_row, out, dtype, n_tokens, n_heads, n_kv_heads, head_dim, v_dim, scale, window, keep_first,
+    return attention_split(nullptr, nullptr, 0, chunk, softcap, q, q_row, out, dtype, n_tokens, n_heads, n_kv_heads, head_dim, v_dim, scale, window, keep_first,
                            sink, token_seq, token_pos, seq_slot, k_pool, v_pool, page_table, table_width, ring_pages,
                            pinned_pages, tokens_per_page, max_keys, parts, parts_floats, gate, ldg, stream);
 }
@@ -507,20 +705,26 @@ extern "C" int abk_attention_split_maps(const void *q, long long q_row, void *ou
                                         long long parts_floats, int chunk, float softcap, float lambda, float eps, float keep,
                                         void *stream) {
     const DifferentialHead diff = {lambda, eps, keep};
-    return attention_split(&diff, 0, chunk, softcap, q, q_row, out, dtype, n_tokens, n_heads, n_kv_heads, head_dim, v_dim, scale, window,
+    return attention_split(nullptr, &diff, 0, chunk, softcap, q, q_row, out, dtype, n_tokens, n_heads, n_kv_heads, head_dim, v_dim, scale, window,
                            keep_first, sink, token_seq, token_pos, seq_slot, k_pool, v_pool, page_table, table_width, ring_pages,
                            pinned_pages, tokens_per_page, max_keys, parts, parts_floats, nullptr, 0, stream);
 }
 
 // Keys that carry their values (a value is the first v_dim elements of its key row; one pool): attention over shared
 // latent rows (csrc/latent.cu), every query head in the one group.
+// w (null: none; bfloat16 [heads][outs][v_dim]): out is then [tokens][ldo], head h's `outs` results at h * outs, the weighted
+// latents times w (times sigmoid(gate) with a gate per token and head); else out is [tokens][n_heads * v_dim], the weighted
+// latents themselves.
 extern "C" int abk_attention_split_values_in_keys(const void *q, long long q_row, void *out, int dtype, int n_tokens,
                                                   int n_heads, int n_kv_heads, int head_dim, int v_dim, float scale,
                                                   const float *sink, const int *token_seq, const int *token_pos,
                                                   const int *seq_slot, const void *k_pool, const int *page_table,
                                                   int table_width, int ring_pages, int tokens_per_page, int window, int max_keys,
-                                                  float *parts, long long parts_floats, void *stream) {
-    return attention_split(nullptr, 1, 0, 0.0f, q, q_row, out, dtype, n_tokens, n_heads, n_kv_heads, head_dim, v_dim, scale, window, 0, sink,
-                           token_seq, token_pos, seq_slot, k_pool, k_pool, page_table, table_width, ring_pages, 0, tokens_per_page,
-                           max_keys, parts, parts_floats, nullptr, 0, stream);
+                                                  float *parts, long long parts_floats, const void *w, int outs, long long ldo,
+                                                  const void *gate, long long ldg, void *stream) {
+    LatentOut to;
+    to.w = (const __nv_bfloat16 *)w, to.out = (__nv_bfloat16 *)out, to.ldo = ldo, to.outs = outs, to.n_rows = 0;
+    return attention_split(w ? &to : nullptr, nullptr, 1, 0, 0.0f, q, q_row, out, dtype, n_tokens, n_heads, n_kv_heads, head_dim, v_dim,
+                           scale, window, 0, sink, token_seq, token_pos, seq_slot, k_pool, k_pool, page_table, table_width, ring_pages,
+                           0, tokens_per_page, max_keys, parts, parts_floats, gate, ldg, stream);
 }

@@ -630,6 +630,73 @@ template <int HD> __global__ void __launch_bounds__(FAST_WARPS * 32) qkv_prep_pr
     }
 }
 
+// The general preparation in 16-byte pieces: bfloat16 heads of 16, 32, 64 or 128 elements (HD / 8 lanes each), values a multiple
+// of 8, the rotation in halves over a multiple of 16 elements (or none). A CTA takes a run of a token's pieces, q heads
+// first, then k, then v; a warp's lanes hold whole heads of q and k (a head's pieces come in an aligned run).
+template <int HD> __global__ void __launch_bounds__(256) qkv_prep_pieces_kernel(QkvPrep p, int per_cta) {
+    constexpr int LPH = HD / 8;
+    const int t = blockIdx.x, lane = threadIdx.x & 31;
+    const int heads = p.n_heads + p.n_kv_heads, n_values = p.n_kv_heads / p.maps, v_pieces = p.v_dim / 8;
+    const int total = heads * LPH + (p.q_only ? 0 : n_values * v_pieces), limit = min((int)(blockIdx.y + 1) * per_cta, total);
+    // the step's indices and the page table were written by kernels further back than the one just before
+    const int seq = p.token_seq[t], pos = p.token_pos[t], half = p.rotary_dim / 16;  // half: pieces of half the rotated part
+    __nv_bfloat16 *row = (__nv_bfloat16 *)p.qkv + (long long)t * p.row_size;
+    int page = -1;
+    if (seq >= 0 && !p.q_only && p.k_pool && cache_keeps(p.cache, pos, p.seq_len_after[seq])) page = cache_page(p.cache, p.seq_slot[seq], pos);
+    pdl_wait();
+    if (seq < 0) return;
+    for (int e = blockIdx.y * per_cta + threadIdx.x; e - lane < limit; e += 256) {
+        const bool live = e < limit;
+        uint4 raw = live ? *(const uint4 *)(row + e * 8) : make_uint4(0, 0, 0, 0);
+        const int head = e / LPH, l = e % LPH;
+        if (__any_sync(0xffffffffu, e < heads * LPH)) {
+            const bool mine = e < heads * LPH && live && !(p.q_only && head >= p.n_heads);
+            const float *w = head < p.n_heads ? p.q_norm : p.k_norm;
+            float v[8], other[8];
+            const __nv_bfloat162 *h2 = (const __nv_bfloat162 *)&raw;
+#pragma unroll
+            for (int j = 0; j < 4; j++) {
+                const float2 f = __bfloat1622float2(h2[j]);
+                v[2 * j] = f.x, v[2 * j + 1] = f.y;
+            }
+            if (p.q_norm) {
+                float ss = 0.0f;
+#pragma unroll
+                for (int j = 0; j < 8; j++) ss = fmaf(v[j], v[j], ss);
+#pragma unroll
+                for (int o = LPH / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+                const float scale = 1.0f / sqrtf(ss / (float)HD + p.eps);
+#pragma unroll
+                for (int j = 0; j < 8; j++) v[j] = w[l * 8 + j] * (v[j] * scale);
+            }
+            if (p.cos) {
+                const int from = lane - l + (l < half ? l + half : l < 2 * half ? l - half : l);  // the lane with the partners
+#pragma unroll
+                for (int j = 0; j < 8; j++) other[j] = __shfl_sync(0xffffffffu, v[j], from);
+                if (l < 2 * half) {
+                    const int i = (l < half ? l : l - half) * 8;
+                    const float *c = p.cos + (long long)pos * (p.rotary_dim / 2) + i, *s = p.sin + (long long)pos * (p.rotary_dim / 2) + i;
+#pragma unroll
+                    for (int j = 0; j < 8; j++) v[j] = l < half ? v[j] * c[j] - other[j] * s[j] : v[j] * c[j] + other[j] * s[j];
+                }
+            }
+            if (mine) {
+                __nv_bfloat162 *o2 = (__nv_bfloat162 *)&raw;
+#pragma unroll
+                for (int j = 0; j < 4; j++) o2[j] = __floats2bfloat162_rn(v[2 * j], v[2 * j + 1]);
+                *(uint4 *)(row + e * 8) = raw;
+                const int k = head - p.n_heads;
+                if (k >= 0 && page >= 0)
+                    *(uint4 *)((__nv_bfloat16 *)p.k_pool + cache_offset(p.cache, page, k / p.maps, n_values, pos, p.maps * HD) + k % p.maps * HD + l * 8) = raw;
+            }
+        }
+        if (live && e >= heads * LPH && page >= 0) {
+            const int f = e - heads * LPH, vh = f / v_pieces;
+            *(uint4 *)((__nv_bfloat16 *)p.v_pool + cache_offset(p.cache, page, vh, n_values, pos, p.v_dim) + (f - vh * v_pieces) * 8) = raw;
+        }
+    }
+}
+
 // v_dim: the size of a value head (0: head_dim); pinned_pages: see PagedCache; row_size: elements between rows of qkv; maps: that
 // many of the n_kv_heads k heads in a row share a value head (there are n_kv_heads / maps of those) and one row of the cache,
 // side by side.
@@ -656,6 +723,21 @@ extern "C" int abk_qkv_prep_general(void *qkv, int dtype, int n_tokens, int n_he
     int total_heads = n_heads + n_kv_heads + n_kv_heads / maps;
     dim3 grid(n_tokens, (total_heads + PREP_WARPS - 1) / PREP_WARPS);
     cudaStream_t s = (cudaStream_t)stream;
+    const int vd = v_dim > 0 ? v_dim : head_dim;
+    if (dtype == ABK_BF16 && (head_dim == 16 || head_dim == 32 || head_dim == 64 || head_dim == 128) && vd % 8 == 0 && row_size > 0 &&
+        row_size % 8 == 0 && (!cos || (!interleaved && rotary_dim % 16 == 0)) && (q_norm != nullptr) == (k_norm != nullptr) &&
+        (((uintptr_t)qkv | (uintptr_t)k_pool | (uintptr_t)v_pool) & 15) == 0) {
+        p.v_dim = vd;
+        // a token's pieces on one CTA in a prompt, a CTA a round in a decode step
+        const int pieces = (n_heads + n_kv_heads) * (head_dim / 8) + (q_only ? 0 : n_kv_heads / maps * (vd / 8));
+        const int rounds = (pieces + 255) / 256, per_cta = n_tokens >= 64 ? rounds * 256 : 256;
+        dim3 runs(n_tokens, (pieces + per_cta - 1) / per_cta);
+        if (head_dim == 16) abk_launch(qkv_prep_pieces_kernel<16>, runs, dim3(256), 0, s, p, per_cta);
+        else if (head_dim == 32) abk_launch(qkv_prep_pieces_kernel<32>, runs, dim3(256), 0, s, p, per_cta);
+        else if (head_dim == 64) abk_launch(qkv_prep_pieces_kernel<64>, runs, dim3(256), 0, s, p, per_cta);
+        else abk_launch(qkv_prep_pieces_kernel<128>, runs, dim3(256), 0, s, p, per_cta);
+        return ABK_LAUNCH_RESULT();
+    }
     if (dtype == ABK_BF16)
         abk_launch(qkv_prep_kernel<__nv_bfloat16>, grid, dim3(PREP_WARPS * 32), 0, s, p);
     else

@@ -14,6 +14,10 @@
 // between them, one turn each; the first CTA of a cluster adds the others' sums, in their order,
 // reading them through distributed shared memory.
 // Formula: src/model.c:299, 302, 307, 309.
+//
+// NORMED: the rows of x are normed on the way, out = (w_x * x / sqrt(mean(x^2) + eps)) . w^T: every warp adds up the squares
+// of the columns it reads (together the CTA reads whole rows), multiplies them by the norm's weight as it makes its
+// fragments, and the row's factor is applied to the sums.
 #define ABK_DEFINE_ERROR
 #include "common.cuh"
 #include "tc_common.cuh"
@@ -51,13 +55,15 @@ __device__ __forceinline__ uint4 load16(const __nv_bfloat16 *p, bool ok) {
 // (src/model.c:274-282) instead of the two sums: the feed-forward's first product and its activation in one.
 __device__ __forceinline__ void prefetch_l2(const void *p) { asm volatile("prefetch.global.L2 [%0];" ::"l"(p)); }
 
-template <int NT, int TILE, bool GATED, typename TO>
+template <int NT, int TILE, bool GATED, typename TO, bool NORMED = false>
 __global__ void __launch_bounds__(ROWS_THREADS) gemm_rows_kernel(const __nv_bfloat16 *__restrict__ x,
                                                                  const __nv_bfloat16 *__restrict__ w, TO *__restrict__ out,
                                                                  int M, int N, int K, long long ldx, long long ldw,
                                                                  long long ldo, int block, long long x_plane, int tanh_from,
-                                                                 int act, float limit) {
+                                                                 int act, float limit, const float *norm_w, int norm_count,
+                                                                 float norm_eps) {
     __shared__ float part[ROWS_WARPS][16][8 * NT + 1];
+    __shared__ float squares[NORMED ? ROWS_WARPS : 1][8 * NT];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, r = lane >> 2, c = lane & 3;
     const int ranks = (int)tc::cluster_size(), rank = (int)tc::cluster_rank();  // the cluster splits K
     const int n0 = (blockIdx.x / ranks) * TILE;
@@ -71,6 +77,10 @@ __global__ void __launch_bounds__(ROWS_THREADS) gemm_rows_kernel(const __nv_bflo
     float acc[NT][4];
 #pragma unroll
     for (int t = 0; t < NT; t++) acc[t][0] = acc[t][1] = acc[t][2] = acc[t][3] = 0.0f;
+    float ss[NORMED ? NT : 1];
+    if (NORMED)
+#pragma unroll
+        for (int t = 0; t < NT; t++) ss[NORMED ? t : 0] = 0.0f;
     const int blocks = (rank + 1) * (K / 32 / ranks), first = rank * (K / 32 / ranks) + warp;  // this CTA's part of K
     // several blocks of 32 columns a turn, so that eight 16-byte loads of weights are in flight per lane
     constexpr int TURN = NT <= 2 ? 4 : 2;
@@ -101,6 +111,26 @@ __global__ void __launch_bounds__(ROWS_THREADS) gemm_rows_kernel(const __nv_bflo
 #pragma unroll
             for (int t = 0; t < NT; t++) b[u][t] = load16(x0 + (long long)(8 * t) * ldx + k, in && 8 * t + r < M);
         }
+        if (NORMED) {
+#pragma unroll
+            for (int u = 0; u < TURN; u++) {
+                const int k = (kb + u * ROWS_WARPS) * 32 + 8 * c;
+                if (kb + u * ROWS_WARPS >= blocks) continue;
+                float nw[8];  // (columns beyond norm_count are padding, zeros in x)
+#pragma unroll
+                for (int j = 0; j < 8; j++) nw[j] = k + j < norm_count ? norm_w[k + j] : 0.0f;
+#pragma unroll
+                for (int t = 0; t < NT; t++) {
+                    __nv_bfloat162 *h = (__nv_bfloat162 *)&b[u][t];
+#pragma unroll
+                    for (int j = 0; j < 4; j++) {
+                        const float2 f = __bfloat1622float2(h[j]);
+                        ss[NORMED ? t : 0] = fmaf(f.x, f.x, fmaf(f.y, f.y, ss[NORMED ? t : 0]));
+                        h[j] = __floats2bfloat162_rn(f.x * nw[2 * j], f.y * nw[2 * j + 1]);
+                    }
+                }
+            }
+        }
 #pragma unroll
         for (int u = 0; u < TURN; u++) {
 #pragma unroll
@@ -115,6 +145,14 @@ __global__ void __launch_bounds__(ROWS_THREADS) gemm_rows_kernel(const __nv_bflo
     for (int t = 0; t < NT; t++) {
         part[warp][r][8 * t + 2 * c] = acc[t][0], part[warp][r][8 * t + 2 * c + 1] = acc[t][1];
         part[warp][r + 8][8 * t + 2 * c] = acc[t][2], part[warp][r + 8][8 * t + 2 * c + 1] = acc[t][3];
+    }
+    if (NORMED) {
+#pragma unroll
+        for (int t = 0; t < NT; t++) {  // row 8 t + r's squares lie in the four lanes of its quad
+            float q = ss[NORMED ? t : 0];
+            q += __shfl_xor_sync(0xffffffffu, q, 1), q += __shfl_xor_sync(0xffffffffu, q, 2);
+            if (c == 0) squares[NORMED ? warp : 0][8 * t + r] = q;
+        }
     }
     __syncthreads();
     if (ranks > 1) {
@@ -165,6 +203,12 @@ __global__ void __launch_bounds__(ROWS_THREADS) gemm_rows_kernel(const __nv_bflo
                 sum = __bfloat162float(__float2bfloat16_rn(sum)), up = __bfloat162float(__float2bfloat16_rn(up));
                 sum = gated_mul(act, sum, up, limit);
             } else {
+                if (NORMED) {
+                    float q = 0.0f;
+#pragma unroll
+                    for (int wv = 0; wv < ROWS_WARPS; wv++) q += squares[NORMED ? wv : 0][token];
+                    sum *= 1.0f / sqrtf(q / (float)norm_count + norm_eps);
+                }
                 if (n0 + row >= tanh_from) sum = tanhf(sum);  // (tanh_from beyond N: no feature)
                 sum = out_act(act, sum);
             }
@@ -198,7 +242,7 @@ static int gemm_rows_launch(const void *x, const void *w, void *out, int out_dty
     const __nv_bfloat16 *xb = (const __nv_bfloat16 *)x, *wb = (const __nv_bfloat16 *)w;
 #define ROWS_LAUNCH(NT, TILE, TO)                                                                                     \
     abk_launch_clusters(gemm_rows_kernel<NT, TILE, false, TO>, grid, dim3(ROWS_THREADS), 0, s, ranks, xb, wb, (TO *)out, M, \
-                        N, K, ldx, ldw, ldo, block, x_plane, tanh_from, act, 0.0f)
+                        N, K, ldx, ldw, ldo, block, x_plane, tanh_from, act, 0.0f, nullptr, 1, 0.0f)
 #define ROWS_BY_M(TO)                                                                     \
     if (M <= 8) { if (narrow) ROWS_LAUNCH(1, 8, TO); else ROWS_LAUNCH(1, 16, TO); }       \
     else if (M <= 16) { if (narrow) ROWS_LAUNCH(2, 8, TO); else ROWS_LAUNCH(2, 16, TO); } \
@@ -219,6 +263,28 @@ extern "C" int abk_gemm_rows(const void *x, const void *w, void *out, int out_dt
 extern "C" int abk_gemm_rows_act(const void *x, const void *w, void *out, int out_dtype, int M, int N, int K, long long ldx,
                                  long long ldw, long long ldo, int act, void *stream) {
     return gemm_rows_launch(x, w, out, out_dtype, M, N, K, ldx, ldw, ldo, 0, 0, 0x7fffffff, act, stream);
+}
+
+// The rows of x normed on the way: out = (norm_w * x / sqrt(mean of the first norm_count columns' squares + eps)) . w^T, columns
+// from norm_count on being zeros. M <= 16, out bfloat16.
+extern "C" int abk_gemm_rows_normed(const void *x, const void *w, void *out, int M, int N, int K, long long ldx, long long ldw,
+                                    long long ldo, const float *norm_w, int norm_count, float eps, void *stream) {
+    if (M <= 0 || N <= 0) return 0;
+    if (M > 16) ABK_REFUSE("gemm_rows_normed: %d rows are more than 16", M);
+    if (K <= 0 || K % 32 || ldx % 8 || ldw % 8 || norm_count < 1 || norm_count > K)
+        ABK_REFUSE("gemm_rows_normed: K = %d must be a multiple of 32, the pitches of 8, and hold the %d columns of the norm", K, norm_count);
+    if (((uintptr_t)x | (uintptr_t)w) & 15) ABK_REFUSE("gemm_rows_normed: operands must be 16-byte aligned");
+    const bool narrow = (N + 15) / 16 < 2 * abk_sm_count();
+    dim3 grid(narrow ? (N + 7) / 8 : (N + 15) / 16);
+    cudaStream_t s = (cudaStream_t)stream;
+#define NORMED_LAUNCH(NT, TILE)                                                                                             \
+    abk_launch(gemm_rows_kernel<NT, TILE, false, __nv_bfloat16, true>, grid, dim3(ROWS_THREADS), 0, s, (const __nv_bfloat16 *)x, \
+               (const __nv_bfloat16 *)w, (__nv_bfloat16 *)out, M, N, K, ldx, ldw, ldo, 0, 0LL, 0x7fffffff, ABK_OUT_PLAIN, 0.0f, norm_w, \
+               norm_count, eps)
+    if (M <= 8) { if (narrow) NORMED_LAUNCH(1, 8); else NORMED_LAUNCH(1, 16); }
+    else { if (narrow) NORMED_LAUNCH(2, 8); else NORMED_LAUNCH(2, 16); }
+#undef NORMED_LAUNCH
+    return ABK_LAUNCH_RESULT();
 }
 
 // Several products of one launch: out[:, i * block : (i + 1) * block] = x_i . w[i * block : (i + 1) * block]^T with
@@ -245,7 +311,7 @@ extern "C" int abk_gemm_rows_gated(const void *x, const void *w, void *act, int 
     cudaStream_t s = (cudaStream_t)stream;
     const __nv_bfloat16 *xb = (const __nv_bfloat16 *)x, *wb = (const __nv_bfloat16 *)w;
 #define GATED_LAUNCH(NT) \
-    abk_launch(gemm_rows_kernel<NT, 8, true, __nv_bfloat16>, grid, dim3(ROWS_THREADS), 0, s, xb, wb, (__nv_bfloat16 *)act, M, N, K, ldx, ldw, ldo, block, 0LL, 0x7fffffff, kind, limit)
+    abk_launch(gemm_rows_kernel<NT, 8, true, __nv_bfloat16>, grid, dim3(ROWS_THREADS), 0, s, xb, wb, (__nv_bfloat16 *)act, M, N, K, ldx, ldw, ldo, block, 0LL, 0x7fffffff, kind, limit, nullptr, 1, 0.0f)
     if (M <= 8) GATED_LAUNCH(1);
     else if (M <= 16) GATED_LAUNCH(2);
     else if (M <= 32) GATED_LAUNCH(4);

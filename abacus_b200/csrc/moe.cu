@@ -28,48 +28,92 @@
 #include "common.cuh"
 
 #define MR_THREADS 256
-template <typename T>
-__global__ void __launch_bounds__(MR_THREADS) moe_route_kernel(const T *x, long long ldx, const float *router, int d, int experts,
+// ROWS router rows `stride` apart (row e0 at w) against TOKENS rows in shared memory `pitch` apart: a lane's shares of the sums.
+template <int ROWS, int TOKENS>
+__device__ __forceinline__ void route_dots(const float *w, long long stride, const float *xs, int pitch, int d, int lane, bool vec,
+                                           float (*acc)[4]) {
+    if (vec) {
+        for (int i = lane * 4; i < d; i += 128) {
+            float4 r[ROWS];
+#pragma unroll
+            for (int u = 0; u < ROWS; u++) r[u] = *(const float4 *)(w + u * stride + i);
+#pragma unroll
+            for (int k = 0; k < TOKENS; k++) {
+                const float4 a = *(const float4 *)(xs + k * pitch + i);
+#pragma unroll
+                for (int u = 0; u < ROWS; u++)
+                    acc[k][u] = fmaf(r[u].w, a.w, fmaf(r[u].z, a.z, fmaf(r[u].y, a.y, fmaf(r[u].x, a.x, acc[k][u]))));
+            }
+        }
+    } else {
+        for (int i = lane; i < d; i += 32)
+#pragma unroll
+            for (int k = 0; k < TOKENS; k++)
+#pragma unroll
+                for (int u = 0; u < ROWS; u++) acc[k][u] = fmaf(w[u * stride + i], xs[k * pitch + i], acc[k][u]);
+    }
+}
+
+// TOKENS tokens a CTA (1 for a decode step, 4 for a prompt: the router's rows are then read once for four).
+template <typename T, int TOKENS>
+__global__ void __launch_bounds__(MR_THREADS) moe_route_kernel(const T *x, long long ldx, const float *router, int n_tokens, int d, int experts,
                                                         int top, int score, int always, const int *token_seq,
                                                         int *pair_expert, float *pair_weight, const float *correction,
                                                         float weight_scale, int n_real, const float *bias, float *shared_weight) {
-    extern __shared__ __align__(16) float mr_smem[];  // [d, rounded up to 4] the row, [experts + 1] logits, [experts] taken flags,
-    float *xs = mr_smem, *z = xs + ((d + 3) & ~3);    // [experts] what the choice goes by
+    // a token's row (d rounded up to 4); its [experts + 1] logits, [experts] taken flags, [experts] what the choice goes by
+    extern __shared__ __align__(16) float mr_smem[];
+    const int pitch = (d + 3) & ~3;
+    float *xs = mr_smem, *scratch = xs + TOKENS * pitch;
     const int outputs = experts + (shared_weight ? 1 : 0);  // router rows: the last may be the shared expert's
-    int *taken = (int *)(z + experts + 1);
-    float *key = (float *)(taken + experts);
     const int softmax_chosen = score == 1;
-    const int t = blockIdx.x, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int t0 = blockIdx.x * TOKENS, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int per = top + (always >= 0 ? 1 : 0);  // pairs a token has: its choices, then the expert every token uses
-    pair_expert += (long long)t * per, pair_weight += (long long)t * per;
+    constexpr int W = MR_THREADS / 32;
+    for (int e = warp; e < outputs; e += W)  // weights: on their way while the kernel before is still running
+        for (int i = lane * 32; i < d; i += 1024) asm volatile("prefetch.global.L2 [%0];" ::"l"(router + (long long)e * d + i));
     pdl_wait();
-    if (token_seq[t] < 0) {
-        for (int k = tid; k < per; k += MR_THREADS) pair_expert[k] = -1, pair_weight[k] = 0.0f;
-        if (shared_weight && tid == 0) shared_weight[t] = 0.0f;
-        return;
+    for (int k = 0; k < TOKENS; k++) {
+        const bool on = t0 + k < n_tokens && token_seq[t0 + k] >= 0;
+        for (int i = tid; i < d; i += MR_THREADS) xs[k * pitch + i] = on ? to_float(x[(long long)(t0 + k) * ldx + i]) : 0.0f;
+        int *taken = (int *)(scratch + k * (3 * experts + 1) + experts + 1);
+        for (int e = tid; e < experts; e += MR_THREADS) taken[e] = 0;
     }
-    if (always >= 0 && tid == 0) pair_expert[top] = always, pair_weight[top] = 1.0f;
-    for (int i = tid; i < d; i += MR_THREADS) xs[i] = to_float(x[(long long)t * ldx + i]);
-    for (int e = tid; e < experts; e += MR_THREADS) taken[e] = 0;
     __syncthreads();
     const bool vec = d % 4 == 0 && ((uintptr_t)router & 15) == 0;
-    constexpr int W = MR_THREADS / 32;
     for (int e = warp; e < outputs;) {  // a warp's router rows, up to four at a time so that their loads are in flight together
         const int left = (outputs - e + W - 1) / W, rows = left < 4 ? left : 4;
-        float acc[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+        float acc[TOKENS][4];
+#pragma unroll
+        for (int k = 0; k < TOKENS; k++) acc[k][0] = acc[k][1] = acc[k][2] = acc[k][3] = 0.0f;
         const float *w = router + (long long)e * d;
-        if (rows == 4) lane_dots<4>(w, (long long)W * d, xs, d, lane, vec, acc);
-        else if (rows == 3) lane_dots<3>(w, (long long)W * d, xs, d, lane, vec, acc);
-        else if (rows == 2) lane_dots<2>(w, (long long)W * d, xs, d, lane, vec, acc);
-        else lane_dots<1>(w, 0, xs, d, lane, vec, acc);
-        for (int u = 0; u < rows; u++) {
-            const float sum = warp_sum(acc[u]);
-            if (lane == 0) z[e + u * W] = bias && e + u * W < experts ? sum + bias[e + u * W] : sum;
+        if (rows == 4) route_dots<4, TOKENS>(w, (long long)W * d, xs, pitch, d, lane, vec, acc);
+        else if (rows == 3) route_dots<3, TOKENS>(w, (long long)W * d, xs, pitch, d, lane, vec, acc);
+        else if (rows == 2) route_dots<2, TOKENS>(w, (long long)W * d, xs, pitch, d, lane, vec, acc);
+        else route_dots<1, TOKENS>(w, 0, xs, pitch, d, lane, vec, acc);
+#pragma unroll
+        for (int k = 0; k < TOKENS; k++) {
+#pragma unroll
+            for (int u = 0; u < 4; u++) {
+                if (u >= rows) break;
+                const float sum = warp_sum(acc[k][u]);
+                if (lane == 0) scratch[k * (3 * experts + 1) + e + u * W] = bias && e + u * W < experts ? sum + bias[e + u * W] : sum;
+            }
         }
         e += rows * W;
     }
     __syncthreads();
-    if (warp != 0) return;
+    if (warp >= TOKENS || t0 + warp >= n_tokens) return;  // a warp a token from here on
+    const int t = t0 + warp;
+    pair_expert += (long long)t * per, pair_weight += (long long)t * per;
+    if (token_seq[t] < 0) {
+        for (int k = lane; k < per; k += 32) pair_expert[k] = -1, pair_weight[k] = 0.0f;
+        if (shared_weight && lane == 0) shared_weight[t] = 0.0f;
+        return;
+    }
+    if (always >= 0 && lane == 0) pair_expert[top] = always, pair_weight[top] = 1.0f;
+    float *z = scratch + warp * (3 * experts + 1);
+    int *taken = (int *)(z + experts + 1);
+    float *key = (float *)(taken + experts);
     if (shared_weight && lane == 0) shared_weight[t] = 1.0f / (1.0f + expf(-z[experts]));
     if (score == 2) {  // z becomes softmax(z) over all outputs; the choice goes by it plus the correction
         float mx = -INFINITY, sum = 0.0f;
@@ -120,25 +164,24 @@ extern "C" int abk_moe_route(const void *x, long long ldx, int dtype, const floa
     if (top < 1 || top > experts) ABK_REFUSE("moe_route: %d of %d experts", top, experts);
     if (score < 0 || score > 2) ABK_REFUSE("moe_route: score %d is not built", score);
     if (n_real < 0 || n_real > experts) n_real = experts;
-    const size_t smem = (size_t)(((d + 3) & ~3) + 3 * experts + 1) * 4;
-    if (smem > 200 * 1024) ABK_REFUSE("moe_route: a row of %d and %d experts do not fit shared memory", d, experts);
+    const size_t token = (size_t)(((d + 3) & ~3) + 3 * experts + 1) * 4;
+    if (token > 200 * 1024) ABK_REFUSE("moe_route: a row of %d and %d experts do not fit shared memory", d, experts);
+    const bool four = n_tokens >= 4 * abk_sm_count() && 4 * token <= 100 * 1024;
+    const size_t smem = four ? 4 * token : token;
     cudaStream_t s = (cudaStream_t)stream;
-    if (dtype == ABK_BF16) {
-        if (smem > 48 * 1024) {
-            cudaError_t e = abk_allow_shared_memory((const void *)moe_route_kernel<__nv_bfloat16>, (int)smem);
-            if (e != cudaSuccess) return (int)e;
-        }
-        abk_launch(moe_route_kernel<__nv_bfloat16>, dim3(n_tokens), dim3(MR_THREADS), smem, s, (const __nv_bfloat16 *)x, ldx, router,
-                   d, experts, top, score, always, token_seq, pair_expert, pair_weight, correction, weight_scale, n_real, bias, shared_weight);
-    } else {
-        if (smem > 48 * 1024) {
-            cudaError_t e = abk_allow_shared_memory((const void *)moe_route_kernel<float>, (int)smem);
-            if (e != cudaSuccess) return (int)e;
-        }
-        abk_launch(moe_route_kernel<float>, dim3(n_tokens), dim3(MR_THREADS), smem, s, (const float *)x, ldx, router, d, experts, top,
-                   score, always, token_seq, pair_expert, pair_weight, correction, weight_scale, n_real,
-                   bias, shared_weight);
-    }
+#define MR_LAUNCH(T, TOKENS)                                                                                                    \
+    do {                                                                                                                        \
+        if (smem > 48 * 1024) {                                                                                                 \
+            cudaError_t e = abk_allow_shared_memory((const void *)moe_route_kernel<T, TOKENS>, (int)smem);                      \
+            if (e != cudaSuccess) return (int)e;                                                                                \
+        }                                                                                                                       \
+        abk_launch(moe_route_kernel<T, TOKENS>, dim3((n_tokens + TOKENS - 1) / TOKENS), dim3(MR_THREADS), smem, s, (const T *)x, ldx, \
+                   router, n_tokens, d, experts, top, score, always, token_seq, pair_expert, pair_weight, correction, weight_scale, \
+                   n_real, bias, shared_weight);                                                                                \
+    } while (0)
+    if (dtype == ABK_BF16) { if (four) MR_LAUNCH(__nv_bfloat16, 4); else MR_LAUNCH(__nv_bfloat16, 1); }
+    else { if (four) MR_LAUNCH(float, 4); else MR_LAUNCH(float, 1); }
+#undef MR_LAUNCH
     return ABK_LAUNCH_RESULT();
 }
 

@@ -273,6 +273,24 @@ def gemm_rows(x, w, out, m=None, activation=None):
                                       _ll(w.stride(0)), _ll(out.stride(0)), _i(OUT_ACTIVATIONS[activation]), _stream()), "gemm_rows")
 
 
+def gemm_rows_normed_takes(x, w, out, m, count):
+    """Whether the product of a handful of rows norms them on the way (the first `count` columns, the rest zeros)."""
+    return m <= 16 and count <= w.shape[1] and out.dtype == torch.bfloat16 and gemm_rows_takes(x, w, out, m)
+
+
+def gemm_rows_normed(x, w, out, norm_w, eps, m=None):
+    """out[:m] = (norm_w * x / sqrt(mean(x^2) + eps)) . w^T for m <= 16 rows whose first norm_w.numel() columns are normed
+    (the rest are zeros): the norm of a latent and the product behind it in one kernel."""
+    _need_cuda(x, w, out, norm_w)
+    lib = load_module("gemm_rows")
+    m = x.shape[0] if m is None else m
+    n, k = w.shape
+    assert x.shape[1] == k and out.shape[1] == n and x.shape[0] >= m and out.shape[0] >= m and out.dtype == torch.bfloat16
+    assert norm_w.dtype == torch.float32 and norm_w.is_contiguous() and norm_w.numel() <= k
+    _check(lib, lib.abk_gemm_rows_normed(_p(x), _p(w), _p(out), _i(m), _i(n), _i(k), _ll(x.stride(0)), _ll(w.stride(0)),
+                                         _ll(out.stride(0)), _p(norm_w), _i(norm_w.numel()), _f(eps), _stream()), "gemm_rows_normed")
+
+
 def gemm_rows_planes(x, w, out, block, m=None, tanh_from=None):
     """Several products of a handful of rows in one launch: out[:m, i * block : (i + 1) * block] =
     x[i, :m] . w[i * block : (i + 1) * block]^T for every run i of `block` rows of w (the last run may be shorter).
@@ -986,7 +1004,7 @@ def gated_head_norm(o, gate, weight, out, n_tokens, n_heads, value_dim, eps, sil
 
 # ------------------------------------------------------------------ latent attention (csrc/latent.cu)
 def latent_prep(proj, down_at, n_heads, dim, rot, rank, rot_dims, norm_w, eps, cos, sin, q_dst, q_head, q_rot_at, copy_plain,
-                cache, batch, interleaved=True, rows=None):
+                cache, batch, interleaved=True, rows=None, product=None):
     """What stands between the projections of a latent-attention layer and its attention kernel, per token: the
     latent c = norm_w * z / sqrt(mean(z^2) + eps) over the first `rank` columns of the down-projection (proj[:,
     down_at:]), the rotation (pairs (2i, 2i+1), or with interleaved False (i, i + rot_dims / 2), of the first rot_dims
@@ -995,8 +1013,10 @@ def latent_prep(proj, down_at, n_heads, dim, rot, rank, rot_dims, norm_w, eps, c
     (cache: a cache.LayerKV whose rows hold at least rank + rot elements; of a window's ring of pages only what is still
     there after the step; None: the entry reads another's cache) and, with `rows`, to rows[token] (the step's own), and
     the query parts put into q_dst: head h of a row at h * q_head, its rotated part at + q_rot_at (zeros behind it up
-    to the head's end), its plain part (copy_plain) at + 0."""
-    _need_cuda(proj, norm_w, cos, sin, q_dst)
+    to the head's end), its plain part (copy_plain) at + 0. product (bfloat16 [heads, rank, dim], where
+    latent_product_takes() says so): the plain part times the head's matrix goes to + 0 instead, in the same launch."""
+    _need_cuda(proj, norm_w, cos, sin, q_dst, product)
+    assert product is None or (product.is_contiguous() and product.shape == (n_heads, rank, dim) and product.dtype == proj.dtype)
     lib = load_module("latent")
     n = batch.n_rows
     assert proj.stride(1) == 1 and q_dst.stride(1) == 1 and q_dst.dtype == proj.dtype and proj.shape[0] >= n
@@ -1019,7 +1039,16 @@ def latent_prep(proj, down_at, n_heads, dim, rot, rank, rot_dims, norm_w, eps, c
         _p(cache.page_table if cache is not None else None), _i(cache.table_width if cache is not None else 0),
         _i(cache.ring_pages if cache is not None else 0), _i(cache.tokens_per_page if cache is not None else 1),
         _p(rows), _ll(rows.stride(0) if rows is not None else 0), _p(batch.token_seq), _p(batch.token_pos), _p(batch.seq_slot),
-        _p(batch.seq_len_after), _stream()), "latent_prep")
+        _p(batch.seq_len_after), _p(product), _stream()), "latent_prep")
+
+
+LATENT_PRODUCT_ROWS = 64  # up to how many rows the query parts go into the latent space by the preparation's own kernel
+
+
+def latent_product_takes(proj, n, dim, rot, w):
+    """Whether latent_prep takes the product of the plain query parts with w [heads, rank, dim] in: a few rows in bfloat16."""
+    return (n <= LATENT_PRODUCT_ROWS and proj.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and dim % 8 == 0
+            and (dim + rot) % 8 == 0 and proj.stride(0) % 8 == 0 and proj.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0)
 
 
 def head_product(x, x_head, w, out, o_head, n, gate=None):
@@ -1061,16 +1090,22 @@ def spread_shared(shared, keys, k_head, at, count, heads, n):
                                       _i(count), _i(heads), _i(_dt(keys)), _i(n), _stream()), "spread_shared")
 
 
-def attention_values_in_keys(q, out, n_heads, head_dim, v_dim, scale, batch, cache, sink=None, ws=None, window=None, rows=None):
+def attention_values_in_keys(q, out, n_heads, head_dim, v_dim, scale, batch, cache, sink=None, ws=None, window=None, rows=None,
+                             values=None, gate=None):
     """Causal attention of every token of the step over a cache with one kv head whose values are the first v_dim
     elements of its keys (latent rows), float32 softmax weights, an optional sink. q [tokens, n_heads * head_dim], out
     [tokens, n_heads * v_dim]. A step of one token a sequence in bfloat16 with rows of up to 256
     runs split along the keys (csrc/attention_split.cu), everything else on the general kernel. window: only the last
-    `window` keys are seen. rows [tokens, head_dim]: keys come from the step's own rows (whole prompts), not the cache."""
-    _need_cuda(q, out, sink, rows)
+    `window` keys are seen. rows [tokens, head_dim]: keys come from the step's own rows (whole prompts), not the cache.
+    values (bfloat16 [heads, outs, v_dim], where latent_values_takes() says so): out [tokens, n_heads * outs] holds head h's
+    result times values[h], and, with gate (a gate per row and head), times its sigmoid."""
+    _need_cuda(q, out, sink, rows, values, gate)
     n = batch.n_rows
+    outs = v_dim if values is None else values.shape[1]
+    assert values is None or (values.is_contiguous() and values.shape == (n_heads, outs, v_dim) and values.dtype == q.dtype)
+    assert gate is None or (values is not None and gate.dtype == q.dtype and gate.stride(1) == 1 and gate.shape[1] >= n_heads)
     assert q.is_contiguous() and q.shape[1] == n_heads * head_dim and out.is_contiguous() and out.dtype == q.dtype
-    assert out.shape[1] == n_heads * v_dim and cache.k.dtype == q.dtype and cache.k.shape[1:] == (1, cache.tokens_per_page, head_dim)
+    assert out.shape[1] == n_heads * outs and cache.k.dtype == q.dtype and cache.k.shape[1:] == (1, cache.tokens_per_page, head_dim)
     assert cache.values_in_keys and v_dim <= head_dim and (rows is None or (rows.is_contiguous() and rows.dtype == q.dtype
                                                                             and rows.shape[1] == head_dim and rows.shape[0] >= n))
     if rows is not None and batch.any_continuation:
@@ -1084,20 +1119,29 @@ def attention_values_in_keys(q, out, n_heads, head_dim, v_dim, scale, batch, cac
         if batch.max_len_after > top:
             raise KernelError(f"a row at position {batch.max_len_after - 1} is beyond the bound {top}")
         top = min(top, window) if window else top
-        n_parts = -(-top // 128)
+        n_parts = -(-top // 64)
         parts = ws.get("attention_parts", (n * n_heads * n_parts * (v_dim + 2),), torch.float32)
         _check(lib, lib.abk_attention_split_values_in_keys(
             _p(q), _ll(q.shape[1]), _p(out), _i(_dt(q)), _i(n), _i(n_heads), _i(1), _i(head_dim), _i(v_dim), _f(scale),
             _p(sink), _p(batch.token_seq), _p(batch.token_pos), _p(batch.seq_slot), _p(cache.k), _p(cache.page_table),
             _i(cache.table_width), _i(cache.ring_pages), _i(cache.tokens_per_page), _i(window or 0), _i(top), _p(parts),
-            _ll(parts.numel()), _stream()), "attention_split", kernels=2)
+            _ll(parts.numel()), _p(values), _i(outs), _ll(out.stride(0)), _p(gate), _ll(gate.stride(0) if gate is not None else 0),
+            _stream()), "attention_split", kernels=2)
         return
+    if values is not None:
+        raise KernelRefused("values out of the latent space go with a step of one token a sequence (latent_values_takes)")
     lib = load_module("attention_generic")
     _check(lib, lib.abk_attention_values_in_keys(
         _p(q), _ll(q.shape[1]), _p(out), _i(_dt(q)), _i(n), _i(n_heads), _i(1), _i(head_dim), _f(scale),
         _p(batch.token_seq), _p(batch.token_pos), _p(batch.seq_slot), _p(batch.seq_start), _p(batch.seq_pos0), _p(cache.k),
         _p(cache.page_table), _i(cache.table_width), _i(cache.ring_pages), _i(cache.tokens_per_page), _p(rows),
         _ll(rows.stride(0) if rows is not None else 0), _i(v_dim), _i(window or 0), _p(sink), _i(1), _stream()), "attention")
+
+
+def latent_values_takes(q, head_dim, v_dim, batch, values):
+    """Whether attention_values_in_keys carries its results out of the latent space (values [heads, outs, v_dim]) itself."""
+    return (batch.is_decode and q.dtype == torch.bfloat16 and values.dtype == torch.bfloat16 and head_dim % 16 == 0 and head_dim <= 256
+            and v_dim % 8 == 0 and values.data_ptr() % 16 == 0 and q.data_ptr() % 16 == 0)
 
 
 def attention_differential(qkv, out, n_heads, n_kv_heads, head_dim, scale, window, batch, cache, lam, eps, keep, from_step=False,

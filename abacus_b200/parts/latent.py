@@ -22,7 +22,7 @@ import torch
 from ..cache.need import CacheNeed
 from ..kernels import ops
 from .base import MIXERS, POSITIONS, to_device
-from .linear import Linear
+from .linear import Linear, rows_kernel_wins
 
 
 def _up8(n):
@@ -139,8 +139,12 @@ class LatentAttention:
         if self.q_up is not None:
             self.in_proj.forward(xn, proj[:, self.down_at:], n)
             q_latent = proj[:, self.q_latent_at:self.q_latent_at + self.q_rank8]  # (its padding columns are zeros)
-            ops.columns_norm(q_latent, q_latent, s.q_rank, self.q_norm, s.norm_eps, n)
-            self.q_up.forward(q_latent, proj[:, :self.q_size], n)
+            q = proj[:, :self.q_size]
+            if rows_kernel_wins(n, self.q_up.weight) and ops.gemm_rows_normed_takes(q_latent, self.q_up.weight, q, n, s.q_rank):
+                ops.gemm_rows_normed(q_latent, self.q_up.weight, q, self.q_norm, s.norm_eps, n)  # a handful of rows: normed on the way
+            else:
+                ops.columns_norm(q_latent, q_latent, s.q_rank, self.q_norm, s.norm_eps, n)
+                self.q_up.forward(q_latent, q, n)
         else:
             self.in_proj.forward(xn, proj, n)
         att = ws.get("att", (n, s.n_heads * s.v_head_dim), dt)
@@ -166,16 +170,24 @@ class LatentAttention:
             ops.attention(qkv, att, s.n_heads, s.n_heads, self.per_head, s.scale, s.window, batch, None, from_step=True, ws=ws,
                           v_dim=s.v_head_dim, sink=self.sink, exact_weights=True, row=qkv.shape[1])
         else:
+            # a few rows: the queries' way into the latent space in the preparation's kernel, the values' way out of it (and
+            # the heads' gates) in the one that folds attention's parts
             q_lat = ws.get("latent_q", (n, s.n_heads * self.row), dt)
+            gates = proj[:, self.gate_at:] if s.head_gate else None
+            product = self.uk_t if own is None and ops.latent_product_takes(proj, n, s.head_dim, s.rot_dim, self.uk_t) else None
             ops.latent_prep(proj, self.down_at, s.n_heads, s.head_dim, s.rot_dim, s.rank, rot_dims, self.down_norm,
                             s.norm_eps, self.cos, self.sin, q_lat, self.row, s.rank, False,
-                            kv if cache.owns_storage else None, batch, interleaved=self.interleaved, rows=own)
-            ops.head_product(proj, self.per_head, self.uk_t, q_lat, self.row, n)
-            mixed = ws.get("latent_mixed", (n, s.n_heads * s.rank), dt)
-            ops.attention_values_in_keys(q_lat, mixed, s.n_heads, self.row, s.rank, s.scale, batch, kv, self.sink, ws,
-                                         window=s.window, rows=own)
-            # (head h's output times sigmoid(g_h . x) where the values leave the latent space)
-            ops.head_product(mixed, s.rank, self.uv, att, s.v_head_dim, n, gate=proj[:, self.gate_at:] if s.head_gate else None)
+                            kv if cache.owns_storage else None, batch, interleaved=self.interleaved, rows=own, product=product)
+            if product is None:
+                ops.head_product(proj, self.per_head, self.uk_t, q_lat, self.row, n)
+            if ops.latent_values_takes(q_lat, self.row, s.rank, batch, self.uv):
+                ops.attention_values_in_keys(q_lat, att, s.n_heads, self.row, s.rank, s.scale, batch, kv, self.sink, ws,
+                                             window=s.window, values=self.uv, gate=gates)
+            else:
+                mixed = ws.get("latent_mixed", (n, s.n_heads * s.rank), dt)
+                ops.attention_values_in_keys(q_lat, mixed, s.n_heads, self.row, s.rank, s.scale, batch, kv, self.sink, ws,
+                                             window=s.window, rows=own)
+                ops.head_product(mixed, s.rank, self.uv, att, s.v_head_dim, n, gate=gates)
             gated = True
         if s.head_gate and not gated:  # head h's output times sigmoid(g_h . x)
             ops.gate_heads(att, proj[:, self.gate_at:], s.n_heads, s.v_head_dim, n)

@@ -591,6 +591,42 @@ def build_lilovik(size):
     return model
 
 
+# Kimilix at the same widths, depths and vocabulary: of every four layers the first differential attention (16 or 32 heads of
+# two maps of 64 and values of 128 over 8 key heads, chunks of 1,024 positions), the others latent attention (heads of
+# 128 + 64 rotated, values of 128, 192 latents, queries through a latent of their own) under a window of 1,024; the first
+# layer's feed-forward plain and dense, the others 16 gated experts of which a token uses 2, and a shared one of their size.
+KIMILIX_SIZES = {
+    "s": dict(heads=16, kv_heads=8, q_rank=384, experts=16, top=2, expert_ff=768),
+    "m": dict(heads=32, kv_heads=8, q_rank=768, experts=16, top=2, expert_ff=2432),
+}
+
+
+def build_kimilix(size):
+    import torch
+    from abacus_b200.config import get_architecture
+    from abacus_b200.config.kimilix import (KimilixAttention, KimilixConfig, KimilixDense, KimilixExperts, KimilixLatent,
+                                            KimilixLayer, KimilixRotation)
+    from abacus_b200.models import Model
+    from abacus_b200.weights import random_tensors
+    z, v = DESIGN_SIZES[size], KIMILIX_SIZES[size]
+    attention = KimilixAttention(v["heads"], v["kv_heads"], 64, 128, 64 ** -0.5, 0.3, 1024,
+                                 KimilixRotation(500000.0, 64, (8.0, 8192.0, 1.0, 4.0)))
+    latent = KimilixLatent(v["heads"], 128, 64, 128, 192, v["q_rank"], 192 ** -0.5, 1024, KimilixRotation(50000.0, 64))
+    experts = KimilixExperts(v["experts"], v["top"], v["expert_ff"], 7.0, v["expert_ff"], 7.0)
+    layers = tuple(KimilixLayer("latent_attention" if i % 4 else "attention", latent if i % 4 else attention,
+                                experts if i else KimilixDense(z["ff"])) for i in range(z["layers"]))
+    config = KimilixConfig(vocab=z["vocab"], width=z["width"], layers=layers, eps=1e-6, embedding_scale=8.0, residual_mult=0.5)
+    arch = get_architecture("Kimilix")
+    spec = config.to_spec()
+    expected, _ = arch.tensor_names(spec, None)
+    device = torch.device("cuda", 0)
+    tensors = random_tensors(expected, seed=5, std=0.02, device=device, rule=arch.random_moments)
+    model = Model(spec, arch.layout(spec), tensors, torch.bfloat16, device)
+    del tensors
+    torch.cuda.empty_cache()
+    return model
+
+
 def state_and_cache_bytes(model, tokens_held, n_seqs):
     """Bytes of keys, values and recurrent state a decode step moves for n_seqs sequences that hold tokens_held
     tokens together: a window's keys at most, the keys of the token's own chunk where attention sees no others, a state
@@ -627,12 +663,12 @@ def routed_expert_bytes(model, n_rows):
         if spec is None or getattr(spec, "kind", "") != "routed_mlp":
             continue
         distinct = spec.experts * (1.0 - (1.0 - 1.0 / spec.experts) ** (n_rows * spec.top))
-        total += distinct * 2 * spec.hidden * spec.expert.inter * ffn.up.element_size()
+        total += distinct * (ffn.up[0].numel() + ffn.down[0].numel()) * ffn.up.element_size()
     return total
 
 
 def run_design(args):
-    """--design temetar | movarax | linonex | tilulorn | lilovik: decode and prefill of the design at DESIGN_SIZES[--size] beside the Qwen3
+    """--design temetar | movarax | linonex | tilulorn | lilovik | kimilix: decode and prefill of the design at DESIGN_SIZES[--size] beside the Qwen3
     shape of equal size (--beside: beside another design of equal size instead)."""
     import torch
     from abacus_b200.kernels import build_all
@@ -647,6 +683,8 @@ def run_design(args):
         shape = {**{k: shape[k] for k in ("width", "ff", "layers", "vocab")}, **LINONEX_SIZES[args.size]}
     if args.design == "tilulorn":
         shape = {**{k: shape[k] for k in ("width", "layers", "vocab")}, **TILULORN_SIZES[args.size]}
+    if args.design == "kimilix":
+        shape = {**{k: shape[k] for k in ("width", "ff", "layers", "vocab")}, **KIMILIX_SIZES[args.size]}
     out = {"design": args.design.capitalize(), "size": args.size, "shape": shape,
            "batch": args.batch, "prompt_tokens": PROMPT, "steps": args.steps, "warmup": args.warmup, "peaks": pk}
     for which in (args.design, args.beside):
@@ -660,6 +698,8 @@ def run_design(args):
             model = build_tilulorn(args.size)
         elif which == "lilovik":
             model = build_lilovik(args.size)
+        elif which == "kimilix":
+            model = build_kimilix(args.size)
         else:
             model, _ = build_model(z["qwen"])
         prompts = prompts_for(args.batch, model.spec.vocab, 10 + args.batch)
@@ -768,7 +808,7 @@ def main():
     ap.add_argument("--config", default="0.6b", choices=sorted(CONFIGS), help="whose workload the line reports")
     ap.add_argument("--skip-large", action="store_true", help="leave the 4b and 8b workloads out of `points`")
     ap.add_argument("--ragged", action="store_true", help="with --only prefill: the configuration's own prompts")
-    ap.add_argument("--design", default=None, choices=["temetar", "movarax", "linonex", "tilulorn", "lilovik"],
+    ap.add_argument("--design", default=None, choices=["temetar", "movarax", "linonex", "tilulorn", "lilovik", "kimilix"],
                     help="instead of the default workload: this design at --size beside the Qwen3 shape of equal size")
     ap.add_argument("--size", default="s", choices=sorted(DESIGN_SIZES), help="with --design: the layer sizes")
     ap.add_argument("--beside", default="qwen3", choices=["qwen3", "temetar", "movarax", "linonex", "tilulorn"],
