@@ -1,6 +1,6 @@
 // Decode attention (one new token per sequence) over the paged cache with the general options (a window that also
 // keeps the first keys, a sink, values of another size than keys, float32 softmax weights), split along the keys so
-// that a handful of rows fills the GPU: a CTA takes 128 of a row's visible keys for all query heads of one kv head
+// that a handful of rows fills the GPU: a CTA takes 64 or 128 of a row's visible keys for all query heads of one kv head
 // (each key and value row is read once for the group), and leaves, per head, the maximum, the sum and the
 // unnormalised weighted values of its keys; a second kernel folds a row's parts, the sink among them.
 //
@@ -13,7 +13,7 @@
 // the same values; the fold makes one head of the two (csrc/differential.cuh), so both maps' sums stay float32.
 //
 // A row's visible keys are numbered: first the kept first keys the window no longer reaches, then the window's
-// (or all). Part t has numbers [128 t, 128 t + 128). All arithmetic is float32.
+// (or all). Part t has numbers [P t, P t + P), P = 128, or 64 where parts of 128 are too few. All arithmetic is float32.
 #define ABK_DEFINE_ERROR
 #include "common.cuh"
 #include "differential.cuh"
@@ -39,7 +39,7 @@ struct AttnSplit {
     const int *token_seq, *token_pos, *seq_slot;
     const void *k_pool, *v_pool;
     PagedCache cache, v_cache;
-    int n_parts, part_keys;  // a row's parts have part_keys keys each (128, or 64 in the kernel for latent rows)
+    int n_parts, part_keys;  // a row's parts have part_keys keys each (128, or 64)
     int values_in_keys;  // a value is the first v_dim elements of its key row (one pool)
     int runs;            // runs of query heads, a CTA each, that share a kv head of the cache; n_kv_heads counts the runs
     const void *gate;    // null, or a gate per token and head (of q's type, at gate + t * ldg + h): the head's output is
@@ -232,21 +232,25 @@ template <typename T, bool STAGED, int GMAX> __global__ void __launch_bounds__(A
     }
 }
 
-// The same for bfloat16 keys that carry their values (latent rows: one kv head, head_dim a multiple of 16, values a multiple of
-// 8 up to 256), both products on the warp-level tensor cores with the group's heads as the 16 rows of a tile. A CTA takes
-// PART keys; they and the queries come into shared memory by cp.async, zeros in the places of keys and heads there are none
-// of. A warp makes the scores of PART / 4 keys and has them in registers: maxima and sums meet over the warps through
-// shared memory. The weighted values: the float32 weights as three bfloat16 parts that hold their 24 bits, each multiplied
-// with the same value fragments, so that the weights stay float32 in effect.
-template <int PART> __global__ void __launch_bounds__(AS_THREADS) attention_split_latent_kernel(AttnSplit p) {
+// The same in bfloat16 with both products on the warp-level tensor cores, the group's heads as the 16 rows of a tile (key rows
+// a multiple of 16 elements, values a multiple of 8 up to 256). A CTA takes PART keys; they, their values (OWN_V; else a
+// value is the first elements of its key row: latent rows) and the queries come into shared memory by cp.async, zeros in
+// the places of keys and heads there are none of. Where a head has two maps its query stands in its map's half of a row as
+// wide as a key's, zeros in the other, so that one product makes both maps' scores. A warp makes the scores of PART / 4 keys and
+// has them in registers: maxima and sums meet over the warps through shared memory. The weighted values: the float32
+// weights as three bfloat16 parts that hold their 24 bits, each multiplied with the same value fragments, so that the
+// weights stay float32 in effect.
+template <int PART, bool OWN_V> __global__ void __launch_bounds__(AS_THREADS) attention_split_tiles_kernel(AttnSplit p) {
     extern __shared__ __align__(16) float as_smem[];
     constexpr int KEYS = PART / 4, NT = KEYS / 8, P_PITCH = PART + 8;  // a warp's keys, its tiles of 8
-    const int group = p.n_heads / p.n_kv_heads, hd = p.head_dim, vd = p.v_dim, pitch = hd * 2 + 16;
+    const int group = p.n_heads / p.n_kv_heads, hd = p.head_dim, vd = p.v_dim, kd = p.maps * hd, pitch = kd * 2 + 16;
+    const int v_pitch = OWN_V ? ((vd + 15) & ~15) * 2 + 16 : pitch;
     float *p_s = as_smem;                           // [16][P_PITCH] weights
     float *red = p_s + 16 * P_PITCH;                // [2][4][16] the warps' maxima, then their sums
     uint8_t *q_s = (uint8_t *)(red + 128);          // [16][pitch]
     uint8_t *k_s = q_s + 16 * pitch;                // [PART][pitch]
-    __shared__ long long k_off[PART];
+    uint8_t *v_s = OWN_V ? k_s + PART * pitch : k_s;  // [PART][v_pitch]
+    __shared__ long long k_off[PART], v_off[OWN_V ? PART : 1];
     const int t = blockIdx.x, run = blockIdx.y, part = blockIdx.z, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int g = lane >> 2, c2 = (lane & 3) * 2;
     // the step's indices, the page table and the keys of earlier steps were written by kernels further back than the one just
@@ -262,11 +266,13 @@ template <int PART> __global__ void __launch_bounds__(AS_THREADS) attention_spli
     const int slot = p.seq_slot[seq], n_valid = min(total - part * PART, PART);
     if (tid < PART) {
         const int number = part * PART + min(tid, n_valid - 1), j = number < kept ? number : lo + number - kept;
-        const int cn = p.n_kv_heads / p.runs;
-        k_off[tid] = cache_offset(p.cache, cache_page(p.cache, slot, j), run / p.runs, cn, j, hd);
+        const int cn = p.n_kv_heads / p.runs, page = cache_page(p.cache, slot, j);
+        k_off[tid] = cache_offset(p.cache, page, run / p.runs, cn, j, kd);
+        if (OWN_V) v_off[OWN_V ? tid : 0] = cache_offset(p.v_cache, page, run / p.runs, cn, j, vd);
     }
     const uint32_t q_at = (uint32_t)__cvta_generic_to_shared(q_s), k_at = (uint32_t)__cvta_generic_to_shared(k_s);
-    const int chunks = hd / 8;
+    const int chunks = kd / 8, v_chunks = vd / 8;
+    const uint32_t v_at = (uint32_t)__cvta_generic_to_shared(v_s);
     const __nv_bfloat16 *q = (const __nv_bfloat16 *)p.q + (long long)t * p.q_row + (long long)run * group * hd;
     // where the token's own key lies among the part's (it is the last that is seen)
     const int own = part * PART + n_valid == total ? n_valid - 1 : PART;
@@ -277,15 +283,29 @@ template <int PART> __global__ void __launch_bounds__(AS_THREADS) attention_spli
         asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(k_at + r * pitch + c * 16),
                      "l"((const __nv_bfloat16 *)p.k_pool + k_off[r] + c * 8), "r"(r < n_valid ? 16 : 0) : "memory");
     }
+    if (OWN_V)
+        for (int e = tid; e < PART * v_chunks; e += AS_THREADS) {
+            const int r = e / v_chunks, c = e - r * v_chunks;
+            if (r == own) continue;
+            asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(v_at + r * v_pitch + c * 16),
+                         "l"((const __nv_bfloat16 *)p.v_pool + v_off[OWN_V ? r : 0] + c * 8), "r"(r < n_valid ? 16 : 0) : "memory");
+        }
     pdl_wait();
-    if (own < PART)
+    if (own < PART) {
         for (int c = tid; c < chunks; c += AS_THREADS)
             asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(k_at + own * pitch + c * 16),
                          "l"((const __nv_bfloat16 *)p.k_pool + k_off[own] + c * 8) : "memory");
+        if (OWN_V)
+            for (int c = tid; c < v_chunks; c += AS_THREADS)
+                asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(v_at + own * v_pitch + c * 16),
+                             "l"((const __nv_bfloat16 *)p.v_pool + v_off[OWN_V ? own : 0] + c * 8) : "memory");
+    }
+    const int slice = chunks / p.maps;  // 16-byte pieces of a map
     for (int e = tid; e < 16 * chunks; e += AS_THREADS) {
-        const int r = e / chunks, c = e - r * chunks;
+        const int r = e / chunks, c = e - r * chunks, first = r % p.maps * slice;
+        const bool in = r < group && c >= first && c < first + slice;
         asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(q_at + r * pitch + c * 16),
-                     "l"(q + (long long)min(r, group - 1) * hd + c * 8), "r"(r < group ? 16 : 0) : "memory");
+                     "l"(q + (long long)min(r, group - 1) * hd + (in ? c - first : 0) * 8), "r"(in ? 16 : 0) : "memory");
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
     asm volatile("cp.async.wait_group 0;" ::: "memory");
@@ -297,7 +317,7 @@ template <int PART> __global__ void __launch_bounds__(AS_THREADS) attention_spli
     const uint32_t qa = q_at + (lane & 15) * pitch + (lane >> 4) * 16;
     const uint32_t ka = k_at + (warp * KEYS + (lane & 7) + ((lane >> 4) << 3)) * pitch + ((lane >> 3) & 1) * 16;
 #pragma unroll 4
-    for (int kk = 0; kk < hd / 16; kk++) {
+    for (int kk = 0; kk < kd / 16; kk++) {
         uint32_t a[4];
         ldsm_x4(qa + kk * 32, a[0], a[1], a[2], a[3]);
 #pragma unroll
@@ -349,7 +369,7 @@ template <int PART> __global__ void __launch_bounds__(AS_THREADS) attention_spli
 #pragma unroll
         for (int e = 0; e < 8; e++) o[i][e] = 0.0f;
     const int n_pairs = (vd + 15) / 16;
-    const uint32_t va = k_at + ((lane & 7) + ((lane >> 3) & 1) * 8) * pitch + (lane >> 4) * 16;
+    const uint32_t va = v_at + ((lane & 7) + ((lane >> 3) & 1) * 8) * v_pitch + (lane >> 4) * 16;
 #pragma unroll
     for (int ks = 0; ks < PART / 16; ks++) {
         if (ks * 16 >= n_valid) break;
@@ -364,7 +384,7 @@ template <int PART> __global__ void __launch_bounds__(AS_THREADS) attention_spli
             const int pair = warp + 4 * i;
             if (pair >= n_pairs) break;
             uint32_t b0, b1, b2, b3;
-            ldsm_x4_t(va + ks * 16 * pitch + pair * 32, b0, b1, b2, b3);
+            ldsm_x4_t(va + ks * 16 * v_pitch + pair * 32, b0, b1, b2, b3);
             mma_bf16(o[i], hi, b0, b1), mma_bf16(o[i] + 4, hi, b2, b3);
             mma_bf16(o[i], mid, b0, b1), mma_bf16(o[i] + 4, mid, b2, b3);
             mma_bf16(o[i], low, b0, b1), mma_bf16(o[i] + 4, low, b2, b3);
@@ -499,42 +519,50 @@ __global__ void __launch_bounds__(AL_THREADS) latent_fold_out_kernel(AttnSplit p
     }
 }
 
-// out[t, h] = sum over the row's parts (and the sink) of their weighted values, over the sum of their sums, all
-// against the largest maximum. One CTA per (token, head), parts in order.
-template <typename T> __global__ void __launch_bounds__(AS_THREADS) attention_fold_kernel(AttnSplit p) {
-    const int t = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, vd = p.v_dim;
-    const float sink = p.sink ? p.sink[h] : -INFINITY;  // a weight: ahead of the wait
-    pdl_wait();
-    T *out = (T *)p.out + ((long long)t * p.n_heads + h) * vd;
-    const int seq = p.token_seq[t];
-    if (seq < 0) {
-        for (int d = tid; d < vd; d += AS_THREADS) out[d] = from_float<T>(0.0f);
-        return;
+// The weighted values of a row's parts over the sum of their sums (and the sink's), all against the largest maximum: columns
+// tid and tid + AS_THREADS of one head. A lane has a part's weight; all parts' loads of a round are in flight together.
+#define AF_PARTS 8
+__device__ __forceinline__ void fold_parts(const float *src, int n, int vd, float sink, bool has_sink, float &a, float &b) {
+    const int tid = threadIdx.x, lane = tid & 31;
+    float top = sink, sum = 0.0f;
+    a = b = 0.0f;
+    if (n > 32) {  // (up to 32 parts a lane's own maximum is the one it has below)
+        for (int k = lane; k < n; k += 32) top = fmaxf(top, src[(long long)k * (vd + 2) + vd]);
+        top = warp_max(top);
     }
-    int lo, kept, total;
-    visible_keys(p, p.token_pos[t], lo, kept, total);
-    const int n = (total + p.part_keys - 1) / p.part_keys;
-    const float *src = p.parts + ((long long)t * p.n_heads + h) * p.n_parts * (vd + 2);
-    float top = sink;
-    for (int i = 0; i < n; i++) top = fmaxf(top, src[(long long)i * (vd + 2) + vd]);
-    float l = p.sink ? expf(sink - top) : 0.0f, a = 0.0f, b = 0.0f;
-    for (int i = 0; i < n; i++) {
-        const float *part = src + (long long)i * (vd + 2);
-        const float w = expf(part[vd] - top);
-        l = fmaf(part[vd + 1], w, l);
-        if (tid < vd) a = fmaf(part[tid], w, a);
-        if (tid + AS_THREADS < vd) b = fmaf(part[tid + AS_THREADS], w, b);
+    for (int k0 = 0; k0 < n; k0 += 32) {
+        const int left = min(32, n - k0);
+        const float *own = src + (long long)(k0 + lane) * (vd + 2) + vd;
+        const float m = lane < left ? own[0] : -INFINITY, l = lane < left ? own[1] : 0.0f;
+        if (n <= 32) top = warp_max(fmaxf(top, m));
+        const float w = expf(m - top);  // (0 in lanes without a part)
+        sum = fmaf(l, w, sum);
+        for (int k = 0; k < left; k += AF_PARTS) {
+            float x[AF_PARTS], y[AF_PARTS];
+#pragma unroll
+            for (int i = 0; i < AF_PARTS; i++) {
+                const float *part = src + (long long)(k0 + k + i) * (vd + 2);
+                x[i] = k + i < left && tid < vd ? part[tid] : 0.0f;
+                y[i] = k + i < left && tid + AS_THREADS < vd ? part[tid + AS_THREADS] : 0.0f;
+            }
+#pragma unroll
+            for (int i = 0; i < AF_PARTS; i++) {
+                const float wk = __shfl_sync(0xffffffffu, w, (k + i) & 31);
+                a = fmaf(x[i], wk, a), b = fmaf(y[i], wk, b);
+            }
+        }
     }
-    const float g = p.gate ? 1.0f / (1.0f + expf(-to_float(((const T *)p.gate)[(long long)t * p.ldg + h]))) : 1.0f;
-    if (tid < vd) out[tid] = from_float<T>(a / l * g);
-    if (tid + AS_THREADS < vd) out[tid + AS_THREADS] = from_float<T>(b / l * g);
+    sum = warp_sum(sum) + (has_sink ? expf(sink - top) : 0.0f);
+    a /= sum, b /= sum;
 }
 
-// The same for differential attention: out[t, h] of the two maps 2 h and 2 h + 1. One CTA per (token, head).
-template <typename T> __global__ void __launch_bounds__(AS_THREADS) attention_fold_maps_kernel(AttnSplit p) {
+// One CTA per (token, head); with two maps a head, per head: out[t, h] of the maps 2 h and 2 h + 1.
+template <typename T, int MAPS> __global__ void __launch_bounds__(AS_THREADS) attention_fold_kernel(AttnSplit p) {
     __shared__ float scratch[33];
-    const int t = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, vd = p.v_dim, heads = p.n_heads / 2;
-    const float sinks[2] = {p.sink ? p.sink[2 * h] : -INFINITY, p.sink ? p.sink[2 * h + 1] : -INFINITY};
+    const int t = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, vd = p.v_dim, heads = p.n_heads / MAPS;
+    float sink[MAPS];
+#pragma unroll
+    for (int m = 0; m < MAPS; m++) sink[m] = p.sink ? p.sink[MAPS * h + m] : -INFINITY;  // weights: ahead of the wait
     const int seq = p.token_seq[t], pos = p.token_pos[t];
     pdl_wait();
     T *out = (T *)p.out + ((long long)t * heads + h) * vd;
@@ -545,32 +573,23 @@ template <typename T> __global__ void __launch_bounds__(AS_THREADS) attention_fo
     int lo, kept, total;
     visible_keys(p, pos, lo, kept, total);
     const int n = (total + p.part_keys - 1) / p.part_keys;
-    float a[2], b[2];
+    float a[MAPS], b[MAPS];
 #pragma unroll
-    for (int m = 0; m < 2; m++) {
-        const float *src = p.parts + ((long long)t * p.n_heads + 2 * h + m) * p.n_parts * (vd + 2);
-        float top = sinks[m];
-        for (int i = 0; i < n; i++) top = fmaxf(top, src[(long long)i * (vd + 2) + vd]);
-        float l = p.sink ? expf(sinks[m] - top) : 0.0f;
-        a[m] = b[m] = 0.0f;
-        for (int i = 0; i < n; i++) {
-            const float *part = src + (long long)i * (vd + 2);
-            const float w = expf(part[vd] - top);
-            l = fmaf(part[vd + 1], w, l);
-            if (tid < vd) a[m] = fmaf(part[tid], w, a[m]);
-            if (tid + AS_THREADS < vd) b[m] = fmaf(part[tid + AS_THREADS], w, b[m]);
-        }
-        a[m] /= l, b[m] /= l;
+    for (int m = 0; m < MAPS; m++)
+        fold_parts(p.parts + ((long long)t * p.n_heads + MAPS * h + m) * p.n_parts * (vd + 2), n, vd, sink[m], p.sink != nullptr, a[m], b[m]);
+    if (MAPS == 2) {
+        a[0] = differential_value(p.diff, a[0], a[MAPS - 1]), b[0] = differential_value(p.diff, b[0], b[MAPS - 1]);  // (0 beyond vd)
+        const float scale = differential_scale(p.diff, block_sum(fmaf(a[0], a[0], b[0] * b[0]), scratch), vd);
+        a[0] *= scale, b[0] *= scale;
     }
-    const float x = differential_value(p.diff, a[0], a[1]), y = differential_value(p.diff, b[0], b[1]);  // (0 beyond vd)
-    const float scale = differential_scale(p.diff, block_sum(fmaf(x, x, y * y), scratch), vd);
-    if (tid < vd) out[tid] = from_float<T>(x * scale);
-    if (tid + AS_THREADS < vd) out[tid + AS_THREADS] = from_float<T>(y * scale);
+    const float g = p.gate ? 1.0f / (1.0f + expf(-to_float(((const T *)p.gate)[(long long)t * p.ldg + h]))) : 1.0f;
+    if (tid < vd) out[tid] = from_float<T>(a[0] * g);
+    if (tid + AS_THREADS < vd) out[tid + AS_THREADS] = from_float<T>(b[0] * g);
 }
 
 // max_keys: an upper bound of the keys any row of the step sees (its position + 1, or window + keep_first);
-// parts: float32 scratch of at least tokens * heads * ceil(max_keys / 128) * (v_dim + 2) (for keys that carry their values
-// twice that: their parts may have 64 keys). to (null: none): the fold carries the heads' results out of the latent space.
+// parts: float32 scratch of at least tokens * heads * ceil(max_keys / 64) * (v_dim + 2). to (null: none): the fold carries the
+// heads' results out of the latent space.
 static int attention_split(const LatentOut *to, const DifferentialHead *diff, int values_in_keys, int chunk, float softcap, const void *q, long long q_row, void *out, int dtype, int n_tokens, int n_heads,
                                    int n_kv_heads, int head_dim, int v_dim, float scale, int window, int keep_first,
                                    const float *sink, const int *token_seq, const int *token_pos, const int *seq_slot,
@@ -604,11 +623,14 @@ static int attention_split(const LatentOut *to, const DifferentialHead *diff, in
     p.cache.page_table = page_table, p.cache.table_width = table_width, p.cache.ring_pages = ring_pages;
     p.cache.tokens_per_page = tokens_per_page, p.cache.pinned_pages = pinned_pages;
     p.v_cache = p.cache;
-    const bool tensor = dtype == ABK_BF16 && values_in_keys && head_dim % 16 == 0 && v_dim % 8 == 0 && q_row % 8 == 0 &&
-                        !(((uintptr_t)k_pool | (uintptr_t)q) & 15);
+    // (with values of their own and few heads to a kv head the other kernel's smaller CTAs do as well or better: 64 rows of 2,176
+    // keys, groups of two, 195 us against 257)
+    const bool tensor = dtype == ABK_BF16 && (values_in_keys || maps == 2 || n_heads / n_kv_heads >= 8) && maps * head_dim % 16 == 0 && v_dim % 8 == 0 && q_row % 8 == 0 &&
+                        !(((uintptr_t)k_pool | (uintptr_t)v_pool | (uintptr_t)q) & 15);
     if (to && (!tensor || ((uintptr_t)to->w & 15))) ABK_REFUSE("attention_split: latents of %d in rows of %d are not what the fused fold takes", v_dim, head_dim);
-    // parts of 64 keys where parts of 128 would not fill the GPU
-    p.part_keys = tensor && (long long)n_tokens * n_kv_heads * ((max_keys + 127) / 128) < 2 * abk_sm_count() ? 64 : 128;
+    // parts of 64 keys where values have rows of their own (more CTAs to an SM: 64 rows of 2,176 keys, two maps a head, 212 us against
+    // 270), and over latent rows where parts of 128 would not fill the GPU
+    p.part_keys = tensor && (!values_in_keys || (long long)n_tokens * n_kv_heads * ((max_keys + 127) / 128) < 2 * abk_sm_count()) ? 64 : 128;
     p.n_parts = (max_keys + p.part_keys - 1) / p.part_keys;
     p.values_in_keys = values_in_keys, p.runs = runs, p.gate = gate, p.ldg = ldg;
     p.maps = maps, p.diff = diff ? *diff : DifferentialHead();
@@ -647,14 +669,20 @@ static int attention_split(const LatentOut *to, const DifferentialHead *diff, in
         else SPLIT_LAUNCH(T, STAGED, 16);           \
     } while (0)
     if (tensor) {
-        const size_t bytes = (16 * (p.part_keys + 8) + 128) * 4 + (size_t)(16 + p.part_keys) * (head_dim * 2 + 16);
-        const void *kernel = p.part_keys == 64 ? (const void *)attention_split_latent_kernel<64> : (const void *)attention_split_latent_kernel<128>;
-        if (bytes + 4096 > 48 * 1024) {
-            cudaError_t e = abk_allow_shared_memory(kernel, (int)bytes);
-            if (e != cudaSuccess) return (int)e;
-        }
-        if (p.part_keys == 64) abk_launch(attention_split_latent_kernel<64>, grid, dim3(AS_THREADS), bytes, s, p);
-        else abk_launch(attention_split_latent_kernel<128>, grid, dim3(AS_THREADS), bytes, s, p);
+        const int v_pitch = values_in_keys ? 0 : ((v_dim + 15) & ~15) * 2 + 16;
+        const size_t bytes = (16 * (p.part_keys + 8) + 128) * 4 + (size_t)(16 + p.part_keys) * (maps * head_dim * 2 + 16) + (size_t)p.part_keys * v_pitch;
+#define TILES_LAUNCH(PART, OWN_V)                                                                                             \
+    do {                                                                                                                      \
+        if (bytes + 4096 > 48 * 1024) {                                                                                       \
+            cudaError_t e = abk_allow_shared_memory((const void *)attention_split_tiles_kernel<PART, OWN_V>, (int)bytes);     \
+            if (e != cudaSuccess) return (int)e;                                                                              \
+        }                                                                                                                     \
+        abk_launch(attention_split_tiles_kernel<PART, OWN_V>, grid, dim3(AS_THREADS), bytes, s, p);                           \
+    } while (0)
+        if (!values_in_keys) TILES_LAUNCH(64, true);
+        else if (p.part_keys == 64) TILES_LAUNCH(64, false);
+        else TILES_LAUNCH(128, false);
+#undef TILES_LAUNCH
         if (to) {
             LatentOut l = *to;
             l.n_rows = n_tokens;
@@ -674,12 +702,12 @@ static int attention_split(const LatentOut *to, const DifferentialHead *diff, in
     int rc = ABK_LAUNCH_RESULT();
     if (rc) return rc;
     if (maps == 2) {
-        if (bf) abk_launch(attention_fold_maps_kernel<__nv_bfloat16>, fold, dim3(AS_THREADS), 0, s, p);
-        else abk_launch(attention_fold_maps_kernel<float>, fold, dim3(AS_THREADS), 0, s, p);
-        return ABK_LAUNCH_RESULT();
+        if (bf) abk_launch(attention_fold_kernel<__nv_bfloat16, 2>, fold, dim3(AS_THREADS), 0, s, p);
+        else abk_launch(attention_fold_kernel<float, 2>, fold, dim3(AS_THREADS), 0, s, p);
+    } else {
+        if (bf) abk_launch(attention_fold_kernel<__nv_bfloat16, 1>, fold, dim3(AS_THREADS), 0, s, p);
+        else abk_launch(attention_fold_kernel<float, 1>, fold, dim3(AS_THREADS), 0, s, p);
     }
-    if (bf) abk_launch(attention_fold_kernel<__nv_bfloat16>, fold, dim3(AS_THREADS), 0, s, p);
-    else abk_launch(attention_fold_kernel<float>, fold, dim3(AS_THREADS), 0, s, p);
     return ABK_LAUNCH_RESULT();
 }
 

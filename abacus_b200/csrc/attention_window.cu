@@ -87,11 +87,12 @@ template <int MAPS> __device__ __forceinline__ void attention_window_cta(const A
     const uint32_t v_s = k_s + p.stages * AW_KEYS * pitch_k;        // p.stages stages
     const int warp = (threadIdx.x >> 5) & 3, map = MAPS == 2 ? threadIdx.x >> 7 : 0, lane = threadIdx.x & 31, g = lane >> 2, c2 = (lane & 3) * 2;
     const int slices = MAPS == 2 ? p.head_dim / 16 : d16 / 16, slice0 = map * slices * 32;  // 16-column steps of a map; its first byte of a row
-    const int h = blockIdx.y, kvh = h / (p.n_heads / p.n_kv_heads);
+    // the CTAs in the order they start: a sequence's last tiles, which see the most keys, first, all heads of a tile together
+    const int order = blockIdx.y * gridDim.x + blockIdx.x, h = order % p.n_heads, kvh = h / (p.n_heads / p.n_kv_heads);
     const float sink2 = p.sink ? p.sink[MAPS * h + map] * 1.4426950408889634f : -INFINITY;  // a weight: ahead of the wait
     pdl_wait();
     // which sequence and which of its tiles of 64 rows this CTA has
-    int seq = -1, tile = blockIdx.x, start = 0, n = 0;
+    int seq = -1, tile = (int)gridDim.x - 1 - order / p.n_heads, start = 0, n = 0;
     for (int s = 0; s < p.n_seqs; s++) {
         start = p.seq_start[s], n = p.seq_start[s + 1] - start;
         const int tiles = (n + AW_ROWS - 1) / AW_ROWS;

@@ -519,7 +519,7 @@ def attention_window(qkv, out, n_heads, n_kv_heads, head_dim, scale, window, bat
 def attention_split(qkv, out, n_heads, n_kv_heads, head_dim, scale, window, batch, cache, ws, v_dim=None, keep_first=0,
                     sink=None, row=None, max_keys=None, chunk=None, softcap=None, gate=None):
     """One new token per sequence against the paged cache with the general options (see attention_generic), split
-    along the keys into parts of 128 that a second kernel folds (csrc/attention_split.cu); softmax weights float32.
+    along the keys into parts of 64 or 128 that a second kernel folds (csrc/attention_split.cu); softmax weights float32.
     max_keys bounds the keys a row sees (by default the window and its kept keys, or the step's position bound).
     gate (of qkv's type, [rows, >= heads]): head h of row t is multiplied by sigmoid(gate[t, h]) where the parts are folded."""
     _need_cuda(qkv, out, sink, gate)
@@ -538,7 +538,7 @@ def attention_split(qkv, out, n_heads, n_kv_heads, head_dim, scale, window, batc
         max_keys = min(top, window + (keep_first or 0)) if window else top
         if chunk:
             max_keys = min(max_keys, chunk)
-    n_parts = -(-max_keys // 128)
+    n_parts = -(-max_keys // 64)
     parts = ws.get("attention_parts", (n * n_heads * n_parts * (vd + 2),), torch.float32)
     _check(lib, lib.abk_attention_split(
         _p(qkv), _ll(row), _p(out), _i(_dt(qkv)), _i(n), _i(n_heads), _i(n_kv_heads), _i(head_dim), _i(vd), _f(scale),
@@ -1165,7 +1165,7 @@ def attention_differential(qkv, out, n_heads, n_kv_heads, head_dim, scale, windo
         if batch.max_len_after > top:
             raise KernelError(f"a row at position {batch.max_len_after - 1} is beyond the bound {top}")
         max_keys = min([top] + [limit for limit in (window, chunk) if limit])
-        parts = ws.get("attention_parts", (n * 2 * n_heads * -(-max_keys // 128) * (vd + 2),), torch.float32)
+        parts = ws.get("attention_parts", (n * 2 * n_heads * -(-max_keys // 64) * (vd + 2),), torch.float32)
         _check(lib, lib.abk_attention_split_maps(
             _p(qkv), _ll(row), _p(out), _i(_dt(qkv)), _i(n), _i(2 * n_heads), _i(n_kv_heads), _i(head_dim), _i(vd), _f(scale),
             _i(window or 0), _i(0), _p(sink), _p(batch.token_seq), _p(batch.token_pos), _p(batch.seq_slot), _p(cache.k),
